@@ -4,14 +4,17 @@ from __future__ import annotations
 import ctypes
 import os
 import threading
+from typing import Optional
 
 _HERE = os.path.dirname(os.path.abspath(__file__))
 _LIB_PATH = os.path.join(_HERE, "libscratchy_cuda.so")
+_MODELS_PATH = os.path.join(_HERE, "libscratchy_models.so")
 
 OK = 0
 STATUS = {0: "SCR_OK", -1: "SCR_E_ARG", -2: "SCR_E_SHAPE", -3: "SCR_E_ALIGN", -4: "SCR_E_DTYPE", -5: "SCR_E_CUDA",
           -6: "SCR_E_WORKSPACE", -7: "SCR_E_UNSUPPORTED", -8: "SCR_E_TIMEOUT", -9: "SCR_E_COMM"}
 DTYPE_F16, DTYPE_BF16 = 0, 1     # the reference's DType discriminants (crates/tensors/src/dtype.rs:7-16)
+DTYPE_F32 = 2
 KIND_AFFINE_B4 = 0
 KIND_FP8_DYNAMIC = 1
 
@@ -90,6 +93,27 @@ SIGNATURES = {
     "scr_argmax_bf16": (_i32, [_vp, _vp, _i64, _i32, _i32, _vp, _vp]),
 }
 
+# the context functions every library of the package exports
+CONTEXT_SIGNATURES = {name: SIGNATURES[name] for name in ("scr_status_string", "scr_last_error", "scr_cuda_init", "scr_cuda_destroy",
+                                                          "scr_launch_count", "scr_device_status")}
+# name -> (restype, argtypes); one row per declaration in include/scratchy_models.h
+MODELS_SIGNATURES = {
+    "scr_dense_workspace_size": (_i32, [_i32, _i32, _i32, _i32, _i32, _psz]),
+    "scr_dense_linear": (_i32, [_vp, _i32, _vp, _vp, _sz, _vp]),
+    "scr_seq_embed": (_i32, [_vp, _i32, _vp, _i32, _vp, _i32, _i32, _vp, _vp, _i64, _vp]),
+    "scr_seq_norm": (_i32, [_vp, _i32, _vp, _vp]),
+    "scr_seq_argmax": (_i32, [_vp, _vp, _i64, _i32, _i32, _vp, _vp]),
+    "scr_latent_prepare": (_i32, [_vp, _i32, _vp, _vp, _vp, _i64, _vp, _vp, _vp, _vp, _vp, _vp, _vp]),
+    "scr_latent_queries": (_i32, [_vp, _i32, _vp, _vp, _vp, _vp, _vp, _vp, _i64, _i64, _vp, _i64, _i64, _vp]),
+    "scr_latent_attention_workspace": (_i32, [_i32, _vp, _vp, _psz]),
+    "scr_latent_attention": (_i32, [_vp, _i32, _vp, _vp, _vp, _vp, _vp, _vp, _sz, _vp]),
+    "scr_latent_prefill_supported": (_i32, [_vp]),
+    "scr_latent_gather": (_i32, [_vp, _vp, _vp, _i32, _vp, _vp, _vp, _vp]),
+    "scr_latent_prefill": (_i32, [_vp, _vp, _vp, _vp, _vp, _vp, _i64, _vp, _i64, _i32, _i32, _vp, _i64, _vp]),
+    "scr_mlstm_run": (_i32, [_vp, _i32, _vp, _vp, _vp, _i64, _vp, _i64, _vp, _vp, _vp, _vp, _vp, _vp, _vp]),
+    "scr_mlstm_finish": (_i32, [_vp, _i32, _vp, _vp, _vp, _vp, _i64, _i32, _vp, _vp]),
+}
+
 
 
 class QmvEnds(ctypes.Structure):
@@ -103,7 +127,41 @@ class TapeLinear(ctypes.Structure):
     _fields_ = [("packed", _vp), ("x", _vp), ("y", _vp), ("N", _i32), ("K", _i32), ("group", _i32), ("dep", _i32 * 3)]
 
 
+class Dense(ctypes.Structure):
+    """`scr_dense` of include/scratchy_models.h."""
+    _fields_ = [("w", _vp), ("x", _vp), ("y", _vp), ("y2", _vp), ("gate", _vp), ("ldx", _i64), ("x_group", _i64), ("ldy", _i64),
+                ("y_group", _i64), ("ldy2", _i64), ("ldg", _i64), ("M", _i32), ("N", _i32), ("K", _i32), ("groups", _i32),
+                ("n_main", _i32), ("y_f32", _i32), ("act", _i32), ("limit", ctypes.c_float), ("alpha", ctypes.c_float)]
+
+
+class SeqNorm(ctypes.Structure):
+    """`scr_seq_norm_args` of include/scratchy_models.h."""
+    _fields_ = [("x", _vp), ("delta", _vp), ("w_delta", _vp), ("bias", _vp), ("w_out", _vp), ("out", _vp), ("row_index", _vp),
+                ("ld_out", _i64), ("rows", _i32), ("x_rows", _i32), ("width", _i32), ("eps", ctypes.c_float)]
+
+
+class LatentShape(ctypes.Structure):
+    """`scr_latent_shape` of include/scratchy_models.h."""
+    _fields_ = [(n, _i32) for n in ("heads", "dim", "rot_dim", "vdim", "kv_rank", "q_rank", "rot_dims", "max_pos", "block_size",
+                                    "num_blocks", "max_blocks")] + [("eps", ctypes.c_float), ("scale", ctypes.c_float)]
+
+
+class Step(ctypes.Structure):
+    """`scr_step` of include/scratchy_models.h."""
+    _fields_ = [(n, _vp) for n in ("tok_seg", "tok_pos", "segs", "block_table")] + \
+               [(n, _i32) for n in ("rows", "batch", "max_count", "max_kv", "num_slots")]
+
+
+class MlstmShape(ctypes.Structure):
+    """`scr_mlstm_shape` of include/scratchy_models.h."""
+    _fields_ = [("heads", _i32), ("dim", _i32), ("vdim", _i32), ("gate_cap", ctypes.c_float), ("eps", ctypes.c_float)]
+
+
+MODELS_STRUCTS = {"scr_dense": Dense, "scr_seq_norm_args": SeqNorm, "scr_latent_shape": LatentShape, "scr_step": Step,
+                  "scr_mlstm_shape": MlstmShape}
+
 _lib = None
+_models = None
 _lock = threading.Lock()
 
 
@@ -123,12 +181,33 @@ def lib() -> ctypes.CDLL:
     return _lib
 
 
-class Context:
-    """Owns one ``scr_ctx`` (one per device).  ``check`` turns a status into an exception."""
+def models_lib(build: bool = False) -> ctypes.CDLL:
+    """The sequence-model library.  `build`: compile it first where it is missing or older than its sources (what a
+    command-line program of a source checkout does); otherwise a missing library raises."""
+    global _models
+    with _lock:
+        if _models is None:
+            if build:
+                from .build import MODELS_LIB, build_library
+                build_library(MODELS_LIB)
+            if not os.path.exists(_MODELS_PATH):
+                raise ScratchyCudaError(-5, f"{_MODELS_PATH} is missing: run `python -m scratchy_b200.build` "
+                                            "(there is no CPU fallback)")
+            L = ctypes.CDLL(_MODELS_PATH)
+            for name, (res, args) in {**CONTEXT_SIGNATURES, **MODELS_SIGNATURES}.items():
+                fn = getattr(L, name)
+                fn.restype, fn.argtypes = res, args
+            _models = L
+    return _models
 
-    def __init__(self, device: int = 0):
+
+class Context:
+    """Owns one ``scr_ctx`` (one per device and library).  ``check`` turns a status into an exception."""
+
+    def __init__(self, device: int = 0, library: Optional[ctypes.CDLL] = None):
         self._h = _vp()
-        st = lib().scr_cuda_init(int(device), ctypes.byref(self._h))
+        self._lib = library if library is not None else lib()
+        st = self._lib.scr_cuda_init(int(device), ctypes.byref(self._h))
         if st != OK:
             raise ScratchyCudaError(st, f"scr_cuda_init(device={device})")
         self.device = int(device)
@@ -139,19 +218,19 @@ class Context:
 
     def check(self, status: int) -> None:
         if status != OK:
-            detail = lib().scr_last_error(self._h)
+            detail = self._lib.scr_last_error(self._h)
             raise ScratchyCudaError(status, detail.decode() if detail else "")
 
     def device_status(self, stream=None) -> None:
         """Synchronise and raise if a bounded device-side wait ran out (`scr_device_status`)."""
-        self.check(lib().scr_device_status(self._h, stream, None))
+        self.check(self._lib.scr_device_status(self._h, stream, None))
 
     def launch_count(self) -> int:
-        return int(lib().scr_launch_count(self._h))
+        return int(self._lib.scr_launch_count(self._h))
 
     def close(self) -> None:
         if self._h:
-            lib().scr_cuda_destroy(self._h)
+            self._lib.scr_cuda_destroy(self._h)
             self._h = _vp()
 
     def __del__(self):
@@ -173,3 +252,15 @@ def context(device: int) -> Context:
         with _lock:
             _contexts[device] = c
     return c
+
+
+_models_contexts: dict[int, Context] = {}
+
+
+def models_context(device: int) -> Context:
+    """Process-wide context of ``device`` in the sequence-model library."""
+    library = models_lib()
+    with _lock:
+        if device not in _models_contexts:
+            _models_contexts[device] = Context(device, library)
+        return _models_contexts[device]

@@ -1,7 +1,9 @@
-"""Builds ``libscratchy_cuda.so`` (the C-ABI library) in-tree with nvcc for sm_100a.
+"""Builds the C-ABI libraries in-tree with nvcc for sm_100a: ``libscratchy_cuda.so`` (quantized linears and the Llama
+decode step) and ``libscratchy_models.so`` (the sequence-model kernels).
 
 Usage: ``python -m scratchy_b200.build [--force] [--verbose]``.  nvcc cross-compiles
-without a GPU; the resulting shared object sits beside this file.
+without a GPU; the resulting shared objects sit beside this file.  A program that needs one library only builds that
+one (`build_library`), so its first call compiles no more than it uses.
 """
 from __future__ import annotations
 
@@ -14,8 +16,12 @@ HERE = os.path.dirname(os.path.abspath(__file__))
 CSRC = os.path.join(HERE, "csrc")
 OBJ = os.path.join(CSRC, "build")
 LIB = os.path.join(HERE, "libscratchy_cuda.so")
+MODELS_LIB = os.path.join(HERE, "libscratchy_models.so")
 
-SOURCES = ["abi.cu", "affine_b4.cu", "affine_b4_gemm.cu", "affine_b4_gemm_pair.cu", "fp8.cu", "fp8_gemm.cu", "fp8_gemm_pair.cu", "decode_ops.cu", "tp_comm.cu"]
+SOURCES = ["context.cu", "abi.cu", "affine_b4.cu", "affine_b4_gemm.cu", "affine_b4_gemm_pair.cu", "fp8.cu", "fp8_gemm.cu", "fp8_gemm_pair.cu", "decode_ops.cu", "tp_comm.cu"]
+MODELS_SOURCES = ["context.cu", "dense_linear.cu", "dense_gemm.cu", "seq_ops.cu", "latent_attention.cu", "latent_attention_mma.cu",
+                  "latent_prefill.cu", "mlstm.cu", "mlstm_chunk.cu"]
+LIBRARIES = {LIB: SOURCES, MODELS_LIB: MODELS_SOURCES}
 
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
@@ -38,11 +44,21 @@ def _newer(target: str, deps: list[str]) -> bool:
 
 
 def build(force: bool = False, verbose: bool = False) -> str:
+    """Every library of the package."""
+    for target in LIBRARIES:
+        build_library(target, force, verbose)
+    return LIB
+
+
+def build_library(target: str, force: bool = False, verbose: bool = False) -> str:
     nvcc = _nvcc()
     os.makedirs(OBJ, exist_ok=True)
     headers = [os.path.join(CSRC, f) for f in os.listdir(CSRC) if f.endswith((".cuh", ".h"))]
-    headers.append(os.path.join(os.path.dirname(HERE), "include", "scratchy_cuda.h"))
-    sources = [s for s in SOURCES if os.path.exists(os.path.join(CSRC, s))]
+    include = os.path.join(os.path.dirname(HERE), "include")
+    headers += [os.path.join(include, f) for f in os.listdir(include) if f.endswith(".h")]
+    sources = [s for s in LIBRARIES[target] if os.path.exists(os.path.join(CSRC, s))]
+    if not force and _newer(target, headers + [os.path.join(CSRC, s) for s in sources]):
+        return target
     objs = []
     procs = []
     for src in sources:
@@ -66,10 +82,10 @@ def build(force: bool = False, verbose: bool = False) -> str:
             sys.stderr.write(f"--- {src}\n{out}\n")
     if failed:
         raise RuntimeError("nvcc failed")
-    if force or procs or not _newer(LIB, objs):
-        subprocess.check_call([nvcc, "-shared", "-o", LIB, *objs, "-gencode", "arch=compute_100a,code=sm_100a",
+    if force or procs or not _newer(target, objs):
+        subprocess.check_call([nvcc, "-shared", "-o", target, *objs, "-gencode", "arch=compute_100a,code=sm_100a",
                                "-Xcompiler", "-fPIC"])
-    return LIB
+    return target
 
 
 if __name__ == "__main__":

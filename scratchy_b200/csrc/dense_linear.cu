@@ -1,0 +1,201 @@
+// Full-precision linears of the sequence models: y = x W^T with the ends of `scr_dense`.
+//
+//   M <= 16, bf16   dense_matvec_kernel   weights streamed once from HBM straight into mma.sync fragments (decode)
+//   M > 16, bf16    dense_gemm.cu         tcgen05 GEMM
+//   otherwise       dense_plain_kernel    f32 arithmetic on any sizes (the f32 data type; bf16 rows that are not a
+//                                         multiple of 16 bytes)
+#include "seq_common.cuh"
+
+#include <algorithm>
+
+size_t dense_gemm_workspace(int M, int N, int K, int groups);
+int32_t dense_gemm_launch(scr_ctx* ctx, const scr_dense& d, void* workspace, size_t workspace_bytes, cudaStream_t stream);
+
+namespace {
+
+// ------------------------------------------------------------------------------- any size, f32 arithmetic
+// 64 rows x 64 columns per CTA, 4 x 4 per thread.  A thread's columns are 8 apart, so a gate column and its up column
+// (8 further on) belong to one thread.
+constexpr int PLAIN_T = 64, PLAIN_K = 16;
+
+template <typename T>
+__global__ void __launch_bounds__(256) dense_plain_kernel(const T* __restrict__ w, const T* __restrict__ x, long long ldx,
+                                                          long long x_group, int M, int N, int K, DenseEnds ends) {
+    __shared__ float xs[PLAIN_K][PLAIN_T + 4], ws[PLAIN_K][PLAIN_T + 4];
+    pdl_trigger();
+    pdl_wait();
+    const int g = blockIdx.z, m0 = blockIdx.y * PLAIN_T, n0 = blockIdx.x * PLAIN_T;
+    const int ty = threadIdx.x >> 4, tx = threadIdx.x & 15;
+    const int cbase = (tx >> 3) * 32 + (tx & 7);
+    w += (size_t)g * N * K;
+    x += g * x_group;
+    float acc[4][4] = {};
+    for (int k0 = 0; k0 < K; k0 += PLAIN_K) {
+        for (int i = threadIdx.x; i < PLAIN_T * PLAIN_K; i += 256) {
+            const int r = i >> 4, k = i & 15;
+            xs[k][r] = (m0 + r < M && k0 + k < K) ? to_f32(x[(m0 + r) * ldx + k0 + k]) : 0.0f;
+            ws[k][r] = (n0 + r < N && k0 + k < K) ? to_f32(w[(size_t)(n0 + r) * K + k0 + k]) : 0.0f;
+        }
+        __syncthreads();
+#pragma unroll
+        for (int k = 0; k < PLAIN_K; ++k) {
+            float a[4], b[4];
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                a[i] = xs[k][ty * 4 + i];
+                b[i] = ws[k][cbase + 8 * i];
+            }
+#pragma unroll
+            for (int i = 0; i < 4; ++i)
+#pragma unroll
+                for (int j = 0; j < 4; ++j) acc[i][j] = fmaf(a[i], b[j], acc[i][j]);
+        }
+        __syncthreads();
+    }
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+        const int m = m0 + ty * 4 + i;
+        if (m >= M) continue;
+        if (ends.act) {
+#pragma unroll
+            for (int j = 0; j < 4; j += 2)
+                if (n0 + cbase + 8 * j < N) dense_put_pair<T>(ends, m, n0 + cbase + 8 * j, acc[i][j], acc[i][j + 1]);
+        } else {
+#pragma unroll
+            for (int j = 0; j < 4; ++j)
+                if (n0 + cbase + 8 * j < N) dense_put<T>(ends, m, g, n0 + cbase + 8 * j, acc[i][j]);
+        }
+    }
+}
+
+// ------------------------------------------------------------------------------- decode matvec
+// A tile is 16 weight rows over the whole K, shared by `wpt` warps that take 64-wide units of K in turn.  In a unit lane
+// (g, t) loads the 16-byte pieces [t*8, t*8+8) and [32 + t*8, ..) of rows g and g + 8, and the same pieces of
+// activation row g: the k order inside a fragment is a permutation both operands share, so the loaded registers are
+// mma operands as they stand (weights = A, 8 tokens per B).  The first pieces of the weights, load-time constants, are
+// requested before the wait for the preceding kernel.  Partial sums of the warps meet in shared memory in warp order.
+constexpr int MV_WARPS = 8, MV_UNROLL = 3;
+
+template <int NT>
+__global__ void __launch_bounds__(MV_WARPS * 32) dense_matvec_kernel(const bf16* __restrict__ w, const bf16* __restrict__ x,
+                                                                     long long ldx, long long x_group, int M, int N, int K,
+                                                                     int wpt, DenseEnds ends) {
+    __shared__ float red[MV_WARPS][16][8 * NT + 1];
+    pdl_trigger();
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
+    const int tiles = MV_WARPS / wpt, part = warp % wpt, grp = blockIdx.y;
+    const int n0 = (blockIdx.x * tiles + warp / wpt) * 16;
+    const int units = (K + 63) >> 6;
+    const bf16* w0 = w + ((size_t)grp * N + min(n0 + g, N - 1)) * K + t * 8;
+    const bf16* w1 = w + ((size_t)grp * N + min(n0 + g + 8, N - 1)) * K + t * 8;
+    uint4 wa[MV_UNROLL][2], wb[MV_UNROLL][2];
+    auto load_w = [&](int u0) {
+#pragma unroll
+        for (int u = 0; u < MV_UNROLL; ++u)
+#pragma unroll
+            for (int h = 0; h < 2; ++h) {
+                const int k = (u0 + u * wpt) * 64 + h * 32;
+                const bool ok = k + t * 8 < K;
+                wa[u][h] = ok ? ld_stream_v4(w0 + k) : make_uint4(0, 0, 0, 0);
+                wb[u][h] = ok ? ld_stream_v4(w1 + k) : make_uint4(0, 0, 0, 0);
+            }
+    };
+    float acc[NT][4] = {};
+    load_w(part);
+    pdl_wait();
+    x += grp * x_group + t * 8;
+    for (int u0 = part; u0 < units; u0 += MV_UNROLL * wpt) {
+        if (u0 != part) load_w(u0);
+#pragma unroll
+        for (int u = 0; u < MV_UNROLL; ++u)
+#pragma unroll
+            for (int h = 0; h < 2; ++h) {
+                const int k = (u0 + u * wpt) * 64 + h * 32;
+#pragma unroll
+                for (int nt = 0; nt < NT; ++nt) {
+                    uint4 xv = make_uint4(0, 0, 0, 0);
+                    if (nt * 8 + g < M && k + t * 8 < K) xv = ld_act_v4(x + (nt * 8 + g) * ldx + k);
+                    mma_16816(acc[nt], wa[u][h].x, wb[u][h].x, wa[u][h].y, wb[u][h].y, xv.x, xv.y);
+                    mma_16816(acc[nt], wa[u][h].z, wb[u][h].z, wa[u][h].w, wb[u][h].w, xv.z, xv.w);
+                }
+            }
+    }
+#pragma unroll
+    for (int nt = 0; nt < NT; ++nt) {
+        red[warp][g][nt * 8 + 2 * t] = acc[nt][0];
+        red[warp][g][nt * 8 + 2 * t + 1] = acc[nt][1];
+        red[warp][g + 8][nt * 8 + 2 * t] = acc[nt][2];
+        red[warp][g + 8][nt * 8 + 2 * t + 1] = acc[nt][3];
+    }
+    __syncthreads();
+    auto total = [&](int tile, int r, int m) {
+        float v = 0.0f;
+        for (int p = 0; p < wpt; ++p) v += red[tile * wpt + p][r][m];
+        return v;
+    };
+    if (ends.act) {
+        for (int i = threadIdx.x; i < tiles * 8 * M; i += MV_WARPS * 32) {
+            const int r = i & 7, tile = (i >> 3) % tiles, m = (i >> 3) / tiles;
+            const int n = (blockIdx.x * tiles + tile) * 16 + r;
+            if (n < N) dense_put_pair<bf16>(ends, m, n, total(tile, r, m), total(tile, r + 8, m));
+        }
+    } else {
+        for (int i = threadIdx.x; i < tiles * 16 * M; i += MV_WARPS * 32) {
+            const int r = i & 15, tile = (i >> 4) % tiles, m = (i >> 4) / tiles;
+            const int n = (blockIdx.x * tiles + tile) * 16 + r;
+            if (n < N) dense_put<bf16>(ends, m, grp, n, total(tile, r, m));
+        }
+    }
+}
+
+int32_t matvec_launch(scr_ctx* ctx, const scr_dense& d, cudaStream_t stream) {
+    const int units = (d.K + 63) / 64, tiles16 = (d.N + 15) / 16;
+    // warps per tile: enough units of K for each, and enough CTAs to fill the GPU
+    int wpt = 1;
+    while (wpt < MV_WARPS && (units >= 4 * wpt || (units >= 2 * wpt && (tiles16 * d.groups * wpt) / MV_WARPS < 2 * ctx->sm_count))) wpt *= 2;
+    const dim3 grid(scr_ceil_div(tiles16, MV_WARPS / wpt), d.groups);
+    const bf16 *w = (const bf16*)d.w, *x = (const bf16*)d.x;
+    const DenseEnds e = dense_ends(d);
+    const cudaError_t err = d.M <= 8 ? launch_pdl(dense_matvec_kernel<1>, grid, dim3(MV_WARPS * 32), 0, stream, w, x, (long long)d.ldx, (long long)d.x_group, d.M, d.N, d.K, wpt, e)
+                                     : launch_pdl(dense_matvec_kernel<2>, grid, dim3(MV_WARPS * 32), 0, stream, w, x, (long long)d.ldx, (long long)d.x_group, d.M, d.N, d.K, wpt, e);
+    if (err != cudaSuccess) return scr_fail(ctx, SCR_E_CUDA, "dense_matvec: %s", cudaGetErrorString(err));
+    return scr_check_launch(ctx, "dense_matvec");
+}
+
+template <typename T>
+int32_t plain_launch(scr_ctx* ctx, const scr_dense& d, cudaStream_t stream) {
+    const dim3 grid(scr_ceil_div(d.N, PLAIN_T), scr_ceil_div(d.M, PLAIN_T), d.groups);
+    const cudaError_t err = launch_pdl(dense_plain_kernel<T>, grid, dim3(256), 0, stream, (const T*)d.w, (const T*)d.x,
+                                       (long long)d.ldx, (long long)d.x_group, d.M, d.N, d.K, dense_ends(d));
+    if (err != cudaSuccess) return scr_fail(ctx, SCR_E_CUDA, "dense_plain: %s", cudaGetErrorString(err));
+    return scr_check_launch(ctx, "dense_plain");
+}
+
+bool rows_of_16_bytes(const scr_dense& d) {
+    return d.K % 8 == 0 && d.ldx % 8 == 0 && d.x_group % 8 == 0 && scr_aligned16(d.w) && scr_aligned16(d.x);
+}
+
+}  // namespace
+
+extern "C" int32_t scr_dense_workspace_size(int32_t dtype, int32_t M, int32_t N, int32_t K, int32_t groups, size_t* bytes) {
+    if (!bytes) return SCR_E_ARG;
+    if (M <= 0 || N <= 0 || K <= 0 || groups <= 0) return SCR_E_SHAPE;
+    *bytes = (dtype == SCR_DTYPE_BF16 && M > 16) ? dense_gemm_workspace(M, N, K, groups) : 0;
+    return SCR_OK;
+}
+
+extern "C" int32_t scr_dense_linear(scr_ctx* ctx, int32_t dtype, const scr_dense* dp, void* workspace, size_t workspace_bytes,
+                                    void* stream) {
+    SCR_REQUIRE_CTX(ctx);
+    if (!dp || !dp->w || !dp->x || !dp->y) return scr_fail(ctx, SCR_E_ARG, "null pointer");
+    const scr_dense& d = *dp;
+    if (d.M <= 0 || d.N <= 0 || d.K <= 0 || d.groups <= 0) return scr_fail(ctx, SCR_E_SHAPE, "empty linear (M %d N %d K %d)", d.M, d.N, d.K);
+    if (d.n_main < d.N && (!d.y2 || d.groups != 1 || d.act)) return scr_fail(ctx, SCR_E_ARG, "a second output needs y2, one group and no activation");
+    if (d.act && (d.N % 16 || d.groups != 1 || d.gate)) return scr_fail(ctx, SCR_E_SHAPE, "gate/up pairs come in runs of 8 + 8 rows");
+    cudaStream_t st = (cudaStream_t)stream;
+    if (dtype == SCR_DTYPE_F32) return plain_launch<float>(ctx, d, st);
+    if (dtype != SCR_DTYPE_BF16) return scr_fail(ctx, SCR_E_DTYPE, "dtype %d", dtype);
+    if (!rows_of_16_bytes(d)) return plain_launch<bf16>(ctx, d, st);
+    if (d.M <= 16) return matvec_launch(ctx, d, st);
+    return dense_gemm_launch(ctx, d, workspace, workspace_bytes, st);
+}
