@@ -1,4 +1,340 @@
+// Latent attention for decoding and short portions, bf16, on mma.sync: the rows of a sequence are its tokens x heads, all
+// of which read the same cache rows [latent | rotated key part].
+//
+// A CTA takes 16 or 32 of those rows and a share of the keys.  Key tiles of 64 cache rows come through two shared-memory
+// stages (cp.async, one warp per row of the paged cache, the next tile in flight while this one is computed).  Per tile:
+// S = Q K^T with the key range dealt to the warps, scores to shared memory in f32; a softmax pass over the rows that keeps
+// the running maximum and sum in f32 and leaves P as a bf16 head and remainder (two products, so the weights keep about
+// 16 bits); O += P V with the latent columns dealt to the warps, V being the first kv_rank columns of the very tile.
+// Shares of the keys that other CTAs took meet in a second kernel.
 #include "seq_common.cuh"
-bool latent_attention_mma_applies(const scr_latent_shape&) { return false; }
-size_t latent_attention_mma_workspace(const scr_latent_shape&, const scr_step&, int) { return 0; }
-int32_t latent_attention_mma_launch(scr_ctx*, const scr_latent_shape&, const scr_step&, const void*, const void*, void*, void*, size_t, cudaStream_t) { return SCR_E_UNSUPPORTED; }
+
+#include <algorithm>
+
+namespace {
+
+constexpr int LM_THREADS = 256, LM_KEYS = 64, LM_P_LD = LM_KEYS + 8, LM_S_LD = LM_KEYS + 4;
+
+struct LmSmem {
+    int ld;                                                    // elements per row of Q and key tiles: odd multiple of 16 bytes
+    size_t q, tile, scores, p_hi, p_lo, corr, total;
+    static __host__ __device__ LmSmem of(int D, int mt) {
+        LmSmem s{};
+        s.ld = (D + 15) / 16 * 16 + 8;
+        s.q = 0;
+        s.tile = s.q + (size_t)mt * 16 * s.ld * 2;
+        s.scores = s.tile + 2 * (size_t)LM_KEYS * s.ld * 2;
+        s.p_hi = s.scores + (size_t)mt * 16 * LM_S_LD * 4;
+        s.p_lo = s.p_hi + (size_t)mt * 16 * LM_P_LD * 2;
+        s.corr = s.p_lo + (size_t)mt * 16 * LM_P_LD * 2;
+        s.total = s.corr + (size_t)mt * 16 * 4 * 2;
+        return s;
+    }
+};
+
+__device__ __forceinline__ void cp_async16(uint32_t dst, const void* src, bool ok) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(ok ? 16 : 0) : "memory");
+}
+__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+__device__ __forceinline__ void cp_async_wait_all() { asm volatile("cp.async.wait_group 0;" ::: "memory"); }
+__device__ __forceinline__ float exp2_fast(float x) {
+    float y;
+    asm volatile("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+
+// MT: 16-row tiles; NTW: 8-column tiles of the latent per warp (kv_rank <= 64 * NTW)
+template <int MT, int NTW>
+__global__ void __launch_bounds__(LM_THREADS) latent_attention_mma_kernel(scr_latent_shape s, scr_step st, const bf16* __restrict__ q,
+                                                                          const bf16* __restrict__ cache, bf16* __restrict__ out,
+                                                                          float* __restrict__ part_o, float* __restrict__ part_ml, int nsplit,
+                                                                          int* __restrict__ status) {
+    extern __shared__ __align__(128) unsigned char lm_smem[];
+    constexpr int ROWS = MT * 16, TPR = LM_THREADS / ROWS, KPT = LM_KEYS / TPR;      // softmax: threads per row, keys per thread
+    const int D = s.kv_rank + s.rot_dim;
+    const LmSmem lay = LmSmem::of(D, MT);
+    bf16* Q = reinterpret_cast<bf16*>(lm_smem + lay.q);
+    float* scores = reinterpret_cast<float*>(lm_smem + lay.scores);
+    bf16* p_hi = reinterpret_cast<bf16*>(lm_smem + lay.p_hi);
+    bf16* p_lo = reinterpret_cast<bf16*>(lm_smem + lay.p_lo);
+    float* corr = reinterpret_cast<float*>(lm_smem + lay.corr);                      // [ROWS] rescale, then [ROWS] final sums
+    pdl_trigger();
+    const int b = blockIdx.z, split = blockIdx.y, r0 = blockIdx.x * ROWS;
+    const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+    const int first = st.segs[b * 4], count = st.segs[b * 4 + 1], pos0 = st.segs[b * 4 + 2];
+    const int nrows = min(ROWS, count * s.heads - r0);
+    if (nrows <= 0 || first < 0 || first + count > st.rows) { pdl_wait(); return; }
+    int kv = pos0 + (r0 + nrows - 1) / s.heads + 1;                                  // keys the last row of this CTA sees
+    if (kv > s.max_blocks * s.block_size) {
+        if (threadIdx.x == 0) atomicCAS(status, 0, SEQ_BAD_POSITION);
+        kv = s.max_blocks * s.block_size;
+    }
+    const int tiles = (kv + LM_KEYS - 1) / LM_KEYS, per = (tiles + nsplit - 1) / nsplit;
+    const int t_lo = min(split * per, tiles), t_hi = min(t_lo + per, tiles);
+    const int* table = st.block_table + (size_t)b * s.max_blocks;
+    const int chunks = D / 8;
+    auto load_tile = [&](int t) {
+        bf16* dst = reinterpret_cast<bf16*>(lm_smem + lay.tile) + (size_t)((t - t_lo) & 1) * LM_KEYS * lay.ld;
+#pragma unroll 2
+        for (int i = 0; i < LM_KEYS / 8; ++i) {
+            const int key = t * LM_KEYS + warp * (LM_KEYS / 8) + i;
+            bool ok = key < kv;
+            int block = ok ? table[key / s.block_size] : 0;
+            if (block < 0 || block >= s.num_blocks) {
+                if (lane == 0) atomicCAS(status, 0, SEQ_BAD_BLOCK);
+                ok = false;
+                block = 0;
+            }
+            const bf16* src = cache + ((size_t)block * s.block_size + key % s.block_size) * D;
+            const uint32_t row = smem_u32(dst + (size_t)(warp * (LM_KEYS / 8) + i) * lay.ld);
+            for (int c = lane; c < chunks; c += 32) cp_async16(row + c * 16, src + (ok ? c * 8 : 0), ok);
+        }
+    };
+    // zero what a key row holds beyond D (the last k step may read it), in both stages and in Q
+    for (int i = threadIdx.x; i < (2 * LM_KEYS + ROWS) * (lay.ld - D); i += LM_THREADS) {
+        const int row = i / (lay.ld - D), c = D + i % (lay.ld - D);
+        (row < ROWS ? Q + (size_t)row * lay.ld : reinterpret_cast<bf16*>(lm_smem + lay.tile) + (size_t)(row - ROWS) * lay.ld)[c] = __float2bfloat16_rn(0.0f);
+    }
+    // cache rows before this step's are there already: their tile does not wait for the preceding kernels
+    const bool early = t_lo < t_hi && (t_lo + 1) * LM_KEYS <= pos0;
+    if (early) load_tile(t_lo);
+    pdl_wait();
+    if (!early && t_lo < t_hi) load_tile(t_lo);
+    for (int i = threadIdx.x; i < ROWS * chunks; i += LM_THREADS) {
+        const int row = i / chunks, c = i - row * chunks;
+        cp_async16(smem_u32(Q + (size_t)row * lay.ld + c * 8), q + ((size_t)first * s.heads + r0 + (row < nrows ? row : 0)) * D + c * 8, row < nrows);
+    }
+    cp_async_commit();
+
+    float acc[MT][NTW][4] = {};
+    const float sl2 = s.scale * 1.4426950408889634f;
+    const int srow = threadIdx.x / TPR, sk0 = (threadIdx.x % TPR) * KPT;              // this thread's softmax row and first key
+    const int limit = pos0 + (r0 + min(srow, nrows - 1)) / s.heads;                  // last key the row sees
+    float m_run = -INFINITY, l_run = 0.0f;
+    const int mt_s = warp % MT, ng = warp / MT;                                      // S phase: row tile, key group (8 * MT keys)
+    const int ksteps = (D + 15) / 16, lm = lane >> 3, lr = lane & 7;
+    for (int t = t_lo; t < t_hi; ++t) {
+        cp_async_wait_all();
+        __syncthreads();
+        if (t + 1 < t_hi) load_tile(t + 1);
+        cp_async_commit();
+        const bf16* K = reinterpret_cast<bf16*>(lm_smem + lay.tile) + (size_t)((t - t_lo) & 1) * LM_KEYS * lay.ld;
+        {
+            float sc[MT][4] = {};
+            const uint32_t qa = smem_u32(Q + (size_t)(mt_s * 16 + (lm & 1) * 8 + lr) * lay.ld + (lm >> 1) * 8);
+            const uint32_t kb = smem_u32(K + (size_t)(ng * 8 * MT + lr) * lay.ld + lm * 8);
+            for (int ks = 0; ks < ksteps; ks += 2) {                                 // (the row beyond D is zero up to ld)
+                uint32_t a0[4], a1[4] = {0, 0, 0, 0};
+                ldsm_x4(qa + ks * 32, a0);
+                if (ks + 1 < ksteps) ldsm_x4(qa + ks * 32 + 32, a1);
+#pragma unroll
+                for (int n = 0; n < MT; ++n) {
+                    uint32_t kf[4];
+                    if (ks + 1 < ksteps) {
+                        ldsm_x4(kb + n * 8 * lay.ld * 2 + ks * 32, kf);
+                    } else {                                                         // half of the pair only
+                        asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0,%1}, [%2];" : "=r"(kf[0]), "=r"(kf[1])
+                                     : "r"(smem_u32(K + (size_t)(ng * 8 * MT + n * 8 + lr) * lay.ld + (lm & 1) * 8) + ks * 32));
+                        kf[2] = kf[3] = 0;
+                    }
+                    mma_16816(sc[n], a0[0], a0[1], a0[2], a0[3], kf[0], kf[1]);
+                    if (ks + 1 < ksteps) mma_16816(sc[n], a1[0], a1[1], a1[2], a1[3], kf[2], kf[3]);
+                }
+            }
+            float* dst = scores + (size_t)(mt_s * 16 + (lane >> 2)) * LM_S_LD + ng * 8 * MT + (lane & 3) * 2;
+#pragma unroll
+            for (int n = 0; n < MT; ++n) {
+                *reinterpret_cast<float2*>(dst + n * 8) = make_float2(sc[n][0], sc[n][1]);
+                *reinterpret_cast<float2*>(dst + 8 * LM_S_LD + n * 8) = make_float2(sc[n][2], sc[n][3]);
+            }
+        }
+        __syncthreads();
+        {
+            float v[KPT], mx = -INFINITY;
+#pragma unroll
+            for (int i = 0; i < KPT; ++i) {
+                const int key = t * LM_KEYS + sk0 + i;
+                v[i] = key <= limit && key < kv ? scores[srow * LM_S_LD + sk0 + i] * sl2 : -INFINITY;
+                mx = fmaxf(mx, v[i]);
+            }
+#pragma unroll
+            for (int o = 1; o < TPR; o <<= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
+            const float mn = fmaxf(m_run, mx);
+            const float keep = m_run == -INFINITY ? 0.0f : exp2_fast(m_run - mn);
+            float sum = 0.0f;
+#pragma unroll
+            for (int i = 0; i < KPT; i += 2) {
+                const float p0 = v[i] == -INFINITY ? 0.0f : exp2_fast(v[i] - mn), p1 = v[i + 1] == -INFINITY ? 0.0f : exp2_fast(v[i + 1] - mn);
+                sum += p0 + p1;
+                const uint32_t hi = pack_bf16x2(p0, p1);
+                *reinterpret_cast<uint32_t*>(p_hi + srow * LM_P_LD + sk0 + i) = hi;
+                *reinterpret_cast<uint32_t*>(p_lo + srow * LM_P_LD + sk0 + i) = pack_bf16x2(p0 - bf16_lo(hi), p1 - bf16_hi(hi));
+            }
+#pragma unroll
+            for (int o = 1; o < TPR; o <<= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);
+            l_run = l_run * keep + sum;
+            m_run = mn;
+            if (sk0 == 0) corr[srow] = keep;
+        }
+        __syncthreads();
+#pragma unroll
+        for (int m = 0; m < MT; ++m) {
+            const float c0 = corr[m * 16 + (lane >> 2)], c1 = corr[m * 16 + (lane >> 2) + 8];
+#pragma unroll
+            for (int n = 0; n < NTW; ++n) {
+                acc[m][n][0] *= c0;
+                acc[m][n][1] *= c0;
+                acc[m][n][2] *= c1;
+                acc[m][n][3] *= c1;
+            }
+        }
+#pragma unroll
+        for (int k32 = 0; k32 < LM_KEYS / 32; ++k32) {
+            uint32_t ph[MT][2][4], pl[MT][2][4];
+#pragma unroll
+            for (int m = 0; m < MT; ++m)
+#pragma unroll
+                for (int h = 0; h < 2; ++h) {
+                    const size_t at = (size_t)(m * 16 + (lm & 1) * 8 + lr) * LM_P_LD + k32 * 32 + h * 16 + (lm >> 1) * 8;
+                    ldsm_x4(smem_u32(p_hi + at), ph[m][h]);
+                    ldsm_x4(smem_u32(p_lo + at), pl[m][h]);
+                }
+#pragma unroll
+            for (int n = 0; n < NTW; ++n) {
+                const int col = (warp * NTW + n) * 8;
+                if (col >= s.kv_rank) continue;                                      // (uniform over the warp)
+                uint32_t vf[4];
+                ldsm_x4_trans(smem_u32(K + (size_t)(k32 * 32 + lm * 8 + lr) * lay.ld + col), vf);
+#pragma unroll
+                for (int m = 0; m < MT; ++m) {
+                    mma_16816(acc[m][n], ph[m][0][0], ph[m][0][1], ph[m][0][2], ph[m][0][3], vf[0], vf[1]);
+                    mma_16816(acc[m][n], ph[m][1][0], ph[m][1][1], ph[m][1][2], ph[m][1][3], vf[2], vf[3]);
+                    mma_16816(acc[m][n], pl[m][0][0], pl[m][0][1], pl[m][0][2], pl[m][0][3], vf[0], vf[1]);
+                    mma_16816(acc[m][n], pl[m][1][0], pl[m][1][1], pl[m][1][2], pl[m][1][3], vf[2], vf[3]);
+                }
+            }
+        }
+    }
+    cp_async_wait_all();
+    const size_t all_rows = (size_t)st.rows * s.heads, row_base = (size_t)first * s.heads + r0;
+    if (sk0 == 0) {
+        corr[ROWS + srow] = l_run;
+        if (nsplit > 1 && srow < nrows) {
+            part_ml[((size_t)split * all_rows + row_base + srow) * 2] = m_run;
+            part_ml[((size_t)split * all_rows + row_base + srow) * 2 + 1] = l_run;
+        }
+    }
+    __syncthreads();
+#pragma unroll
+    for (int m = 0; m < MT; ++m)
+#pragma unroll
+        for (int hf = 0; hf < 2; ++hf) {
+            const int row = m * 16 + hf * 8 + (lane >> 2);
+            if (row >= nrows) continue;
+            const float inv = 1.0f / corr[ROWS + row];
+#pragma unroll
+            for (int n = 0; n < NTW; ++n) {
+                const int col = (warp * NTW + n) * 8 + (lane & 3) * 2;
+                if (col >= s.kv_rank) continue;
+                const float v0 = acc[m][n][hf * 2], v1 = acc[m][n][hf * 2 + 1];
+                if (nsplit > 1) *reinterpret_cast<float2*>(part_o + ((size_t)split * all_rows + row_base + row) * s.kv_rank + col) = make_float2(v0, v1);
+                else *reinterpret_cast<uint32_t*>(out + (row_base + row) * s.kv_rank + col) = pack_bf16x2(v0 * inv, v1 * inv);
+            }
+        }
+}
+
+// One CTA per row: the key shares' states into one.
+__global__ void __launch_bounds__(128) latent_attention_merge_kernel(const float* __restrict__ part_o, const float* __restrict__ part_ml,
+                                                                     int nsplit, long long all_rows, int kv_rank, bf16* __restrict__ out) {
+    __shared__ float w[64];
+    pdl_trigger();
+    pdl_wait();
+    const long long r = blockIdx.x;
+    if (threadIdx.x < 32) {
+        float m = -INFINITY, l = 0.0f;
+        for (int k = threadIdx.x; k < nsplit; k += 32) m = fmaxf(m, part_ml[(k * all_rows + r) * 2]);
+#pragma unroll
+        for (int o = 16; o > 0; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
+        for (int k = threadIdx.x; k < nsplit; k += 32) {
+            const float mk = part_ml[(k * all_rows + r) * 2], c = mk == -INFINITY ? 0.0f : exp2f(mk - m);
+            w[k] = c;
+            l += c * part_ml[(k * all_rows + r) * 2 + 1];
+        }
+        l = warp_sum(l);
+        __syncwarp();
+        for (int k = threadIdx.x; k < nsplit; k += 32) w[k] = l > 0.0f ? w[k] / l : 0.0f;
+    }
+    __syncthreads();
+    for (int i = threadIdx.x * 2; i < kv_rank; i += 256) {
+        float a = 0.0f, b = 0.0f;
+        for (int k = 0; k < nsplit; ++k)
+            if (w[k] != 0.0f) {                              // (a share without keys)
+                const float2 v = *reinterpret_cast<const float2*>(part_o + (k * all_rows + r) * kv_rank + i);
+                a = fmaf(v.x, w[k], a);
+                b = fmaf(v.y, w[k], b);
+            }
+        *reinterpret_cast<uint32_t*>(out + r * kv_rank + i) = pack_bf16x2(a, b);
+    }
+}
+
+// Two row tiles share a key tile's loads; one is quicker where even single key tiles would not fill the GPU.
+int lm_mt(const scr_latent_shape& s, const scr_step& st, int sms) {
+    const int rows = s.heads * st.max_count;
+    return rows > 16 && (long long)scr_ceil_div(rows, 32) * st.batch * scr_ceil_div(st.max_kv, LM_KEYS) >= sms ? 2 : 1;
+}
+
+// Key shares: enough CTAs to fill the GPU, at least one tile each.
+int lm_splits(const scr_latent_shape& s, const scr_step& st, int sms) {
+    const int blocks = scr_ceil_div(s.heads * st.max_count, 16 * lm_mt(s, st, sms)) * st.batch, tiles = scr_ceil_div(st.max_kv, LM_KEYS);
+    int n = std::max(1, sms / std::max(1, blocks));
+    return std::min(std::min(n, tiles), 64);
+}
+
+template <int MT, int NTW>
+cudaError_t lm_launch(const scr_latent_shape& s, const scr_step& st, const void* q, const void* cache, void* out, float* po, float* ml, int nsplit,
+                      int* status, cudaStream_t stream) {
+    const size_t smem = LmSmem::of(s.kv_rank + s.rot_dim, MT).total;
+    const cudaError_t e = seq_smem(latent_attention_mma_kernel<MT, NTW>, smem);
+    if (e != cudaSuccess) return e;
+    return launch_pdl(latent_attention_mma_kernel<MT, NTW>, dim3(scr_ceil_div(s.heads * st.max_count, 16 * MT), nsplit, st.batch), dim3(LM_THREADS), smem,
+                      stream, s, st, (const bf16*)q, (const bf16*)cache, (bf16*)out, po, ml, nsplit, status);
+}
+
+}  // namespace
+
+bool latent_attention_mma_applies(const scr_latent_shape& s) {
+    const int D = s.kv_rank + s.rot_dim;
+    return s.kv_rank % 8 == 0 && D % 8 == 0 && s.kv_rank <= 512 && LmSmem::of(D, 2).total <= 227 * 1024;
+}
+
+size_t latent_attention_mma_workspace(const scr_latent_shape& s, const scr_step& st, int sms) {
+    const int n = lm_splits(s, st, sms);
+    return n > 1 ? (size_t)n * st.rows * s.heads * (s.kv_rank + 2) * sizeof(float) : 0;
+}
+
+int32_t latent_attention_mma_launch(scr_ctx* ctx, const scr_latent_shape& s, const scr_step& st, const void* q, const void* cache, void* out,
+                                    void* workspace, size_t workspace_bytes, cudaStream_t stream) {
+    if (st.max_count <= 0 || st.max_kv <= 0 || st.batch <= 0) return scr_fail(ctx, SCR_E_SHAPE, "an empty step");
+    if (!scr_aligned16(q) || !scr_aligned16(cache) || !scr_aligned16(out)) return scr_fail(ctx, SCR_E_ALIGN, "q, cache and out must be 16-byte aligned");
+    const int n = lm_splits(s, st, ctx->sm_count), ntw = s.kv_rank <= 64 ? 1 : s.kv_rank <= 128 ? 2 : s.kv_rank <= 256 ? 4 : 8;
+    if (n > 1 && (!workspace || workspace_bytes < latent_attention_mma_workspace(s, st, ctx->sm_count)))
+        return scr_fail(ctx, SCR_E_WORKSPACE, "latent attention over %d key shares needs %zu bytes", n, latent_attention_mma_workspace(s, st, ctx->sm_count));
+    float* po = (float*)workspace;
+    float* ml = po ? po + (size_t)n * st.rows * s.heads * s.kv_rank : nullptr;
+    const bool two = lm_mt(s, st, ctx->sm_count) == 2;
+    cudaError_t e = cudaErrorInvalidValue;
+#define LM_CASE(NTW)                                                                                                                     \
+    case NTW:                                                                                                                            \
+        e = two ? lm_launch<2, NTW>(s, st, q, cache, out, po, ml, n, ctx->dev_status, stream)                                            \
+                : lm_launch<1, NTW>(s, st, q, cache, out, po, ml, n, ctx->dev_status, stream);                                           \
+        break;
+    switch (ntw) { LM_CASE(1) LM_CASE(2) LM_CASE(4) LM_CASE(8) }
+#undef LM_CASE
+    if (e != cudaSuccess) return scr_fail(ctx, SCR_E_CUDA, "latent_attention_mma: %s", cudaGetErrorString(e));
+    int32_t rc = scr_check_launch(ctx, "latent_attention_mma");
+    if (rc || n == 1) return rc;
+    e = launch_pdl(latent_attention_merge_kernel, dim3(st.rows * s.heads), dim3(128), 0, stream, (const float*)po, (const float*)ml, n,
+                   (long long)st.rows * s.heads, s.kv_rank, (bf16*)out);
+    if (e != cudaSuccess) return scr_fail(ctx, SCR_E_CUDA, "latent_attention_merge: %s", cudaGetErrorString(e));
+    return scr_check_launch(ctx, "latent_attention_merge");
+}
