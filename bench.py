@@ -1132,6 +1132,230 @@ def run_case_attention(device, batch, context, reps, layers=28, block_size=16):
     print(json.dumps({"case": f"attn,{batch},{context}", "us": dt * 1e6, "kv_bytes": kv, "GBps": kv / dt / 1e9}))
 
 
+# ------------------------------------------------------------------------------------ hybrid sequence model
+def vumipel_like_llama_3b():
+    """A Vumipel of Llama-3.2-3B's width, feed-forward, vocabulary and number of layer runs: three matrix-memory layers to one
+    of latent attention, 24 layers of which four run twice (28 layer runs)."""
+    def mem():
+        return {"type": "mlstm", "mixer": {"heads": 12, "dim": 128, "vdim": 256, "gate_cap": 15.0}}
+
+    def att():
+        return {"type": "latent_attention", "mixer": {"heads": 24, "dim": 128, "rot_dim": 64, "vdim": 128, "kv_rank": 512, "q_rank": 1536,
+                                                      "rot": {"base": 5e5, "dims": 64}, "scale": 192 ** -0.5}}
+    layers = [{**(att() if i % 4 == 3 else mem()), "mlp": {"kind": "dense", "ff": 8192, "limit": 7.0}} for i in range(24)]
+    return {"architecture": "Vumipel", "layers": layers, "loop": {"start": 8, "stop": 12, "times": 2}, "norm": {"eps": 1e-5}, "vocab": 128256,
+            "width": 3072}
+
+
+class RandomCheckpoint:
+    """Tensors of a Vumipel configuration drawn on the device when they are taken."""
+
+    def __init__(self, cfg, device):
+        import torch
+        self.cfg, self.device, self.gen = cfg, device, torch.Generator(device=device)
+        self.gen.manual_seed(1)
+
+    def shape(self, name):
+        c, W = self.cfg, self.cfg["width"]
+        fixed = {"embed": (c["vocab"], W), "final.norm": (W,), "loop.in": (W, 2 * W)}
+        if name in fixed:
+            return fixed[name]
+        if name == "loop.step":
+            return (c["loop"]["times"], W)
+        layer, rest = name.split(".", 1)
+        spec = c["layers"][int(layer[1:])]
+        if rest.startswith("norm"):
+            return (W,)
+        if rest.startswith("mlp."):
+            return (W, spec["mlp"]["ff"]) if rest == "mlp.down" else (spec["mlp"]["ff"], W)
+        m, part = spec["mixer"], rest[4:]
+        H = m["heads"]
+        if spec["type"] == "mlstm":
+            return {"q": (H * m["dim"], W), "k": (H * m["dim"], W), "v": (H * m["vdim"], W), "g": (H * m["vdim"], W), "i": (H, W), "f": (H, W), "i.b": (H,),
+                    "f.b": (H,), "norm": (H * m["vdim"],), "o": (W, H * m["vdim"])}[part]
+        return {"dq": (m["q_rank"], W), "dq.norm": (m["q_rank"],), "uq": (H * (m["dim"] + m["rot_dim"]), m["q_rank"]),
+                "dkv": (m["kv_rank"] + m["rot_dim"], W), "dkv.norm": (m["kv_rank"],), "uk": (H * m["dim"], m["kv_rank"]),
+                "uv": (H * m["vdim"], m["kv_rank"]), "g": (H * m["vdim"], W), "o": (W, H * m["vdim"])}[part]
+
+    def take(self, name):
+        import torch
+        shape = self.shape(name)
+        t = torch.randn(shape, device=self.device, generator=self.gen)
+        return (t * (shape[1] ** -0.5 if len(shape) == 2 and name != "embed" else 0.1) + (3.0 if name.endswith("f.b") else 0.0)).to(torch.bfloat16)
+
+
+def run_sequence_model(device, steps=20, batches=(1, 8, 32), context=2048, prompts=(512, 2048, 8192)):
+    """`--sequence-model`: prefill and decode throughput of a 2.8-billion-parameter Vumipel in bf16 (random weights), beside
+    the int4 Llama-3.2-3B decode step of the same width, depth, feed-forward and vocabulary.  Every weight is distinct and
+    the step streams 7 GB, far more than L2 holds."""
+    import torch
+    from scratchy_b200 import _lib
+    from scratchy_b200.vumipel import Vumipel, VumipelConfig
+    peaks = measured_peaks()
+    raw = vumipel_like_llama_3b()
+    longest = max(max(prompts), max(batches) * (context + 64))
+    model = Vumipel(VumipelConfig.from_dict(raw), RandomCheckpoint(raw, device), device, "bfloat16", max_tokens=longest, max_sequences=max(batches))
+    ctx = _lib.models_context(device.index or 0)
+    run_weights = sum(2 * w.weight.numel() for i, _ in model.runs for m in (model.layers[i].mixer, model.layers[i].mlp)
+                      for w in vars(m).values() if hasattr(w, "weight") and w is not getattr(m, "uk_rows", None))
+    run_weights += 2 * model.embed.numel() + 2 * model.loop_in.weight.numel() * raw["loop"]["times"]
+    att_runs = sum(1 for i, _ in model.runs if raw["layers"][i]["type"] == "latent_attention")
+    mem_runs = len(model.runs) - att_runs
+    out = {"workload": "Vumipel, random weights, bf16: width 3072, 24 layers (28 runs), feed-forward 8192, vocabulary 128256, 3 mlstm : 1 latent attention",
+           "weight_bytes_per_step": run_weights, "prefill": [], "decode": []}
+
+    def timed(call, reps, warm=3):
+        for _ in range(warm):
+            call()
+        torch.cuda.synchronize(device)
+        a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+        a.record()
+        for _ in range(reps):
+            call()
+        b.record()
+        torch.cuda.synchronize(device)
+        return a.elapsed_time(b) * 1e-3 / reps
+
+    g = torch.Generator().manual_seed(0)
+    flops_per_token = 2 * (run_weights / 2 - model.embed.numel())               # (the vocabulary head runs for one position)
+    for n in prompts:
+        tokens = torch.randint(0, raw["vocab"], (n,), generator=g).tolist()
+
+        def prefill():
+            seq = model.table.open("p")
+            model.forward([(seq, tokens)], [[n - 1]])
+            model.table.close("p")
+        dt = timed(prefill, 5)
+        out["prefill"].append({"tokens": n, "ms": dt * 1e3, "tok_per_s": n / dt, "TFLOPs_linears": n * flops_per_token / dt / 1e12,
+                               "frac_bf16_sustained": n * flops_per_token / dt / 1e12 / peaks["bf16_tflops_sustained"]})
+    for batch in batches:
+        seqs = [model.table.open(("d", b)) for b in range(batch)]
+        for seq in seqs:                                                        # sequences of `context` tokens: blocks handed out, contents left as they are
+            model.table.extend(seq, context + 1)
+            model.table.advance(seq, context)
+        n0 = ctx.launch_count()
+        dg = model.decode_graph(batch, 1 << (context).bit_length())
+        launches = (ctx.launch_count() - n0) // 2                               # the warm-up step and the captured one
+        dg.inputs.fill([(seq, [1]) for seq in seqs], list(range(batch)))
+        dt = timed(dg.graph.replay, steps)
+        model.check_health()
+        cache = att_runs * batch * context * 576 * 2
+        state = mem_runs * batch * 12 * 128 * 256 * 4 * 2                       # read and written
+        moved = run_weights + cache + state
+        out["decode"].append({"batch": batch, "context": context, "ms_per_step": dt * 1e3, "tok_per_s": batch / dt, "launches_per_step": int(launches),
+                              "cache_bytes": cache, "state_bytes": state, "GBps": moved / dt / 1e9, "frac_hbm": moved / dt / 1e9 / peaks["hbm_gbs"]})
+        for b in range(batch):
+            model.table.close(("d", b))
+    out["kernels"] = run_sequence_kernels(device, model, peaks)
+    del model
+    torch.cuda.empty_cache()
+    out["llama_3b_int4_decode"] = run_decode(device, steps=steps, batches=batches, context=context)
+    return out
+
+
+def run_sequence_kernels(device, model, peaks, context=2048):
+    """The kernels of the hybrid model alone at its sizes, each call on its own weights, cache or state (CUDA graph)."""
+    import ctypes
+    import torch
+    from scratchy_b200 import _lib
+    from scratchy_b200.dense import Arena, DenseLinear, StepInputs, dtype_code, seq_norm
+    from scratchy_b200.layers import _ptr, _stream
+    from scratchy_b200.mixers import StepContext
+    lib, c = _lib.models_lib(), _lib.models_context(device.index or 0)
+    bf, rows, arena = torch.bfloat16, [], Arena(device)
+    att = [l.mixer for l in model.layers if hasattr(l.mixer, "kv_rank")]
+    mem = [l.mixer for l in model.layers if not hasattr(l.mixer, "kv_rank")]
+    mlps = [l.mlp for l in model.layers]
+    code = dtype_code(bf)
+
+    def add(kernel, us, flops=None, nbytes=None, **more):
+        row = {"kernel": kernel, **more, "us": us * 1e6}
+        if flops:
+            row.update({"TFLOPs": flops / us / 1e12, "frac_bf16_burst": flops / us / 1e12 / peaks["bf16_tflops"]})
+        if nbytes:
+            row.update({"GBps": nbytes / us / 1e9, "frac_hbm": nbytes / us / 1e9 / peaks["hbm_gbs"]})
+        rows.append(row)
+    for M in (1, 8, 32, 512, 2048):
+        for name, lins in (("gate_up", [m.gate_up for m in mlps]), ("down", [m.down for m in mlps]), ("mlstm proj", [m.proj for m in mem]), ("o", [m.o for m in mem])):
+            lins = lins[:8]
+            x = torch.randn((M, lins[0].in_features), device=device).to(bf)
+            cols = lins[0].out_features // (2 if name == "gate_up" else 1)
+            y = torch.empty((M, cols), dtype=bf if name == "gate_up" else torch.float32, device=device)
+            dt = _time_calls(device, [(lambda l=l: l(arena, x, y)) for l in lins], 10)
+            N, K = lins[0].out_features, lins[0].in_features
+            add("dense " + name, dt, 2.0 * M * N * K if M > 32 else None, (N * K * 2 + M * K * 2 + M * cols * y.element_size()) if M <= 32 else None, M=M, N=N, K=K)
+
+    def context_of(batch, count, kv, prompt):
+        T = batch * count
+        blocks = -(-kv // model.table.block_size)
+        inputs = StepInputs(device, T, batch, 1, blocks)
+
+        class S:
+            pass
+        entries = []
+        perm = torch.randperm(batch * blocks).tolist()
+        for b in range(batch):
+            s = S()
+            s.length, s.slot, s.blocks = kv - count, b, perm[b * blocks:(b + 1) * blocks]
+            entries.append((s, [0] * count))
+        inputs.fill(entries, [0])
+        return StepContext(arena, inputs, inputs.struct(model.table.max_sequences), [(s, count) for s, _ in entries], model.table.block_size, batch * blocks, T,
+                           prompt)
+    m = att[0]
+    for batch in (1, 8, 32):
+        sc = context_of(batch, 1, context, False)
+        copies = max(2, (256 << 20) // (batch * context * m.row_size * 2))
+        copies = min(copies, 24)
+        caches = [torch.randn((sc.num_blocks * sc.block_size, m.row_size), device=device).to(bf) for _ in range(copies)]
+        q = torch.randn((batch, m.heads * m.row_size), device=device).to(bf)
+        o = torch.empty((batch, m.heads * m.kv_rank), dtype=bf, device=device)
+        shape, need = m.shape(sc), ctypes.c_size_t(0)
+        lib.scr_latent_attention_workspace(code, ctypes.byref(shape), ctypes.byref(sc.step), ctypes.byref(need))
+        ws = torch.empty(max(16, need.value), dtype=torch.uint8, device=device)
+        call = lambda k: c.check(lib.scr_latent_attention(c.handle, code, ctypes.byref(shape), ctypes.byref(sc.step), _ptr(q), _ptr(k), _ptr(o), _ptr(ws), need,
+                                                          _stream(device)))
+        dt = _time_calls(device, [(lambda k=k: call(k)) for k in caches], 10)
+        add("latent attention decode", dt, None, batch * context * m.row_size * 2, batch=batch, context=context,
+            TFLOPs=2.0 * batch * context * m.heads * (m.row_size + m.kv_rank) / dt / 1e12, cache_copies=copies)
+        del caches
+    for T in (2048, 8192):
+        sc = context_of(1, T, T, True)
+        q, k, r = (torch.randn((T, n), device=device).to(bf) for n in (m.heads * (m.dim + m.rot_dim), m.heads * m.dim, m.rot_dim))
+        v, gate, o = torch.randn((m.heads * m.vdim, T), device=device).to(bf), torch.randn((T, m.heads * m.vdim), device=device).to(bf), torch.empty((T, m.heads * m.vdim), dtype=bf, device=device)
+        shape = m.shape(sc)
+        call = lambda: c.check(lib.scr_latent_prefill(c.handle, ctypes.byref(shape), _ptr(q), _ptr(k), _ptr(r), _ptr(v), T, _ptr(gate), m.heads * m.vdim, T, 0, _ptr(o),
+                                                      m.heads * m.vdim, _stream(device)))
+        dt = _time_calls(device, [call] * 4, 5)
+        add("latent attention prompt", dt, 2.0 * m.heads * (m.dim + m.rot_dim + m.vdim) * T * (T + 1) / 2, None, T=T)
+    m = mem[0]
+    for batch, count in ((1, 1), (8, 1), (32, 1), (1, 2048), (4, 2048)):
+        sc = context_of(batch, count, count + 64, count > 1)
+        T = batch * count
+        n_main = 2 * m.heads * m.dim + 2 * m.heads * m.vdim
+        proj, gates, o = torch.randn((T, n_main), device=device).to(bf), torch.randn((T, 2 * m.heads), device=device), torch.empty((T, m.heads * m.vdim), device=device)
+        copies = 2 if count > 1 else min(24, max(2, (256 << 20) // (batch * m.heads * m.dim * m.vdim * 4)))
+        states = [m.state(batch, device) for _ in range(copies)]
+        shape = _lib.MlstmShape(m.heads, m.dim, m.vdim, m.gate_cap, m.eps)
+        call = lambda s: c.check(lib.scr_mlstm_run(c.handle, code, ctypes.byref(shape), ctypes.byref(sc.step), _ptr(proj), n_main, _ptr(gates), 2 * m.heads,
+                                                   _ptr(m.bias_i), _ptr(m.bias_f), *[_ptr(t) for t in s], _ptr(o), _stream(device)))
+        dt = _time_calls(device, [(lambda s=s: call(s)) for s in states], 10)
+        state_bytes = batch * m.heads * m.dim * m.vdim * 8
+        if count == 1:
+            add("matrix memory step", dt, None, state_bytes, batch=batch, state_copies=copies)
+        else:
+            L = 64                                   # the closed form of a 64-token chunk: q k, P v, q S, k v
+            add("matrix memory prompt", dt, 2.0 * T * m.heads * (L / 2 * (m.dim + m.vdim) + 2 * m.dim * m.vdim), T * (n_main - m.heads * m.vdim) * 2 + T * m.heads * m.vdim * 4, batch=batch, T=count)
+        del states
+    for T in (1, 2048):
+        copies = 8 if T > 1 else 24
+        xs, ds = [torch.randn((T, 3072), device=device) for _ in range(copies)], [torch.randn((T, 3072), device=device) for _ in range(copies)]
+        w, h = torch.randn(3072, device=device), torch.empty((T, 3072), dtype=bf, device=device)
+        dt = _time_calls(device, [(lambda x=x, d=d: seq_norm(x, 1e-5, delta=d, w_delta=w, out=h, w_out=w)) for x, d in zip(xs, ds)], 10)
+        add("norm, add, norm", dt, None, T * 3072 * (4 * 3 + 2), T=T)
+    c.device_status(None)
+    return rows
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -1149,6 +1373,9 @@ def main():
     ap.add_argument("--tp-separate-exchange", action="store_true",
                     help="tensor-parallel section: row-parallel matvec and all-reduce as two launches instead of "
                          "scr_linear_fp8_dynamic_allreduce (measured: equal at TP=2, 9 %% slower at TP=8)")
+    ap.add_argument("--sequence-model", action="store_true",
+                    help="prefill and decode throughput of a hybrid sequence model (Vumipel, bf16, random weights) beside the int4 Llama of "
+                         "equal size, and its kernels alone; prints one JSON line of its own")
     ap.add_argument("--case", default=None, help="kind,shape,M e.g. int4,gate,2048: time one linear alone")
     args = ap.parse_args()
     if args.case:
@@ -1161,6 +1388,14 @@ def main():
         cases = run_decode(device, steps=args.steps, batches=tuple(int(b) for b in args.decode_batches.split(",")),
                            fuse_rope=not args.no_fuse_rope)
         print(json.dumps({"decode": cases}))
+        return
+    if args.sequence_model:
+        import torch
+        device = torch.device("cuda", 0)
+        torch.cuda.set_device(device)
+        sampler = ClockSampler(0)
+        res = run_sequence_model(device, steps=min(args.steps, 50))
+        print(json.dumps({"sequence_model": res, "clocks": sampler.stop()}))
         return
     if args.impl == "reference":
         run_reference(args)

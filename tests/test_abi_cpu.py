@@ -10,8 +10,8 @@ from scratchy_b200 import _lib
 ROOT = os.path.dirname(os.path.dirname(os.path.abspath(__file__)))
 
 
-def header_symbols():
-    text = open(os.path.join(ROOT, "include", "scratchy_cuda.h")).read()
+def header_symbols(name="scratchy_cuda.h"):
+    text = open(os.path.join(ROOT, "include", name)).read()
     text = re.sub(r"/\*.*?\*/", "", text, flags=re.S)
     return sorted(set(re.findall(r"\b(scr_[a-z0-9_]+)\s*\(", text)))
 
@@ -26,6 +26,19 @@ def test_library_exports_every_declared_symbol():
 
 def test_binding_table_matches_header():
     assert sorted(_lib.SIGNATURES) == header_symbols()
+
+
+def test_models_library_and_its_binding_table_match_their_header():
+    names = header_symbols("scratchy_models.h")
+    assert sorted(_lib.MODELS_SIGNATURES) == names
+    L = _lib.models_lib()
+    for n in names + sorted(_lib.CONTEXT_SIGNATURES):
+        assert hasattr(L, n), f"{n} is not exported by the models library"
+    assert L.scr_status_string(-4) == b"SCR_E_DTYPE"
+    s = ctypes.c_size_t(1)
+    assert L.scr_dense_workspace_size(_lib.DTYPE_BF16, 16, 64, 64, 1, ctypes.byref(s)) == 0 and s.value == 0
+    assert L.scr_dense_workspace_size(_lib.DTYPE_BF16, 0, 64, 64, 1, ctypes.byref(s)) == -2
+    assert L.scr_dense_linear(None, _lib.DTYPE_BF16, None, None, 0, None) == -1
 
 
 def test_status_strings():
@@ -101,8 +114,9 @@ def test_struct_mirrors_have_the_layout_the_c_compiler_gives(tmp_path):
     cc = shutil.which("gcc") or shutil.which("cc")
     if cc is None:
         pytest.skip("no C compiler")
-    fields = {"scr_qmv_ends": [f[0] for f in _lib.QmvEnds._fields_], "scr_tape_linear": [f[0] for f in _lib.TapeLinear._fields_]}
-    lines = ['#include <stdio.h>', '#include <stddef.h>', '#include "scratchy_cuda.h"', 'int main(void) {']
+    mirrors = {"scr_qmv_ends": _lib.QmvEnds, "scr_tape_linear": _lib.TapeLinear, **_lib.MODELS_STRUCTS}
+    fields = {s: [f[0] for f in cls._fields_] for s, cls in mirrors.items()}
+    lines = ['#include <stdio.h>', '#include <stddef.h>', '#include "scratchy_models.h"', 'int main(void) {']
     for s, fs in fields.items():
         lines.append(f'  printf("{s} %zu\\n", sizeof({s}));')
         for f in fs:
@@ -113,7 +127,7 @@ def test_struct_mirrors_have_the_layout_the_c_compiler_gives(tmp_path):
     exe = tmp_path / "layout"
     subprocess.check_call([cc, "-I", os.path.join(ROOT, "include"), str(src), "-o", str(exe)])
     got = dict(line.split() for line in subprocess.check_output([str(exe)], text=True).splitlines())
-    for s, cls in (("scr_qmv_ends", _lib.QmvEnds), ("scr_tape_linear", _lib.TapeLinear)):
+    for s, cls in mirrors.items():
         assert int(got[s]) == ctypes.sizeof(cls), s
         for f in fields[s]:
             assert int(got[f"{s}.{f}"]) == getattr(cls, f).offset, f"{s}.{f}"
