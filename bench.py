@@ -1336,8 +1336,11 @@ def run_sequence_kernels(device, model, peaks, context=2048):
         copies = 2 if count > 1 else min(24, max(2, (256 << 20) // (batch * m.heads * m.dim * m.vdim * 4)))
         states = [m.state(batch, device) for _ in range(copies)]
         shape = _lib.MlstmShape(m.heads, m.dim, m.vdim, m.gate_cap, m.eps)
+        need = ctypes.c_size_t(0)
+        c.check(lib.scr_mlstm_workspace(code, ctypes.byref(shape), ctypes.byref(sc.step), ctypes.byref(need)))
+        ws = torch.empty(max(16, need.value), dtype=torch.uint8, device=device)
         call = lambda s: c.check(lib.scr_mlstm_run(c.handle, code, ctypes.byref(shape), ctypes.byref(sc.step), _ptr(proj), n_main, _ptr(gates), 2 * m.heads,
-                                                   _ptr(m.bias_i), _ptr(m.bias_f), *[_ptr(t) for t in s], _ptr(o), _stream(device)))
+                                                   _ptr(m.bias_i), _ptr(m.bias_f), *[_ptr(t) for t in s], _ptr(o), _ptr(ws), need, _stream(device)))
         dt = _time_calls(device, [(lambda s=s: call(s)) for s in states], 10)
         state_bytes = batch * m.heads * m.dim * m.vdim * 8
         if count == 1:

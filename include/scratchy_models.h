@@ -136,9 +136,12 @@ typedef struct scr_mlstm_shape {
     int32_t heads, dim, vdim;
     float gate_cap, eps;
 } scr_mlstm_shape;
+/* `workspace`: states between the groups of a long prompt that is cut to fill the GPU. */
+int32_t scr_mlstm_workspace(int32_t dtype, const scr_mlstm_shape* s, const scr_step* st, size_t* bytes);
 int32_t scr_mlstm_run(scr_ctx* ctx, int32_t dtype, const scr_mlstm_shape* s, const scr_step* st, const void* proj,
                       int64_t ld, const float* gates, int64_t ld_gates, const float* bias_i, const float* bias_f,
-                      float* state_s, float* state_n, float* state_m, float* out, void* stream);
+                      float* state_s, float* state_n, float* state_m, float* out, void* workspace,
+                      size_t workspace_bytes, void* stream);
 /* y[t, h, :] (dtype) = out / rms(out over the head) * norm * sigmoid(gate[t, h, :]) */
 int32_t scr_mlstm_finish(scr_ctx* ctx, int32_t dtype, const scr_mlstm_shape* s, const float* out, const float* norm,
                          const void* gate, int64_t ld_gate, int32_t rows, void* y, void* stream);

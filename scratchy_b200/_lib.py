@@ -110,7 +110,8 @@ MODELS_SIGNATURES = {
     "scr_latent_prefill_supported": (_i32, [_vp]),
     "scr_latent_gather": (_i32, [_vp, _vp, _vp, _i32, _vp, _vp, _vp, _vp]),
     "scr_latent_prefill": (_i32, [_vp, _vp, _vp, _vp, _vp, _vp, _i64, _vp, _i64, _i32, _i32, _vp, _i64, _vp]),
-    "scr_mlstm_run": (_i32, [_vp, _i32, _vp, _vp, _vp, _i64, _vp, _i64, _vp, _vp, _vp, _vp, _vp, _vp, _vp]),
+    "scr_mlstm_workspace": (_i32, [_i32, _vp, _vp, _psz]),
+    "scr_mlstm_run": (_i32, [_vp, _i32, _vp, _vp, _vp, _i64, _vp, _i64, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _sz, _vp]),
     "scr_mlstm_finish": (_i32, [_vp, _i32, _vp, _vp, _vp, _vp, _i64, _i32, _vp, _vp]),
 }
 

@@ -69,56 +69,74 @@ __global__ void __launch_bounds__(256) dense_plain_kernel(const T* __restrict__ 
 }
 
 // ------------------------------------------------------------------------------- decode matvec
-// A tile is 16 weight rows over the whole K, shared by `wpt` warps that take 64-wide units of K in turn.  In a unit lane
-// (g, t) loads the 16-byte pieces [t*8, t*8+8) and [32 + t*8, ..) of rows g and g + 8, and the same pieces of
-// activation row g: the k order inside a fragment is a permutation both operands share, so the loaded registers are
-// mma operands as they stand (weights = A, 8 tokens per B).  The first pieces of the weights, load-time constants, are
-// requested before the wait for the preceding kernel.  Partial sums of the warps meet in shared memory in warp order.
-constexpr int MV_WARPS = 8, MV_UNROLL = 3;
+// A tile is 16 weight rows over the whole K, shared by `wpt` warps of each CTA of a cluster, which take 64-wide units of K
+// in turn.  In a unit lane (g, t) loads the 16-byte pieces [t*8, t*8+8) and [32 + t*8, ..) of rows g and g + 8, and the
+// same pieces of activation row g: the k order inside a fragment is a permutation both operands share, so the loaded
+// registers are mma operands as they stand (weights = A, 8 tokens per B).  A warp keeps SLOTS units in flight and refills a
+// unit's registers as soon as they are used; the first ones, load-time constants, are requested before the wait for the
+// preceding kernel.  Partial sums meet in shared memory in warp order, then in the cluster's first CTA in rank order.
+constexpr int MV_WARPS = 8, MV_MAX_CLUSTER = 4;
 
-template <int NT>
-__global__ void __launch_bounds__(MV_WARPS * 32) dense_matvec_kernel(const bf16* __restrict__ w, const bf16* __restrict__ x,
-                                                                     long long ldx, long long x_group, int M, int N, int K,
-                                                                     int wpt, DenseEnds ends) {
+__device__ __forceinline__ uint32_t mv_cluster_rank() {
+    uint32_t r;
+    asm volatile("mov.u32 %0, %%cluster_ctarank;" : "=r"(r));
+    return r;
+}
+
+template <int NT, int SLOTS>
+__global__ void __launch_bounds__(MV_WARPS * 32, 2) dense_matvec_kernel(const bf16* __restrict__ w, const bf16* __restrict__ x,
+                                                                        long long ldx, long long x_group, int M, int N, int K,
+                                                                        int wpt, int cluster, DenseEnds ends) {
     __shared__ float red[MV_WARPS][16][8 * NT + 1];
+    __shared__ float peers[MV_MAX_CLUSTER - 1][MV_WARPS][16][8 * NT];          // [rank - 1][tile][row][token], filled on rank 0
     pdl_trigger();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g = lane >> 2, t = lane & 3;
-    const int tiles = MV_WARPS / wpt, part = warp % wpt, grp = blockIdx.y;
-    const int n0 = (blockIdx.x * tiles + warp / wpt) * 16;
+    const int rank = cluster > 1 ? (int)mv_cluster_rank() : 0;
+    const int tiles = MV_WARPS / wpt, part = warp % wpt + rank * wpt, step = wpt * cluster, grp = blockIdx.y;
+    const int tile0 = (blockIdx.x / cluster) * tiles;
+    const int n0 = (tile0 + warp / wpt) * 16;
     const int units = (K + 63) >> 6;
     const bf16* w0 = w + ((size_t)grp * N + min(n0 + g, N - 1)) * K + t * 8;
     const bf16* w1 = w + ((size_t)grp * N + min(n0 + g + 8, N - 1)) * K + t * 8;
-    uint4 wa[MV_UNROLL][2], wb[MV_UNROLL][2];
-    auto load_w = [&](int u0) {
+    x += grp * x_group + t * 8;
+    uint4 wa[SLOTS][2], wb[SLOTS][2], xv[SLOTS][2][NT];
+    const uint4 zero = make_uint4(0, 0, 0, 0);
+    auto load_w = [&](int s, int u) {
 #pragma unroll
-        for (int u = 0; u < MV_UNROLL; ++u)
+        for (int h = 0; h < 2; ++h) {
+            const int k = u * 64 + h * 32;
+            const bool ok = k + t * 8 < K;
+            wa[s][h] = ok ? ld_stream_v4(w0 + k) : zero;
+            wb[s][h] = ok ? ld_stream_v4(w1 + k) : zero;
+        }
+    };
+    auto load_x = [&](int s, int u) {
 #pragma unroll
-            for (int h = 0; h < 2; ++h) {
-                const int k = (u0 + u * wpt) * 64 + h * 32;
-                const bool ok = k + t * 8 < K;
-                wa[u][h] = ok ? ld_stream_v4(w0 + k) : make_uint4(0, 0, 0, 0);
-                wb[u][h] = ok ? ld_stream_v4(w1 + k) : make_uint4(0, 0, 0, 0);
-            }
+        for (int h = 0; h < 2; ++h) {
+            const int k = u * 64 + h * 32;
+#pragma unroll
+            for (int nt = 0; nt < NT; ++nt) xv[s][h][nt] = (nt * 8 + g < M && k + t * 8 < K) ? ld_act_v4(x + (nt * 8 + g) * ldx + k) : zero;
+        }
     };
     float acc[NT][4] = {};
-    load_w(part);
+#pragma unroll
+    for (int s = 0; s < SLOTS; ++s) load_w(s, part + s * step);
     pdl_wait();
-    x += grp * x_group + t * 8;
-    for (int u0 = part; u0 < units; u0 += MV_UNROLL * wpt) {
-        if (u0 != part) load_w(u0);
 #pragma unroll
-        for (int u = 0; u < MV_UNROLL; ++u)
+    for (int s = 0; s < SLOTS; ++s) load_x(s, part + s * step);
+    for (int u0 = part; u0 < units; u0 += SLOTS * step) {
 #pragma unroll
-            for (int h = 0; h < 2; ++h) {
-                const int k = (u0 + u * wpt) * 64 + h * 32;
+        for (int s = 0; s < SLOTS; ++s) {
+#pragma unroll
+            for (int h = 0; h < 2; ++h)
 #pragma unroll
                 for (int nt = 0; nt < NT; ++nt) {
-                    uint4 xv = make_uint4(0, 0, 0, 0);
-                    if (nt * 8 + g < M && k + t * 8 < K) xv = ld_act_v4(x + (nt * 8 + g) * ldx + k);
-                    mma_16816(acc[nt], wa[u][h].x, wb[u][h].x, wa[u][h].y, wb[u][h].y, xv.x, xv.y);
-                    mma_16816(acc[nt], wa[u][h].z, wb[u][h].z, wa[u][h].w, wb[u][h].w, xv.z, xv.w);
+                    mma_16816(acc[nt], wa[s][h].x, wb[s][h].x, wa[s][h].y, wb[s][h].y, xv[s][h][nt].x, xv[s][h][nt].y);
+                    mma_16816(acc[nt], wa[s][h].z, wb[s][h].z, wa[s][h].w, wb[s][h].w, xv[s][h][nt].z, xv[s][h][nt].w);
                 }
-            }
+            load_w(s, u0 + (s + SLOTS) * step);
+            load_x(s, u0 + (s + SLOTS) * step);
+        }
     }
 #pragma unroll
     for (int nt = 0; nt < NT; ++nt) {
@@ -133,17 +151,34 @@ __global__ void __launch_bounds__(MV_WARPS * 32) dense_matvec_kernel(const bf16*
         for (int p = 0; p < wpt; ++p) v += red[tile * wpt + p][r][m];
         return v;
     };
+    if (cluster > 1) {
+        if (rank > 0) {
+            for (int i = threadIdx.x; i < tiles * 16 * M; i += MV_WARPS * 32) {
+                const int r = i & 15, tile = (i >> 4) % tiles, m = (i >> 4) / tiles;
+                uint32_t dst;
+                asm volatile("mapa.shared::cluster.u32 %0, %1, 0;" : "=r"(dst) : "r"(smem_u32(&peers[rank - 1][tile][r][m])));
+                asm volatile("st.shared::cluster.f32 [%0], %1;" ::"r"(dst), "f"(total(tile, r, m)) : "memory");
+            }
+        }
+        asm volatile("barrier.cluster.arrive.release.aligned;\n\tbarrier.cluster.wait.acquire.aligned;" ::: "memory");
+        if (rank > 0) return;
+    }
+    auto whole = [&](int tile, int r, int m) {
+        float v = total(tile, r, m);
+        for (int c = 1; c < cluster; ++c) v += peers[c - 1][tile][r][m];
+        return v;
+    };
     if (ends.act) {
         for (int i = threadIdx.x; i < tiles * 8 * M; i += MV_WARPS * 32) {
             const int r = i & 7, tile = (i >> 3) % tiles, m = (i >> 3) / tiles;
-            const int n = (blockIdx.x * tiles + tile) * 16 + r;
-            if (n < N) dense_put_pair<bf16>(ends, m, n, total(tile, r, m), total(tile, r + 8, m));
+            const int n = (tile0 + tile) * 16 + r;
+            if (n < N) dense_put_pair<bf16>(ends, m, n, whole(tile, r, m), whole(tile, r + 8, m));
         }
     } else {
         for (int i = threadIdx.x; i < tiles * 16 * M; i += MV_WARPS * 32) {
             const int r = i & 15, tile = (i >> 4) % tiles, m = (i >> 4) / tiles;
-            const int n = (blockIdx.x * tiles + tile) * 16 + r;
-            if (n < N) dense_put<bf16>(ends, m, grp, n, total(tile, r, m));
+            const int n = (tile0 + tile) * 16 + r;
+            if (n < N) dense_put<bf16>(ends, m, grp, n, whole(tile, r, m));
         }
     }
 }
@@ -153,11 +188,27 @@ int32_t matvec_launch(scr_ctx* ctx, const scr_dense& d, cudaStream_t stream) {
     // warps per tile: enough units of K for each, and enough CTAs to fill the GPU
     int wpt = 1;
     while (wpt < MV_WARPS && (units >= 4 * wpt || (units >= 2 * wpt && (tiles16 * d.groups * wpt) / MV_WARPS < 2 * ctx->sm_count))) wpt *= 2;
-    const dim3 grid(scr_ceil_div(tiles16, MV_WARPS / wpt), d.groups);
+    const int blocks = scr_ceil_div(tiles16, MV_WARPS / wpt);
+    // few, long tiles: a cluster shares each, so that the SMs' shares come out even
+    int cluster = 1;
+    while (cluster < MV_MAX_CLUSTER && blocks * d.groups * cluster < 2 * ctx->sm_count && units >= 16 * wpt * cluster) cluster *= 2;
+    cudaLaunchConfig_t cfg = {};
+    cfg.gridDim = dim3(blocks * cluster, d.groups);
+    cfg.blockDim = dim3(MV_WARPS * 32);
+    cfg.stream = stream;
+    cudaLaunchAttribute attr[2];
+    attr[0].id = cudaLaunchAttributeProgrammaticStreamSerialization;
+    attr[0].val.programmaticStreamSerializationAllowed = 1;
+    attr[1].id = cudaLaunchAttributeClusterDimension;
+    attr[1].val.clusterDim.x = cluster;
+    attr[1].val.clusterDim.y = attr[1].val.clusterDim.z = 1;
+    cfg.attrs = attr;
+    cfg.numAttrs = cluster > 1 ? 2 : 1;
     const bf16 *w = (const bf16*)d.w, *x = (const bf16*)d.x;
+    const long long ldx = d.ldx, xg = d.x_group;
     const DenseEnds e = dense_ends(d);
-    const cudaError_t err = d.M <= 8 ? launch_pdl(dense_matvec_kernel<1>, grid, dim3(MV_WARPS * 32), 0, stream, w, x, (long long)d.ldx, (long long)d.x_group, d.M, d.N, d.K, wpt, e)
-                                     : launch_pdl(dense_matvec_kernel<2>, grid, dim3(MV_WARPS * 32), 0, stream, w, x, (long long)d.ldx, (long long)d.x_group, d.M, d.N, d.K, wpt, e);
+    const cudaError_t err = d.M <= 8 ? cudaLaunchKernelEx(&cfg, dense_matvec_kernel<1, 3>, w, x, ldx, xg, d.M, d.N, d.K, wpt, cluster, e)
+                                     : cudaLaunchKernelEx(&cfg, dense_matvec_kernel<2, 2>, w, x, ldx, xg, d.M, d.N, d.K, wpt, cluster, e);
     if (err != cudaSuccess) return scr_fail(ctx, SCR_E_CUDA, "dense_matvec: %s", cudaGetErrorString(err));
     return scr_check_launch(ctx, "dense_matvec");
 }

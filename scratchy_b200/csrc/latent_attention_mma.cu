@@ -2,10 +2,12 @@
 // of which read the same cache rows [latent | rotated key part].
 //
 // A CTA takes 16 or 32 of those rows and a share of the keys.  Key tiles of 64 cache rows come through two shared-memory
-// stages (cp.async, one warp per row of the paged cache, the next tile in flight while this one is computed).  Per tile:
-// S = Q K^T with the key range dealt to the warps, scores to shared memory in f32; a softmax pass over the rows that keeps
-// the running maximum and sum in f32 and leaves P as a bf16 head and remainder (two products, so the weights keep about
-// 16 bits); O += P V with the latent columns dealt to the warps, V being the first kv_rank columns of the very tile.
+// stages (cp.async, one warp per row of the paged cache, the next tile in flight while this one is computed, its rows'
+// addresses looked up a tile earlier).  Per tile: S = Q K^T with warp = (quarter of the dimensions, half of the keys), so
+// that a warp keeps its part of Q in registers and every key element is read once; the quarters meet in shared memory in
+// f32; a softmax pass over the rows that keeps the running maximum and sum in f32 and leaves P as a bf16 head and
+// remainder (two products, so the weights keep about 16 bits); O += P V with the latent columns dealt to the warps, V
+// being the first kv_rank columns of the very tile.
 // Shares of the keys that other CTAs took meet in a second kernel.
 #include "seq_common.cuh"
 
@@ -21,10 +23,10 @@ struct LmSmem {
     static __host__ __device__ LmSmem of(int D, int mt) {
         LmSmem s{};
         s.ld = (D + 15) / 16 * 16 + 8;
-        s.q = 0;
-        s.tile = s.q + (size_t)mt * 16 * s.ld * 2;
-        s.scores = s.tile + 2 * (size_t)LM_KEYS * s.ld * 2;
-        s.p_hi = s.scores + (size_t)mt * 16 * LM_S_LD * 4;
+        s.q = s.scores = 0;                                    // Q moves to registers before the first scores are written
+        const size_t q = (size_t)mt * 16 * s.ld * 2, part = 4 * (size_t)mt * 16 * LM_S_LD * 4;
+        s.tile = q > part ? q : part;
+        s.p_hi = s.tile + 2 * (size_t)LM_KEYS * s.ld * 2;
         s.p_lo = s.p_hi + (size_t)mt * 16 * LM_P_LD * 2;
         s.corr = s.p_lo + (size_t)mt * 16 * LM_P_LD * 2;
         s.total = s.corr + (size_t)mt * 16 * 4 * 2;
@@ -39,11 +41,11 @@ __device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commi
 __device__ __forceinline__ void cp_async_wait_all() { asm volatile("cp.async.wait_group 0;" ::: "memory"); }
 __device__ __forceinline__ float exp2_fast(float x) {
     float y;
-    asm volatile("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
     return y;
 }
 
-// MT: 16-row tiles; NTW: 8-column tiles of the latent per warp (kv_rank <= 64 * NTW)
+// MT: 16-row tiles; NTW: 8-column tiles of the latent per warp (kv_rank <= 64 * NTW, kv_rank + rot_dim <= 64 * (NTW + 1))
 template <int MT, int NTW>
 __global__ void __launch_bounds__(LM_THREADS) latent_attention_mma_kernel(scr_latent_shape s, scr_step st, const bf16* __restrict__ q,
                                                                           const bf16* __restrict__ cache, bf16* __restrict__ out,
@@ -73,21 +75,26 @@ __global__ void __launch_bounds__(LM_THREADS) latent_attention_mma_kernel(scr_la
     const int t_lo = min(split * per, tiles), t_hi = min(t_lo + per, tiles);
     const int* table = st.block_table + (size_t)b * s.max_blocks;
     const int chunks = D / 8;
-    auto load_tile = [&](int t) {
+    constexpr int RPW = LM_KEYS / 8;                                                 // key rows a warp loads per tile
+    // lane i of a warp: where row i of the warp's share of tile t lives in the cache, -1 outside
+    auto look_up = [&](int t) {
+        const int key = t * LM_KEYS + warp * RPW + (lane & (RPW - 1));
+        if (t >= t_hi || key >= kv) return -1ll;
+        const int blk = key / s.block_size, block = table[blk];
+        if (block < 0 || block >= s.num_blocks) {
+            atomicCAS(status, 0, SEQ_BAD_BLOCK);
+            return -1ll;
+        }
+        return ((long long)block * s.block_size + (key - blk * s.block_size)) * D;
+    };
+    auto load_tile = [&](int t, long long where) {
         bf16* dst = reinterpret_cast<bf16*>(lm_smem + lay.tile) + (size_t)((t - t_lo) & 1) * LM_KEYS * lay.ld;
-#pragma unroll 2
-        for (int i = 0; i < LM_KEYS / 8; ++i) {
-            const int key = t * LM_KEYS + warp * (LM_KEYS / 8) + i;
-            bool ok = key < kv;
-            int block = ok ? table[key / s.block_size] : 0;
-            if (block < 0 || block >= s.num_blocks) {
-                if (lane == 0) atomicCAS(status, 0, SEQ_BAD_BLOCK);
-                ok = false;
-                block = 0;
-            }
-            const bf16* src = cache + ((size_t)block * s.block_size + key % s.block_size) * D;
-            const uint32_t row = smem_u32(dst + (size_t)(warp * (LM_KEYS / 8) + i) * lay.ld);
-            for (int c = lane; c < chunks; c += 32) cp_async16(row + c * 16, src + (ok ? c * 8 : 0), ok);
+#pragma unroll
+        for (int i = 0; i < RPW; ++i) {
+            const long long off = __shfl_sync(0xffffffffu, where, i);
+            const bf16* src = cache + (off < 0 ? 0 : off);
+            const uint32_t row = smem_u32(dst + (size_t)(warp * RPW + i) * lay.ld);
+            for (int c = lane; c < chunks; c += 32) cp_async16(row + c * 16, src + c * 8, off >= 0);
         }
     };
     // zero what a key row holds beyond D (the last k step may read it), in both stages and in Q
@@ -97,9 +104,10 @@ __global__ void __launch_bounds__(LM_THREADS) latent_attention_mma_kernel(scr_la
     }
     // cache rows before this step's are there already: their tile does not wait for the preceding kernels
     const bool early = t_lo < t_hi && (t_lo + 1) * LM_KEYS <= pos0;
-    if (early) load_tile(t_lo);
+    if (early) load_tile(t_lo, look_up(t_lo));
     pdl_wait();
-    if (!early && t_lo < t_hi) load_tile(t_lo);
+    if (!early && t_lo < t_hi) load_tile(t_lo, look_up(t_lo));
+    long long where_next = look_up(t_lo + 1);
     for (int i = threadIdx.x; i < ROWS * chunks; i += LM_THREADS) {
         const int row = i / chunks, c = i - row * chunks;
         cp_async16(smem_u32(Q + (size_t)row * lay.ld + c * 8), q + ((size_t)first * s.heads + r0 + (row < nrows ? row : 0)) * D + c * 8, row < nrows);
@@ -111,41 +119,50 @@ __global__ void __launch_bounds__(LM_THREADS) latent_attention_mma_kernel(scr_la
     const int srow = threadIdx.x / TPR, sk0 = (threadIdx.x % TPR) * KPT;              // this thread's softmax row and first key
     const int limit = pos0 + (r0 + min(srow, nrows - 1)) / s.heads;                  // last key the row sees
     float m_run = -INFINITY, l_run = 0.0f;
-    const int mt_s = warp % MT, ng = warp / MT;                                      // S phase: row tile, key group (8 * MT keys)
-    const int ksteps = (D + 15) / 16, lm = lane >> 3, lr = lane & 7;
+    constexpr int KQ = NTW + 1;                                                      // k steps of 16 per quarter of the dimensions
+    const int kq = warp & 3, kh = warp >> 2;                                         // S phase: quarter of the dimensions, half of the keys
+    const int k_lo = kq * KQ, k_n = min(KQ, (D + 15) / 16 - k_lo), lm = lane >> 3, lr = lane & 7;   // (zero from D up to ld)
+    uint32_t qf[MT][KQ][4];
+    cp_async_wait_all();
+    __syncthreads();
+#pragma unroll
+    for (int m = 0; m < MT; ++m)
+#pragma unroll
+        for (int k = 0; k < KQ; ++k) {
+            qf[m][k][0] = qf[m][k][1] = qf[m][k][2] = qf[m][k][3] = 0;
+            if (k < k_n) ldsm_x4(smem_u32(Q + (size_t)(m * 16 + (lm & 1) * 8 + lr) * lay.ld + (k_lo + k) * 16 + (lm >> 1) * 8), qf[m][k]);
+        }
     for (int t = t_lo; t < t_hi; ++t) {
         cp_async_wait_all();
         __syncthreads();
-        if (t + 1 < t_hi) load_tile(t + 1);
+        if (t + 1 < t_hi) load_tile(t + 1, where_next);
         cp_async_commit();
+        where_next = look_up(t + 2);
         const bf16* K = reinterpret_cast<bf16*>(lm_smem + lay.tile) + (size_t)((t - t_lo) & 1) * LM_KEYS * lay.ld;
         {
-            float sc[MT][4] = {};
-            const uint32_t qa = smem_u32(Q + (size_t)(mt_s * 16 + (lm & 1) * 8 + lr) * lay.ld + (lm >> 1) * 8);
-            const uint32_t kb = smem_u32(K + (size_t)(ng * 8 * MT + lr) * lay.ld + lm * 8);
-            for (int ks = 0; ks < ksteps; ks += 2) {                                 // (the row beyond D is zero up to ld)
-                uint32_t a0[4], a1[4] = {0, 0, 0, 0};
-                ldsm_x4(qa + ks * 32, a0);
-                if (ks + 1 < ksteps) ldsm_x4(qa + ks * 32 + 32, a1);
+            float sc[MT][4][4] = {};
+            const uint32_t kb = smem_u32(K + (size_t)(kh * 32 + (lm >> 1) * 8 + lr) * lay.ld + k_lo * 16 + (lm & 1) * 8);
 #pragma unroll
-                for (int n = 0; n < MT; ++n) {
-                    uint32_t kf[4];
-                    if (ks + 1 < ksteps) {
-                        ldsm_x4(kb + n * 8 * lay.ld * 2 + ks * 32, kf);
-                    } else {                                                         // half of the pair only
-                        asm volatile("ldmatrix.sync.aligned.m8n8.x2.shared.b16 {%0,%1}, [%2];" : "=r"(kf[0]), "=r"(kf[1])
-                                     : "r"(smem_u32(K + (size_t)(ng * 8 * MT + n * 8 + lr) * lay.ld + (lm & 1) * 8) + ks * 32));
-                        kf[2] = kf[3] = 0;
-                    }
-                    mma_16816(sc[n], a0[0], a0[1], a0[2], a0[3], kf[0], kf[1]);
-                    if (ks + 1 < ksteps) mma_16816(sc[n], a1[0], a1[1], a1[2], a1[3], kf[2], kf[3]);
+            for (int k = 0; k < KQ; ++k) {
+                if (k < k_n) {
+                    uint32_t kf[2][4];
+#pragma unroll
+                    for (int n2 = 0; n2 < 2; ++n2) ldsm_x4(kb + (uint32_t)(n2 * 16 * lay.ld * 2) + k * 32, kf[n2]);
+#pragma unroll
+                    for (int m = 0; m < MT; ++m)
+#pragma unroll
+                        for (int n = 0; n < 4; ++n)
+                            mma_16816(sc[m][n], qf[m][k][0], qf[m][k][1], qf[m][k][2], qf[m][k][3], kf[n >> 1][(n & 1) * 2], kf[n >> 1][(n & 1) * 2 + 1]);
                 }
             }
-            float* dst = scores + (size_t)(mt_s * 16 + (lane >> 2)) * LM_S_LD + ng * 8 * MT + (lane & 3) * 2;
 #pragma unroll
-            for (int n = 0; n < MT; ++n) {
-                *reinterpret_cast<float2*>(dst + n * 8) = make_float2(sc[n][0], sc[n][1]);
-                *reinterpret_cast<float2*>(dst + 8 * LM_S_LD + n * 8) = make_float2(sc[n][2], sc[n][3]);
+            for (int m = 0; m < MT; ++m) {
+                float* dst = scores + (size_t)(kq * ROWS + m * 16 + (lane >> 2)) * LM_S_LD + kh * 32 + (lane & 3) * 2;
+#pragma unroll
+                for (int n = 0; n < 4; ++n) {
+                    *reinterpret_cast<float2*>(dst + n * 8) = make_float2(sc[m][n][0], sc[m][n][1]);
+                    *reinterpret_cast<float2*>(dst + 8 * LM_S_LD + n * 8) = make_float2(sc[m][n][2], sc[m][n][3]);
+                }
             }
         }
         __syncthreads();
@@ -154,7 +171,10 @@ __global__ void __launch_bounds__(LM_THREADS) latent_attention_mma_kernel(scr_la
 #pragma unroll
             for (int i = 0; i < KPT; ++i) {
                 const int key = t * LM_KEYS + sk0 + i;
-                v[i] = key <= limit && key < kv ? scores[srow * LM_S_LD + sk0 + i] * sl2 : -INFINITY;
+                float sum = 0.0f;
+#pragma unroll
+                for (int p = 0; p < 4; ++p) sum += scores[(p * ROWS + srow) * LM_S_LD + sk0 + i];
+                v[i] = key <= limit && key < kv ? sum * sl2 : -INFINITY;
                 mx = fmaxf(mx, v[i]);
             }
 #pragma unroll
@@ -267,14 +287,21 @@ __global__ void __launch_bounds__(128) latent_attention_merge_kernel(const float
     __syncthreads();
     for (int i = threadIdx.x * 2; i < kv_rank; i += 256) {
         float a = 0.0f, b = 0.0f;
-        for (int k = 0; k < nsplit; ++k)
-            if (w[k] != 0.0f) {                              // (a share without keys)
-                const float2 v = *reinterpret_cast<const float2*>(part_o + (k * all_rows + r) * kv_rank + i);
-                a = fmaf(v.x, w[k], a);
-                b = fmaf(v.y, w[k], b);
-            }
+#pragma unroll 16
+        for (int k = 0; k < nsplit; ++k) {
+            const float2 v = *reinterpret_cast<const float2*>(part_o + (k * all_rows + r) * kv_rank + i);
+            a = fmaf(v.x, w[k], a);
+            b = fmaf(v.y, w[k], b);
+        }
         *reinterpret_cast<uint32_t*>(out + r * kv_rank + i) = pack_bf16x2(a, b);
     }
+}
+
+// The kernel variant of a shape, 0 = none.
+int lm_ntw(const scr_latent_shape& s) {
+    for (int n = 1; n <= 8; n *= 2)
+        if (s.kv_rank <= 64 * n && s.kv_rank + s.rot_dim <= 64 * (n + 1)) return n;
+    return 0;
 }
 
 // Two row tiles share a key tile's loads; one is quicker where even single key tiles would not fill the GPU.
@@ -304,7 +331,7 @@ cudaError_t lm_launch(const scr_latent_shape& s, const scr_step& st, const void*
 
 bool latent_attention_mma_applies(const scr_latent_shape& s) {
     const int D = s.kv_rank + s.rot_dim;
-    return s.kv_rank % 8 == 0 && D % 8 == 0 && s.kv_rank <= 512 && LmSmem::of(D, 2).total <= 227 * 1024;
+    return s.kv_rank % 8 == 0 && D % 8 == 0 && lm_ntw(s) != 0 && LmSmem::of(D, 2).total <= 227 * 1024;
 }
 
 size_t latent_attention_mma_workspace(const scr_latent_shape& s, const scr_step& st, int sms) {
@@ -316,7 +343,7 @@ int32_t latent_attention_mma_launch(scr_ctx* ctx, const scr_latent_shape& s, con
                                     void* workspace, size_t workspace_bytes, cudaStream_t stream) {
     if (st.max_count <= 0 || st.max_kv <= 0 || st.batch <= 0) return scr_fail(ctx, SCR_E_SHAPE, "an empty step");
     if (!scr_aligned16(q) || !scr_aligned16(cache) || !scr_aligned16(out)) return scr_fail(ctx, SCR_E_ALIGN, "q, cache and out must be 16-byte aligned");
-    const int n = lm_splits(s, st, ctx->sm_count), ntw = s.kv_rank <= 64 ? 1 : s.kv_rank <= 128 ? 2 : s.kv_rank <= 256 ? 4 : 8;
+    const int n = lm_splits(s, st, ctx->sm_count), ntw = lm_ntw(s);
     if (n > 1 && (!workspace || workspace_bytes < latent_attention_mma_workspace(s, st, ctx->sm_count)))
         return scr_fail(ctx, SCR_E_WORKSPACE, "latent attention over %d key shares needs %zu bytes", n, latent_attention_mma_workspace(s, st, ctx->sm_count));
     float* po = (float*)workspace;

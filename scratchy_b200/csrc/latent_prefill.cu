@@ -64,7 +64,7 @@ __device__ __forceinline__ void tmem_st_32x32(uint32_t taddr, const uint32_t (&r
 __device__ __forceinline__ void tmem_st_wait() { asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory"); }
 __device__ __forceinline__ float lf_exp2(float x) {
     float y;
-    asm volatile("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
     return y;
 }
 
@@ -97,7 +97,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_co
     auto o_full = [&](int t) { return bars + 8u * (17 + t); };
     volatile uint32_t* tmem_slot = reinterpret_cast<volatile uint32_t*>(gen + L.bars + 8 * 19);
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int head = blockIdx.y, q0 = ((int)gridDim.x - 1 - (int)blockIdx.x) * 256;      // the longest tiles first
+    const int head = blockIdx.x, q0 = ((int)gridDim.y - 1 - (int)blockIdx.y) * 256;      // the longest tiles first
     int n[2];                                                                          // key tiles of the two query tiles
 #pragma unroll
     for (int t = 0; t < 2; ++t) {
@@ -218,10 +218,10 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_co
                 for (int i = 0; i < 64; ++i)
                     if (i > left) v[i] = -INFINITY;
             }
-            float mx = v[0];
+            float m4[4] = {v[0], v[1], v[2], v[3]};
 #pragma unroll
-            for (int i = 1; i < 64; ++i) mx = fmaxf(mx, v[i]);
-            mx *= a.scale_log2;
+            for (int i = 4; i < 64; ++i) m4[i & 3] = fmaxf(m4[i & 3], v[i]);
+            const float mx = fmaxf(fmaxf(m4[0], m4[1]), fmaxf(m4[2], m4[3])) * a.scale_log2;
             if (j == 0) {
                 m_ref = mx;
             } else {
@@ -241,15 +241,15 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_co
                 }
             }
             uint32_t hi[32], lo[32];
-            float sum = 0.0f;
+            float sum[4] = {0.0f, 0.0f, 0.0f, 0.0f};
 #pragma unroll
             for (int i = 0; i < 32; ++i) {
                 const float p0 = lf_exp2(fmaf(v[2 * i], a.scale_log2, -m_ref)), p1 = lf_exp2(fmaf(v[2 * i + 1], a.scale_log2, -m_ref));
-                sum += p0 + p1;
+                sum[i & 3] += p0 + p1;
                 hi[i] = pack_bf16x2(p0, p1);
                 lo[i] = pack_bf16x2(p0 - bf16_lo(hi[i]), p1 - bf16_hi(hi[i]));
             }
-            l += sum;
+            l += (sum[0] + sum[1]) + (sum[2] + sum[3]);
             tmem_st_32x32(ph_col(t) + lanes, hi);
             tmem_st_32x32(pl_col(t) + lanes, lo);
             tmem_st_wait();
@@ -327,7 +327,7 @@ extern "C" int32_t scr_latent_prefill(scr_ctx* ctx, const scr_latent_shape* s, c
         !lf_map(&vm, v_t, kv, s->vdim, H, (uint64_t)ld_v * 2, (uint64_t)ld_v * 2 * s->vdim, a.lay.vp, 1))
         return scr_fail(ctx, SCR_E_CUDA, "latent_prefill: tensor map");
     cudaError_t e = seq_smem(latent_prefill_kernel, a.lay.total);
-    if (e == cudaSuccess) e = launch_pdl(latent_prefill_kernel, dim3(scr_ceil_div(rows, 256), s->heads), dim3(LF_THREADS), a.lay.total, (cudaStream_t)stream, qm, qrm, km, krm, vm, a);
+    if (e == cudaSuccess) e = launch_pdl(latent_prefill_kernel, dim3(s->heads, scr_ceil_div(rows, 256)), dim3(LF_THREADS), a.lay.total, (cudaStream_t)stream, qm, qrm, km, krm, vm, a);
     if (e != cudaSuccess) return scr_fail(ctx, SCR_E_CUDA, "latent_prefill: %s", cudaGetErrorString(e));
     return scr_check_launch(ctx, "latent_prefill");
 }

@@ -14,7 +14,8 @@
 #include <algorithm>
 
 bool mlstm_chunk_applies(const scr_mlstm_shape& s, const scr_step& st);
-int32_t mlstm_chunk_launch(scr_ctx* ctx, const MlstmArgs& a, cudaStream_t stream);
+size_t mlstm_chunk_workspace(const scr_mlstm_shape& s, const scr_step& st, int sms);
+int32_t mlstm_chunk_launch(scr_ctx* ctx, const MlstmArgs& a, void* workspace, size_t workspace_bytes, cudaStream_t stream);
 
 namespace {
 
@@ -168,16 +169,23 @@ int32_t recur_launch(scr_ctx* ctx, const MlstmArgs& a, cudaStream_t stream) {
 
 }  // namespace
 
+extern "C" int32_t scr_mlstm_workspace(int32_t dtype, const scr_mlstm_shape* s, const scr_step* st, size_t* bytes) {
+    if (!s || !st || !bytes) return SCR_E_ARG;
+    *bytes = dtype == SCR_DTYPE_BF16 && mlstm_chunk_applies(*s, *st) ? mlstm_chunk_workspace(*s, *st, tc_sm_count()) : 0;
+    return SCR_OK;
+}
+
 extern "C" int32_t scr_mlstm_run(scr_ctx* ctx, int32_t dtype, const scr_mlstm_shape* s, const scr_step* st, const void* proj, int64_t ld,
                                  const float* gates, int64_t ld_gates, const float* bias_i, const float* bias_f, float* state_s,
-                                 float* state_n, float* state_m, float* out, void* stream) {
+                                 float* state_n, float* state_m, float* out, void* workspace, size_t workspace_bytes,
+                                 void* stream) {
     SCR_REQUIRE_CTX(ctx);
     if (!s || !st || !proj || !gates || !bias_i || !bias_f || !state_s || !state_n || !state_m || !out) return scr_fail(ctx, SCR_E_ARG, "null pointer");
     if (st->rows <= 0 || st->batch <= 0 || s->heads <= 0 || s->dim <= 0 || s->vdim <= 0) return scr_fail(ctx, SCR_E_SHAPE, "mlstm shape");
     const MlstmArgs a{*s, *st, proj, ld, gates, ld_gates, bias_i, bias_f, state_s, state_n, state_m, out, ctx->dev_status};
     if (dtype == SCR_DTYPE_F32) return recur_launch<float>(ctx, a, (cudaStream_t)stream);
     if (dtype != SCR_DTYPE_BF16) return scr_fail(ctx, SCR_E_DTYPE, "dtype %d", dtype);
-    if (mlstm_chunk_applies(*s, *st)) return mlstm_chunk_launch(ctx, a, (cudaStream_t)stream);
+    if (mlstm_chunk_applies(*s, *st)) return mlstm_chunk_launch(ctx, a, workspace, workspace_bytes, (cudaStream_t)stream);
     return recur_launch<bf16>(ctx, a, (cudaStream_t)stream);
 }
 

@@ -161,8 +161,11 @@ class MatrixMemory:
         gates = a.get("mm.gates", (T, 2 * H), torch.float32)
         self.proj(a, h, proj, y2=gates, n_main=n_main)
         out = a.get("mm.out", (T, H * self.vdim), torch.float32)
+        need = ctypes.c_size_t(0)
+        c.check(lib.scr_mlstm_workspace(code, ctypes.byref(shape), ctypes.byref(ctx.step), ctypes.byref(need)))
+        ws = a.get("mm.workspace", (need.value,), torch.uint8) if need.value else None
         c.check(lib.scr_mlstm_run(c.handle, code, ctypes.byref(shape), ctypes.byref(ctx.step), _ptr(proj), n_main, _ptr(gates), 2 * H,
-                                  _ptr(self.bias_i), _ptr(self.bias_f), *(_ptr(t) for t in state), _ptr(out), stream))
+                                  _ptr(self.bias_i), _ptr(self.bias_f), *(_ptr(t) for t in state), _ptr(out), _ptr(ws), need, stream))
         heads = a.get("mm.heads", (T, H * self.vdim), dt)
         gate = ctypes.c_void_p(proj.data_ptr() + qkv * proj.element_size())
         for r0 in range(0, T, 32768):
