@@ -127,7 +127,7 @@ int32_t scr_latent_prefill(scr_ctx* ctx, const scr_latent_shape* s, const void* 
 
 /* ---- matrix-memory recurrence (mLSTM) -----------------------------------------------------------
  * proj (dtype, row stride ld): q [heads * dim] | k [heads * dim] | v [heads * vdim]; gates (f32, row stride ld_gates):
- * input gates [heads] | forget gates [heads], without their biases.  State per slot, f32: S [heads, dim, vdim] and, for
+ * input gates [heads] | forget gates [heads], without their biases (a prompt's call leaves the log gates there).  State per slot, f32: S [heads, dim, vdim] and, for
  * every slice of SCR_MLSTM_SLICE value columns (slices = ceil(vdim / 32)) a copy of the normaliser and of the running
  * maximum, n [heads, slices, dim] and m [heads, slices] (the CTAs of a head then share nothing); a sequence whose rows start at position 0 starts from zero whatever the slot holds.
  * out f32 [rows, heads * vdim]: the readout of every token, before its norm. */
@@ -139,7 +139,7 @@ typedef struct scr_mlstm_shape {
 /* `workspace`: states between the groups of a long prompt that is cut to fill the GPU. */
 int32_t scr_mlstm_workspace(int32_t dtype, const scr_mlstm_shape* s, const scr_step* st, size_t* bytes);
 int32_t scr_mlstm_run(scr_ctx* ctx, int32_t dtype, const scr_mlstm_shape* s, const scr_step* st, const void* proj,
-                      int64_t ld, const float* gates, int64_t ld_gates, const float* bias_i, const float* bias_f,
+                      int64_t ld, float* gates, int64_t ld_gates, const float* bias_i, const float* bias_f,
                       float* state_s, float* state_n, float* state_m, float* out, void* workspace,
                       size_t workspace_bytes, void* stream);
 /* y[t, h, :] (dtype) = out / rms(out over the head) * norm * sigmoid(gate[t, h, :]) */

@@ -116,7 +116,7 @@ __global__ void __launch_bounds__(LM_THREADS) latent_attention_mma_kernel(scr_la
 
     float acc[MT][NTW][4] = {};
     const float sl2 = s.scale * 1.4426950408889634f;
-    const int srow = threadIdx.x / TPR, sk0 = (threadIdx.x % TPR) * KPT;              // this thread's softmax row and first key
+    const int srow = threadIdx.x / TPR, sk0 = (threadIdx.x % TPR) * 4;               // this thread's softmax row; its keys: runs of 4, 4 * TPR apart
     const int limit = pos0 + (r0 + min(srow, nrows - 1)) / s.heads;                  // last key the row sees
     float m_run = -INFINITY, l_run = 0.0f;
     constexpr int KQ = NTW + 1;                                                      // k steps of 16 per quarter of the dimensions
@@ -169,13 +169,24 @@ __global__ void __launch_bounds__(LM_THREADS) latent_attention_mma_kernel(scr_la
         {
             float v[KPT], mx = -INFINITY;
 #pragma unroll
-            for (int i = 0; i < KPT; ++i) {
-                const int key = t * LM_KEYS + sk0 + i;
-                float sum = 0.0f;
+            for (int i = 0; i < KPT; i += 4) {
+                const int k0 = i * TPR + sk0;
+                float4 sum = make_float4(0, 0, 0, 0);
 #pragma unroll
-                for (int p = 0; p < 4; ++p) sum += scores[(p * ROWS + srow) * LM_S_LD + sk0 + i];
-                v[i] = key <= limit && key < kv ? sum * sl2 : -INFINITY;
-                mx = fmaxf(mx, v[i]);
+                for (int p = 0; p < 4; ++p) {
+                    const float4 q4 = *reinterpret_cast<const float4*>(scores + (p * ROWS + srow) * LM_S_LD + k0);
+                    sum.x += q4.x;
+                    sum.y += q4.y;
+                    sum.z += q4.z;
+                    sum.w += q4.w;
+                }
+                const float e[4] = {sum.x, sum.y, sum.z, sum.w};
+#pragma unroll
+                for (int j = 0; j < 4; ++j) {
+                    const int key = t * LM_KEYS + k0 + j;
+                    v[i + j] = key <= limit && key < kv ? e[j] * sl2 : -INFINITY;
+                    mx = fmaxf(mx, v[i + j]);
+                }
             }
 #pragma unroll
             for (int o = 1; o < TPR; o <<= 1) mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, o));
@@ -183,12 +194,15 @@ __global__ void __launch_bounds__(LM_THREADS) latent_attention_mma_kernel(scr_la
             const float keep = m_run == -INFINITY ? 0.0f : exp2_fast(m_run - mn);
             float sum = 0.0f;
 #pragma unroll
-            for (int i = 0; i < KPT; i += 2) {
-                const float p0 = v[i] == -INFINITY ? 0.0f : exp2_fast(v[i] - mn), p1 = v[i + 1] == -INFINITY ? 0.0f : exp2_fast(v[i + 1] - mn);
-                sum += p0 + p1;
-                const uint32_t hi = pack_bf16x2(p0, p1);
-                *reinterpret_cast<uint32_t*>(p_hi + srow * LM_P_LD + sk0 + i) = hi;
-                *reinterpret_cast<uint32_t*>(p_lo + srow * LM_P_LD + sk0 + i) = pack_bf16x2(p0 - bf16_lo(hi), p1 - bf16_hi(hi));
+            for (int i = 0; i < KPT; i += 4) {
+                float p[4];
+#pragma unroll
+                for (int j = 0; j < 4; ++j) p[j] = v[i + j] == -INFINITY ? 0.0f : exp2_fast(v[i + j] - mn);
+                sum += (p[0] + p[1]) + (p[2] + p[3]);
+                const uint32_t h0 = pack_bf16x2(p[0], p[1]), h1 = pack_bf16x2(p[2], p[3]);
+                const size_t at = (size_t)srow * LM_P_LD + i * TPR + sk0;
+                *reinterpret_cast<uint2*>(p_hi + at) = make_uint2(h0, h1);
+                *reinterpret_cast<uint2*>(p_lo + at) = make_uint2(pack_bf16x2(p[0] - bf16_lo(h0), p[1] - bf16_hi(h0)), pack_bf16x2(p[2] - bf16_lo(h1), p[3] - bf16_hi(h1)));
             }
 #pragma unroll
             for (int o = 1; o < TPR; o <<= 1) sum += __shfl_xor_sync(0xffffffffu, sum, o);

@@ -176,7 +176,7 @@ extern "C" int32_t scr_mlstm_workspace(int32_t dtype, const scr_mlstm_shape* s, 
 }
 
 extern "C" int32_t scr_mlstm_run(scr_ctx* ctx, int32_t dtype, const scr_mlstm_shape* s, const scr_step* st, const void* proj, int64_t ld,
-                                 const float* gates, int64_t ld_gates, const float* bias_i, const float* bias_f, float* state_s,
+                                 float* gates, int64_t ld_gates, const float* bias_i, const float* bias_f, float* state_s,
                                  float* state_n, float* state_m, float* out, void* workspace, size_t workspace_bytes,
                                  void* stream) {
     SCR_REQUIRE_CTX(ctx);

@@ -8,7 +8,7 @@ struct MlstmArgs {
     scr_step st;
     const void* proj;
     long long ld;
-    const float* gates;
+    float* gates;
     long long ld_gates;
     const float* bias_i;
     const float* bias_f;

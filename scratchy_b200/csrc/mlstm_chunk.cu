@@ -8,8 +8,8 @@
 // A CTA owns COLS value columns of one head of one sequence and walks chunks; the state slice stays in registers as mma
 // accumulators (f32), with the normaliser n as one more column (its "values" are ones).  What enters a product besides the
 // projections themselves — S, P and the weighted values — is split into a bf16 head and remainder (two products), so
-// state and weights keep about 16 bits on the tensor cores; their sums are f32.  Sixteen warps compute; one more works out
-// the gates of the next chunk meanwhile.  Query, key and value tiles of the next chunk load (cp.async) while this one is
+// state and weights keep about 16 bits on the tensor cores; their sums are f32.  Sixteen warps compute; one more sums up
+// the gates of the next chunk meanwhile (their values come from a small kernel before).  Query, key and value tiles of the next chunk load (cp.async) while this one is
 // computed.
 //
 // The chunks of a head are a chain.  Where heads and slices do not fill the GPU, a long sequence is cut into groups of
@@ -206,17 +206,21 @@ __global__ void __launch_bounds__(CH_THREADS, 1) mlstm_chunk_kernel(MlstmArgs a,
         *reinterpret_cast<uint32_t*>(lo + x) = 0;
     }
     __syncthreads();
+    float next_f[2], next_i[2];                             // log gates of the next chunk, two tokens per lane
+    auto fetch = [&](int c) {
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+            const int t = c * CH_L + lane * 2 + e;
+            const float* z = a.gates + (size_t)(first + t) * a.ld_gates + h;
+            next_i[e] = t < count ? z[0] : -INFINITY;       // past the end: nothing is written or forgotten
+            next_f[e] = t < count ? z[H] : 0.0f;
+        }
+    };
     // Gates of chunk c into their set, by one warp: two tokens per lane, prefix sums and maxima over the warp.
     auto gates = [&](int c) {
         float* F = sets + (c & 1) * SET;
-        const int len = min(CH_L, count - c * CH_L);
-        float f[2], gi[2];
-#pragma unroll
-        for (int e = 0; e < 2; ++e) {
-            const int t = lane * 2 + e, row = first + c * CH_L + t;
-            f[e] = t < len ? mlstm_gate_f(a, row, h) : 0.0f;               // past the end: nothing is forgotten or written
-            gi[e] = t < len ? mlstm_gate_i(a, row, h) : -INFINITY;
-        }
+        float f[2] = {next_f[0], next_f[1]}, gi[2] = {next_i[0], next_i[1]};
+        fetch(c + 1);
         float run = f[0] + f[1];
 #pragma unroll
         for (int o = 1; o < 32; o <<= 1) {
@@ -244,7 +248,10 @@ __global__ void __launch_bounds__(CH_THREADS, 1) mlstm_chunk_kernel(MlstmArgs a,
         m_run = mL;
         f_sum += FL;
     };
-    if (!worker) gates(c_lo);
+    if (!worker) {
+        fetch(c_lo);
+        gates(c_lo);
+    }
 
     const int rt = warp & 3, quarter = (warp >> 2) & 3;     // P and O: 16-row tile, quarter of the keys / columns
     for (int c = c_lo; c < c_hi; ++c) {
@@ -414,6 +421,15 @@ __global__ void __launch_bounds__(CH_THREADS, 1) mlstm_chunk_kernel(MlstmArgs a,
     }
 }
 
+// The log gates in place of the projections' sums: one thread per value.
+__global__ void __launch_bounds__(256) mlstm_gates_kernel(MlstmArgs a) {
+    pdl_trigger();
+    pdl_wait();
+    const int i = blockIdx.x * 256 + threadIdx.x, per = 2 * a.s.heads, row = i / per, c = i - row * per;
+    if (row >= a.st.rows) return;
+    a.gates[row * a.ld_gates + c] = c < a.s.heads ? mlstm_gate_i(a, row, c) : mlstm_gate_f(a, row, c - a.s.heads);
+}
+
 // Columns per CTA and the cut into groups.
 struct ChPlan {
     int cols, groups, chunks;
@@ -476,6 +492,10 @@ int32_t mlstm_chunk_launch(scr_ctx* ctx, const MlstmArgs& a, void* workspace, si
     const ChPlan p = ch_plan(a.s, a.st, ctx->sm_count);
     if (p.bytes > workspace_bytes || (p.bytes && !workspace)) return scr_fail(ctx, SCR_E_WORKSPACE, "mlstm in %d groups needs %zu bytes", p.groups, p.bytes);
     float* ws = (float*)workspace;
+    const cudaError_t e = launch_pdl(mlstm_gates_kernel, dim3(scr_ceil_div(a.st.rows * 2 * a.s.heads, 256)), dim3(256), 0, stream, a);
+    if (e != cudaSuccess) return scr_fail(ctx, SCR_E_CUDA, "mlstm_gates: %s", cudaGetErrorString(e));
+    const int32_t rc = scr_check_launch(ctx, "mlstm_gates");
+    if (rc) return rc;
     if (a.s.dim > 128) return ch_launch<32, 16>(ctx, a, p, ws, stream);
     return p.cols == 64 ? ch_launch<64, 8>(ctx, a, p, ws, stream) : ch_launch<32, 8>(ctx, a, p, ws, stream);
 }
