@@ -34,7 +34,21 @@ extern "C" {
  *   gate (may be NULL): the sum is multiplied by sigmoid(gate[m * ldg + g * y_group + n]) (dtype)
  *   act 1: rows of W hold, per 16, 8 gate rows then the 8 up rows of the same channels; y has N / 2 columns
  *          a sigmoid(alpha a) (b + 1),  a = min(gate, limit), b = clamp(up, -limit, limit)
+ *   n_parts > 0: several linears over one x as one matrix.  Part p takes the columns from the end of part p - 1 to its n_end and
+ *          writes them by its kind to its own y (row stride ld), column n - start of the part; y, y2, gate and act are unused
+ *   residual (may be NULL): residual[m * ld_residual + n] += sum (f32); with tanh_w, y gets the norm of the new residual,
+ *          tanh(tanh_alpha * residual) * tanh_w[n] + tanh_b[n] (dtype), otherwise y is unused
  * `workspace` (f32 slabs of a k-split) may be NULL when `scr_dense_workspace_size` reports 0. */
+#define SCR_PART_STORE 0            /* dtype */
+#define SCR_PART_F32 1              /* f32 */
+#define SCR_PART_SILU 2             /* v sigmoid(v), dtype */
+#define SCR_PART_GELU_GLU 3         /* rows in runs of 8 gate + 8 up as for act 1: gelu_tanh(gate) * up, half the columns, dtype */
+#define SCR_DENSE_PARTS 6
+typedef struct scr_dense_part {
+    void* y;
+    int64_t ld;
+    int32_t n_end, kind;
+} scr_dense_part;
 typedef struct scr_dense {
     const void* w;
     const void* x;
@@ -45,6 +59,13 @@ typedef struct scr_dense {
     int32_t M, N, K, groups;
     int32_t n_main, y_f32, act;
     float limit, alpha;
+    float* residual;
+    int64_t ld_residual;
+    const float* tanh_w;
+    const float* tanh_b;
+    float tanh_alpha;
+    int32_t n_parts;
+    scr_dense_part parts[SCR_DENSE_PARTS];
 } scr_dense;
 int32_t scr_dense_workspace_size(int32_t dtype, int32_t M, int32_t N, int32_t K, int32_t groups, size_t* bytes);
 int32_t scr_dense_linear(scr_ctx* ctx, int32_t dtype, const scr_dense* d, void* workspace, size_t workspace_bytes,
@@ -59,7 +80,8 @@ int32_t scr_seq_embed(scr_ctx* ctx, int32_t dtype, const int32_t* ids, int32_t r
  *   delta, w_delta         x <- x + norm(delta, w_delta)      (delta f32 [rows, width])
  *   delta, no w_delta      x <- delta + bias                  (bias f32 [width] or NULL)
  *   no delta               x unchanged
- * then, with `out` (dtype, row stride ld_out): out <- norm(x, w_out), or the row itself when w_out is NULL.
+ * then, with `out` (dtype, row stride ld_out): out <- norm(x, w_out), or the row itself when w_out is NULL; with b_out the
+ * dynamic tanh instead, out <- tanh(alpha x) * w_out + b_out.
  * `row_index` (may be NULL): out row i is made from row row_index[i] of x (no delta then). */
 typedef struct scr_seq_norm_args {
     float* x;
@@ -72,6 +94,8 @@ typedef struct scr_seq_norm_args {
     int64_t ld_out;
     int32_t rows, x_rows, width;
     float eps;
+    const float* b_out;
+    float alpha;
 } scr_seq_norm_args;
 int32_t scr_seq_norm(scr_ctx* ctx, int32_t dtype, const scr_seq_norm_args* a, void* stream);
 
@@ -145,6 +169,47 @@ int32_t scr_mlstm_run(scr_ctx* ctx, int32_t dtype, const scr_mlstm_shape* s, con
 /* y[t, h, :] (dtype) = out / rms(out over the head) * norm * sigmoid(gate[t, h, :]) */
 int32_t scr_mlstm_finish(scr_ctx* ctx, int32_t dtype, const scr_mlstm_shape* s, const float* out, const float* norm,
                          const void* gate, int64_t ld_gate, int32_t rows, void* y, void* stream);
+
+/* ---- sliding-window attention whose values are its keys before their norm --------------------------
+ * Grouped heads (query head h reads key/value head h / (heads / kv_heads)).  Queries and keys pass a causal convolution of
+ * `taps` taps per channel and an RMS norm over the whole projection; the values are the convolved keys themselves.  The cache
+ * therefore holds the values only, [num_blocks * block_size, kv_heads * dim] of dtype, and one f32 per token, the reciprocal
+ * root mean square of its keys (key_inv); the key norm's weight is folded into the queries.
+ * Position i sees j <= i with i - j < window or j < keep_first.  Score: q.k * scale + bias[h][min(i - j, n_bias - 1)]. */
+typedef struct scr_window_shape {
+    int32_t heads, kv_heads, dim, taps;
+    int32_t window, keep_first, n_bias;
+    int32_t block_size, num_blocks, max_blocks;
+    float eps, scale, out_scale;
+} scr_window_shape;
+/* proj (dtype, row stride ld): q [heads * dim] | k [kv_heads * dim] as projected; conv [taps, (heads + kv_heads) * dim] and
+ * norm [(heads + kv_heads) * dim] f32.  conv_state (dtype) [num_slots, taps - 1, (heads + kv_heads) * dim] holds the last
+ * projected rows of every sequence, oldest first; zeros precede position 0 whatever the slot holds.  Writes the queries
+ * (dtype [rows, heads * dim], normed, times the key norm's weight), the cache rows, key_inv and conv_state. */
+int32_t scr_window_prepare(scr_ctx* ctx, int32_t dtype, const scr_window_shape* s, const scr_step* st, const void* proj, int64_t ld,
+                           const float* conv, const float* norm, void* conv_state, void* q, void* cache, float* key_inv,
+                           void* stream);
+/* out (dtype, row stride ld_out) [rows, heads * dim] = softmax(scores) v * sigmoid(gate[t * ld_gate + h]) * out_scale.
+ * Blocks that no visible key lies in may be missing from the block table (any negative number). */
+int32_t scr_window_attention(scr_ctx* ctx, int32_t dtype, const scr_window_shape* s, const scr_step* st, const void* q, const void* cache,
+                             const float* key_inv, const float* bias, const float* gate, int64_t ld_gate, void* out, int64_t ld_out,
+                             void* stream);
+
+/* ---- matrix memory with a constant decay per head (lightning attention) -----------------------------
+ * S <- decay_h S + k v^T, o = S^T q.  proj (dtype, row stride ld): q [heads * dim] | k [heads * dim] | v [heads * vdim];
+ * powers f32 [heads][SCR_DECAY_POWERS]: decay_h^n.  State per slot f32 [num_slots, heads, dim, vdim]; a sequence whose rows start
+ * at position 0 starts from zero whatever the slot holds.  out f32 [rows, heads * vdim]. */
+#define SCR_DECAY_POWERS 65
+typedef struct scr_lightning_shape {
+    int32_t heads, dim, vdim;
+    float eps, out_scale;
+} scr_lightning_shape;
+int32_t scr_lightning_workspace(int32_t dtype, const scr_lightning_shape* s, const scr_step* st, size_t* bytes);
+int32_t scr_lightning_run(scr_ctx* ctx, int32_t dtype, const scr_lightning_shape* s, const scr_step* st, const void* proj, int64_t ld,
+                          const float* powers, float* state, float* out, void* workspace, size_t workspace_bytes, void* stream);
+/* y[t, :] (dtype, row stride ld_y) = out / rms(out over all heads) * norm * sigmoid(gate[t, :]) * out_scale */
+int32_t scr_lightning_finish(scr_ctx* ctx, int32_t dtype, const scr_lightning_shape* s, const float* out, const float* norm,
+                             const void* gate, int64_t ld_gate, int32_t rows, void* y, int64_t ld_y, void* stream);
 
 #ifdef __cplusplus
 }

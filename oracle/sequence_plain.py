@@ -105,6 +105,93 @@ def dense_mlp(h, w, m):
     return clamped_glu(h @ w["gate"].T, h @ w["up"].T, m["limit"]) @ w["down"].T
 
 
+def dynamic_tanh(x, alpha, w, b):
+    """A norm without statistics: a squashed, scaled and shifted copy of every value."""
+    return np.tanh(alpha * x) * w + b
+
+
+def silu(z):
+    return z * sigmoid(z)
+
+
+def gelu_tanh(z):
+    return 0.5 * z * (1.0 + np.tanh(np.sqrt(2.0 / np.pi) * (z + 0.044715 * z ** 3)))
+
+
+def causal_conv(u, w):
+    """Each channel of u [T, C] with its taps w [C, taps]; the last tap meets the token itself, nothing precedes the first."""
+    taps = w.shape[1]
+    padded = np.concatenate([np.zeros((taps - 1, u.shape[1])), u])
+    return sum(w[:, j] * padded[j:j + u.shape[0]] for j in range(taps))
+
+
+def distance_bucket(n, rows, far):
+    """Row of a bias table of `rows` rows for a key n tokens back: one row per distance in the first half, the second half
+    spaced logarithmically up to `far`."""
+    half = rows // 2
+    if n < half:
+        return n
+    return min(rows - 1, half + int(np.floor(np.log(n / half) / np.log(far / half) * (rows - half) + 1e-12)))
+
+
+def window_visible(T, size, keep_first):
+    """[query, key]: the last `size` tokens up to the query itself, and the first `keep_first` of the sequence."""
+    i, j = np.arange(T)[:, None], np.arange(T)[None, :]
+    return (j <= i) & ((i - j < size) | (j < keep_first))
+
+
+def window_attention(h, w, m, eps):
+    """Grouped heads over a sliding window with kept first tokens.  Queries and keys pass a short convolution and an RMS norm
+    over the whole projection; the values are the keys before that norm; a bias per distance and head joins the scores;
+    each head's output is gated by one number.  -> [T, width]."""
+    T, H, G, dim = h.shape[0], m["heads"], m["kv_heads"], m["dim"]
+    q = causal_conv(h @ w["q"].T, w["q.conv"])
+    k = causal_conv(h @ w["k"].T, w["k.conv"])
+    v = k.reshape(T, G, dim)
+    q = (unit_rms(q, eps) * w["q.norm"]).reshape(T, H, dim)
+    k = (unit_rms(k, eps) * w["k.norm"]).reshape(T, G, dim)
+    rows = np.array([distance_bucket(n, w["rel"].shape[0], m["bias_max"]) for n in range(T)])
+    back = np.maximum(np.arange(T)[:, None] - np.arange(T)[None, :], 0)
+    seen = window_visible(T, m["mask"]["size"], m["mask"]["keep_first"])
+    out = np.zeros((T, H, dim))
+    for head in range(H):
+        g = head // (H // G)
+        score = q[:, head] @ k[:, g].T * m["scale"] + w["rel"][rows[back], head]
+        score = np.where(seen, score, -np.inf)
+        p = np.exp(score - score.max(axis=1, keepdims=True))
+        out[:, head] = (p / p.sum(axis=1, keepdims=True)) @ v[:, g]
+    out *= sigmoid(h @ w["g"].T)[:, :, None]
+    return out.reshape(T, H * dim) @ w["o"].T
+
+
+def decayed_memory(q, k, v, decay):
+    """One head's matrix memory with a constant decay, token by token.  q, k [T, dim], v [T, vdim] -> o [T, vdim]."""
+    S, out = np.zeros((k.shape[1], v.shape[1])), np.zeros((q.shape[0], v.shape[1]))
+    for t in range(q.shape[0]):
+        S = decay * S + np.outer(k[t], v[t])
+        out[t] = S.T @ q[t]
+    return out
+
+
+def lightning_attention(h, w, m, eps):
+    T, H, dim, vdim = h.shape[0], m["heads"], m["dim"], m["vdim"]
+    q, k = (silu(h @ w[n].T).reshape(T, H, dim) for n in ("q", "k"))
+    v = silu(h @ w["v"].T).reshape(T, H, vdim)
+    o = np.concatenate([decayed_memory(q[:, a], k[:, a], v[:, a], m["decay"][a]) for a in range(H)], axis=1)
+    return (unit_rms(o, eps) * w["norm"] * sigmoid(h @ w["g"].T)) @ w["o"].T
+
+
+def side_by_side(h, w, m, eps):
+    """Two mixers over the same input, their outputs added with a scale each."""
+    left = window_attention(h, {k[5:]: v for k, v in w.items() if k.startswith("left.")}, m["left"], eps)
+    right = lightning_attention(h, {k[6:]: v for k, v in w.items() if k.startswith("right.")}, m["right"], eps)
+    return m["left_scale"] * left + m["right_scale"] * right
+
+
+def gelu_mlp(h, w):
+    return (gelu_tanh(h @ w["gate"].T) * (h @ w["up"].T)) @ w["down"].T
+
+
 MIXERS = {"latent_attention": latent_attention, "mlstm": mlstm}
 
 
@@ -147,3 +234,24 @@ def vumipel(cfg, weights, tokens):
             i += 1
     x = norm_around_zero(x, np.asarray(weights["final.norm"], np.float64), cfg["norm"]["eps"])
     return x @ embed.T, runs
+
+
+def tanh_norm_of(weights, name):
+    w, b = (np.asarray(weights[n], np.float64) for n in (name, name + ".b"))
+    return lambda x: dynamic_tanh(x, float(weights[name + ".alpha"]), w, b)
+
+
+def vekurax(cfg, weights, tokens):
+    """Logits [T, vocab] and the residual stream after every layer."""
+    embed, eps = np.asarray(weights["embed"], np.float64), cfg["norm"]["eps"]
+    x, runs = embed[np.asarray(tokens)], []
+    for i, spec in enumerate(cfg["layers"]):
+        while "weights_of" in cfg["layers"][i]:
+            i = cfg["layers"][i]["weights_of"]
+        h = tanh_norm_of(weights, f"l{i}.norm1")(x)
+        y = side_by_side(h, short_names(weights, f"l{i}.mix."), spec["mixer"], eps)
+        if spec.get("mlp") is not None:
+            y = y + gelu_mlp(h, short_names(weights, f"l{i}.mlp."))
+        x = x + y
+        runs.append(x)
+    return tanh_norm_of(weights, "final.norm")(x) @ embed.T, runs

@@ -5,14 +5,13 @@ from __future__ import annotations
 import argparse
 import sys
 
-from . import _lib, trace
+from . import trace
 
 
 def generate(args) -> int:
     from .engine import Engine
-    from .registry import architecture_of, load_model, read_config
-    if architecture_of(read_config(args.model)) != "LlamaForCausalLM":
-        _lib.models_lib(build=True)
+    from .registry import load_model, prepare_library
+    prepare_library(args.model)
     prompts = [[int(t) for t in p.split(",")] for p in args.tokens]
     model = load_model(args.model, "cuda", args.dtype, max_tokens=args.max_tokens, max_sequences=args.max_sequences)
     engine = Engine(model, step_tokens=args.step_tokens, max_batch=args.max_sequences)

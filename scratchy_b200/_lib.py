@@ -113,6 +113,11 @@ MODELS_SIGNATURES = {
     "scr_mlstm_workspace": (_i32, [_i32, _vp, _vp, _psz]),
     "scr_mlstm_run": (_i32, [_vp, _i32, _vp, _vp, _vp, _i64, _vp, _i64, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _sz, _vp]),
     "scr_mlstm_finish": (_i32, [_vp, _i32, _vp, _vp, _vp, _vp, _i64, _i32, _vp, _vp]),
+    "scr_window_prepare": (_i32, [_vp, _i32, _vp, _vp, _vp, _i64, _vp, _vp, _vp, _vp, _vp, _vp, _vp]),
+    "scr_window_attention": (_i32, [_vp, _i32, _vp, _vp, _vp, _vp, _vp, _vp, _vp, _i64, _vp, _i64, _vp]),
+    "scr_lightning_workspace": (_i32, [_i32, _vp, _vp, _psz]),
+    "scr_lightning_run": (_i32, [_vp, _i32, _vp, _vp, _vp, _i64, _vp, _vp, _vp, _vp, _sz, _vp]),
+    "scr_lightning_finish": (_i32, [_vp, _i32, _vp, _vp, _vp, _vp, _i64, _i32, _vp, _i64, _vp]),
 }
 
 
@@ -128,17 +133,29 @@ class TapeLinear(ctypes.Structure):
     _fields_ = [("packed", _vp), ("x", _vp), ("y", _vp), ("N", _i32), ("K", _i32), ("group", _i32), ("dep", _i32 * 3)]
 
 
+PART_STORE, PART_F32, PART_SILU, PART_GELU_GLU = 0, 1, 2, 3
+DENSE_PARTS = 6
+DECAY_POWERS = 65
+
+
+class DensePart(ctypes.Structure):
+    """`scr_dense_part` of include/scratchy_models.h."""
+    _fields_ = [("y", _vp), ("ld", _i64), ("n_end", _i32), ("kind", _i32)]
+
+
 class Dense(ctypes.Structure):
     """`scr_dense` of include/scratchy_models.h."""
     _fields_ = [("w", _vp), ("x", _vp), ("y", _vp), ("y2", _vp), ("gate", _vp), ("ldx", _i64), ("x_group", _i64), ("ldy", _i64),
                 ("y_group", _i64), ("ldy2", _i64), ("ldg", _i64), ("M", _i32), ("N", _i32), ("K", _i32), ("groups", _i32),
-                ("n_main", _i32), ("y_f32", _i32), ("act", _i32), ("limit", ctypes.c_float), ("alpha", ctypes.c_float)]
+                ("n_main", _i32), ("y_f32", _i32), ("act", _i32), ("limit", ctypes.c_float), ("alpha", ctypes.c_float),
+                ("residual", _vp), ("ld_residual", _i64), ("tanh_w", _vp), ("tanh_b", _vp), ("tanh_alpha", ctypes.c_float), ("n_parts", _i32),
+                ("parts", DensePart * DENSE_PARTS)]
 
 
 class SeqNorm(ctypes.Structure):
     """`scr_seq_norm_args` of include/scratchy_models.h."""
     _fields_ = [("x", _vp), ("delta", _vp), ("w_delta", _vp), ("bias", _vp), ("w_out", _vp), ("out", _vp), ("row_index", _vp),
-                ("ld_out", _i64), ("rows", _i32), ("x_rows", _i32), ("width", _i32), ("eps", ctypes.c_float)]
+                ("ld_out", _i64), ("rows", _i32), ("x_rows", _i32), ("width", _i32), ("eps", ctypes.c_float), ("b_out", _vp), ("alpha", ctypes.c_float)]
 
 
 class LatentShape(ctypes.Structure):
@@ -158,7 +175,18 @@ class MlstmShape(ctypes.Structure):
     _fields_ = [("heads", _i32), ("dim", _i32), ("vdim", _i32), ("gate_cap", ctypes.c_float), ("eps", ctypes.c_float)]
 
 
-MODELS_STRUCTS = {"scr_dense": Dense, "scr_seq_norm_args": SeqNorm, "scr_latent_shape": LatentShape, "scr_step": Step,
+class WindowShape(ctypes.Structure):
+    """`scr_window_shape` of include/scratchy_models.h."""
+    _fields_ = [(n, _i32) for n in ("heads", "kv_heads", "dim", "taps", "window", "keep_first", "n_bias", "block_size", "num_blocks",
+                                    "max_blocks")] + [(n, ctypes.c_float) for n in ("eps", "scale", "out_scale")]
+
+
+class LightningShape(ctypes.Structure):
+    """`scr_lightning_shape` of include/scratchy_models.h."""
+    _fields_ = [("heads", _i32), ("dim", _i32), ("vdim", _i32), ("eps", ctypes.c_float), ("out_scale", ctypes.c_float)]
+
+
+MODELS_STRUCTS = {"scr_dense_part": DensePart, "scr_window_shape": WindowShape, "scr_lightning_shape": LightningShape, "scr_dense": Dense, "scr_seq_norm_args": SeqNorm, "scr_latent_shape": LatentShape, "scr_step": Step,
                   "scr_mlstm_shape": MlstmShape}
 
 _lib = None
@@ -182,20 +210,24 @@ def lib() -> ctypes.CDLL:
     return _lib
 
 
-def models_lib(build: bool = False) -> ctypes.CDLL:
-    """The sequence-model library.  `build`: compile it first where it is missing or older than its sources (what a
-    command-line program of a source checkout does); otherwise a missing library raises."""
+def models_lib(build_for: Optional[str] = None) -> ctypes.CDLL:
+    """The sequence-model library.  `build_for` an architecture: where the library is missing or older than its sources, compile
+    the part of it that this architecture runs on (what a command-line program of a source checkout does); otherwise a missing
+    library raises."""
     global _models
     with _lock:
         if _models is None:
-            if build:
-                from .build import MODELS_LIB, build_library
-                build_library(MODELS_LIB)
-            if not os.path.exists(_MODELS_PATH):
-                raise ScratchyCudaError(-5, f"{_MODELS_PATH} is missing: run `python -m scratchy_b200.build` "
+            path = _MODELS_PATH
+            if build_for is not None:
+                from .build import design_library
+                path = design_library(build_for)
+            if not os.path.exists(path):
+                raise ScratchyCudaError(-5, f"{path} is missing: run `python -m scratchy_b200.build` "
                                             "(there is no CPU fallback)")
-            L = ctypes.CDLL(_MODELS_PATH)
+            L = ctypes.CDLL(path)
             for name, (res, args) in {**CONTEXT_SIGNATURES, **MODELS_SIGNATURES}.items():
+                if path != _MODELS_PATH and not hasattr(L, name):
+                    continue                       # the other designs' kernels
                 fn = getattr(L, name)
                 fn.restype, fn.argtypes = res, args
             _models = L

@@ -2,8 +2,8 @@
 decode step) and ``libscratchy_models.so`` (the sequence-model kernels).
 
 Usage: ``python -m scratchy_b200.build [--force] [--verbose]``.  nvcc cross-compiles
-without a GPU; the resulting shared objects sit beside this file.  A program that needs one library only builds that
-one (`build_library`), so its first call compiles no more than it uses.
+without a GPU; the resulting shared objects sit beside this file.  A program that serves one design of a source checkout
+builds a library of that design's kernels only (`design_library`), so its first call compiles no more than it uses.
 """
 from __future__ import annotations
 
@@ -19,9 +19,20 @@ LIB = os.path.join(HERE, "libscratchy_cuda.so")
 MODELS_LIB = os.path.join(HERE, "libscratchy_models.so")
 
 SOURCES = ["context.cu", "abi.cu", "affine_b4.cu", "affine_b4_gemm.cu", "affine_b4_gemm_pair.cu", "fp8.cu", "fp8_gemm.cu", "fp8_gemm_pair.cu", "decode_ops.cu", "tp_comm.cu"]
-MODELS_SOURCES = ["context.cu", "dense_linear.cu", "dense_gemm.cu", "seq_ops.cu", "latent_attention.cu", "latent_attention_mma.cu",
-                  "latent_prefill.cu", "mlstm.cu", "mlstm_chunk.cu"]
-LIBRARIES = {LIB: SOURCES, MODELS_LIB: MODELS_SOURCES}
+MODELS_COMMON = ["context.cu", "dense_linear.cu", "dense_gemm.cu", "seq_ops.cu"]
+# what the layers of a design run on
+DESIGNS = {
+    "Vumipel": ["latent_attention.cu", "latent_attention_mma.cu", "latent_prefill.cu", "mlstm.cu", "mlstm_chunk.cu"],
+    "Vekurax": ["window_attention.cu", "window_attention_mma.cu", "window_prefill.cu", "lightning.cu", "lightning_chunk.cu"],
+}
+MODELS_SOURCES = MODELS_COMMON + [s for sources in DESIGNS.values() for s in sources]
+
+
+def design_path(name: str) -> str:
+    return os.path.join(HERE, f"libscratchy_models_{name.lower()}.so")
+
+
+LIBRARIES = {LIB: SOURCES, MODELS_LIB: MODELS_SOURCES, **{design_path(n): MODELS_COMMON + sources for n, sources in DESIGNS.items()}}
 
 NVCC_FLAGS = [
     "-gencode", "arch=compute_100a,code=sm_100a", "-lineinfo", "-O3", "-std=c++17",
@@ -45,19 +56,34 @@ def _newer(target: str, deps: list[str]) -> bool:
 
 def build(force: bool = False, verbose: bool = False) -> str:
     """Every library of the package."""
-    for target in LIBRARIES:
+    for target in (LIB, MODELS_LIB):
         build_library(target, force, verbose)
     return LIB
+
+
+def design_library(name: str) -> str:
+    """The library to run a design from: the whole one where it is up to date, else one with the design's own sources."""
+    if up_to_date(MODELS_LIB):
+        return MODELS_LIB
+    return build_library(design_path(name))
+
+
+def headers() -> list[str]:
+    found = []
+    for folder in (CSRC, os.path.join(os.path.dirname(HERE), "include")):
+        found += [os.path.join(folder, f) for f in os.listdir(folder) if f.endswith((".cuh", ".h"))]
+    return found
+
+
+def up_to_date(target: str) -> bool:
+    return _newer(target, headers() + [os.path.join(CSRC, s) for s in LIBRARIES[target]])
 
 
 def build_library(target: str, force: bool = False, verbose: bool = False) -> str:
     nvcc = _nvcc()
     os.makedirs(OBJ, exist_ok=True)
-    headers = [os.path.join(CSRC, f) for f in os.listdir(CSRC) if f.endswith((".cuh", ".h"))]
-    include = os.path.join(os.path.dirname(HERE), "include")
-    headers += [os.path.join(include, f) for f in os.listdir(include) if f.endswith(".h")]
-    sources = [s for s in LIBRARIES[target] if os.path.exists(os.path.join(CSRC, s))]
-    if not force and _newer(target, headers + [os.path.join(CSRC, s) for s in sources]):
+    sources, shared = LIBRARIES[target], headers()
+    if not force and up_to_date(target):
         return target
     objs = []
     procs = []
@@ -65,7 +91,7 @@ def build_library(target: str, force: bool = False, verbose: bool = False) -> st
         s = os.path.join(CSRC, src)
         o = os.path.join(OBJ, src.replace(".cu", ".o"))
         objs.append(o)
-        if not force and _newer(o, [s] + headers):
+        if not force and _newer(o, [s] + shared):
             continue
         cmd = [nvcc, *[f for f in NVCC_FLAGS if f != "--use_fast_math=false"], "-c", s, "-o", o]
         if verbose:

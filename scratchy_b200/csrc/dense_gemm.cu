@@ -51,13 +51,75 @@ DgPlan dg_plan(int M, int N, int K, int groups, int sms) {
     return best;
 }
 
-__device__ __forceinline__ void dg_load_3d(uint32_t dst, const CUtensorMap* map, int c0, int c1, int c2, uint32_t bar) {
-    asm volatile("cp.async.bulk.tensor.3d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3, %4}], [%5];"
-                 ::"r"(dst), "l"(map), "r"(c0), "r"(c1), "r"(c2), "r"(bar) : "memory");
+__device__ __forceinline__ uint4 dg_pack8(const float* v) {
+    return make_uint4(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3]), pack_bf16x2(v[4], v[5]), pack_bf16x2(v[6], v[7]));
+}
+
+// The residual end: 32 columns of a row of the stream, and their norm
+__device__ __forceinline__ void dg_residual32(const DenseEnds& e, int m, int n0, int N, float (&v)[32]) {
+    float* r = e.residual + m * e.ld_residual + n0;
+    bf16* h = reinterpret_cast<bf16*>(e.y) + m * e.ldy + n0;
+    if (n0 + 32 <= N && (reinterpret_cast<uintptr_t>(r) & 15) == 0 && (!e.tanh_w || (reinterpret_cast<uintptr_t>(h) & 15) == 0)) {
+#pragma unroll
+        for (int j = 0; j < 32; j += 4) {
+            float4 x = *reinterpret_cast<const float4*>(r + j);
+            v[j] += x.x;
+            v[j + 1] += x.y;
+            v[j + 2] += x.z;
+            v[j + 3] += x.w;
+            *reinterpret_cast<float4*>(r + j) = make_float4(v[j], v[j + 1], v[j + 2], v[j + 3]);
+        }
+        if (!e.tanh_w) return;
+#pragma unroll
+        for (int j = 0; j < 32; ++j) v[j] = fmaf(tanhf(e.tanh_alpha * v[j]), __ldg(e.tanh_w + n0 + j), __ldg(e.tanh_b + n0 + j));
+#pragma unroll
+        for (int j = 0; j < 32; j += 8) *reinterpret_cast<uint4*>(h + j) = dg_pack8(v + j);
+    } else {
+#pragma unroll
+        for (int j = 0; j < 32; ++j)
+            if (n0 + j < N) dense_put<bf16>(e, m, 0, n0 + j, v[j]);
+    }
+}
+
+// Several linears in one matrix: 32 columns, inside one part as a rule
+__device__ __forceinline__ void dg_parts32(const DenseEnds& e, int m, int n0, int N, float (&v)[32]) {
+    int start;
+    const int pi = dense_part(e, n0, start);
+    const scr_dense_part p = e.parts[pi];
+    if (n0 + 32 <= p.n_end) {
+        const bool glu = p.kind == SCR_PART_GELU_GLU;
+        const int cols = glu ? 16 : 32, size = p.kind == SCR_PART_F32 ? 4 : 2;
+        char* dst = reinterpret_cast<char*>(p.y) + (m * p.ld + (glu ? (n0 - start) >> 1 : n0 - start)) * size;
+        if ((reinterpret_cast<uintptr_t>(dst) & 15) == 0 && (!glu || ((n0 - start) & 15) == 0)) {
+            if (p.kind == SCR_PART_F32) {
+#pragma unroll
+                for (int j = 0; j < 32; j += 4) reinterpret_cast<float4*>(dst)[j >> 2] = make_float4(v[j], v[j + 1], v[j + 2], v[j + 3]);
+                return;
+            }
+            if (glu) {
+#pragma unroll
+                for (int j = 0; j < 16; ++j) v[j] = gelu_glu(v[(j >> 3) * 16 + (j & 7)], v[(j >> 3) * 16 + 8 + (j & 7)]);
+            } else if (p.kind == SCR_PART_SILU) {
+#pragma unroll
+                for (int j = 0; j < 32; ++j) v[j] *= sigmoid_f32(v[j]);
+            }
+#pragma unroll
+            for (int j = 0; j < 32; j += 8)
+                if (j < cols) reinterpret_cast<uint4*>(dst)[j >> 3] = dg_pack8(v + j);
+            return;
+        }
+    }
+#pragma unroll
+    for (int j = 0; j < 16; ++j) {
+        const int c = (j >> 3) * 16 + (j & 7);
+        if (n0 + c < N) dense_put_two<bf16>(e, m, 0, n0 + c, N, v[c], v[c + 8]);
+    }
 }
 
 // 32 consecutive columns n0.. of row m: the ends, with 16-byte stores where the destination allows
-__device__ __forceinline__ void dg_store32(const DenseEnds& e, int m, int g, int n0, int N, const float (&v)[32]) {
+__device__ __forceinline__ void dg_store32(const DenseEnds& e, int m, int g, int n0, int N, float (&v)[32]) {
+    if (e.residual) return dg_residual32(e, m, n0, N, v);
+    if (e.n_parts) return dg_parts32(e, m, n0, N, v);
     if (e.act) {
         // columns 0..7 gate, 8..15 up, 16..23 gate, 24..31 up -> channels c0 .. c0 + 16
         const int c0 = (n0 >> 4) * 8;
@@ -146,8 +208,8 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap x_map, const __grid_consta
                     mbar_wait(empty_bar(s), ph ^ 1u, status, TC_ERR_EMPTY_WAIT);
                     const uint32_t sa = smem_base + s * S::kStageBytes;
                     mbar_arrive_expect_tx(full_bar(s), S::kStageBytes);
-                    dg_load_3d(sa, &x_map, kt * 64, g, mt * 128, full_bar(s));
-                    dg_load_3d(sa + DG_A_BYTES, &w_map, kt * 64, nb * BN, g, full_bar(s));
+                    tma_load_3d(sa, &x_map, kt * 64, g, mt * 128, full_bar(s));
+                    tma_load_3d(sa + DG_A_BYTES, &w_map, kt * 64, nb * BN, g, full_bar(s));
                     if (++s == S::kStages) { s = 0; ph ^= 1u; }
                 }
             }
@@ -240,12 +302,7 @@ __global__ void __launch_bounds__(256) dense_gemm_finish_kernel(const float* __r
         a += src[(size_t)k * n_tail * tile_elems];
         b += src[(size_t)k * n_tail * tile_elems + 8];
     }
-    if (ends.act) {
-        dense_put_pair<bf16>(ends, m, n, a, b);
-    } else {
-        dense_put<bf16>(ends, m, g, n, a);
-        if (n + 8 < N) dense_put<bf16>(ends, m, g, n + 8, b);
-    }
+    dense_put_two<bf16>(ends, m, g, n, N, a, b);
 }
 
 bool dg_map(CUtensorMap* map, const void* base, uint64_t d0, uint64_t d1, uint64_t d2, uint64_t s1, uint64_t s2, uint32_t b1, uint32_t b2) {

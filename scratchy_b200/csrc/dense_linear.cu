@@ -56,15 +56,9 @@ __global__ void __launch_bounds__(256) dense_plain_kernel(const T* __restrict__ 
     for (int i = 0; i < 4; ++i) {
         const int m = m0 + ty * 4 + i;
         if (m >= M) continue;
-        if (ends.act) {
 #pragma unroll
-            for (int j = 0; j < 4; j += 2)
-                if (n0 + cbase + 8 * j < N) dense_put_pair<T>(ends, m, n0 + cbase + 8 * j, acc[i][j], acc[i][j + 1]);
-        } else {
-#pragma unroll
-            for (int j = 0; j < 4; ++j)
-                if (n0 + cbase + 8 * j < N) dense_put<T>(ends, m, g, n0 + cbase + 8 * j, acc[i][j]);
-        }
+        for (int j = 0; j < 4; j += 2)
+            if (n0 + cbase + 8 * j < N) dense_put_two<T>(ends, m, g, n0 + cbase + 8 * j, N, acc[i][j], acc[i][j + 1]);
     }
 }
 
@@ -168,11 +162,11 @@ __global__ void __launch_bounds__(MV_WARPS * 32, 2) dense_matvec_kernel(const bf
         for (int c = 1; c < cluster; ++c) v += peers[c - 1][tile][r][m];
         return v;
     };
-    if (ends.act) {
+    if (ends.act || ends.n_parts) {
         for (int i = threadIdx.x; i < tiles * 8 * M; i += MV_WARPS * 32) {
             const int r = i & 7, tile = (i >> 3) % tiles, m = (i >> 3) / tiles;
             const int n = (tile0 + tile) * 16 + r;
-            if (n < N) dense_put_pair<bf16>(ends, m, n, whole(tile, r, m), whole(tile, r + 8, m));
+            if (n < N) dense_put_two<bf16>(ends, m, grp, n, N, whole(tile, r, m), whole(tile, r + 8, m));
         }
     } else {
         for (int i = threadIdx.x; i < tiles * 16 * M; i += MV_WARPS * 32) {
@@ -238,10 +232,21 @@ extern "C" int32_t scr_dense_workspace_size(int32_t dtype, int32_t M, int32_t N,
 extern "C" int32_t scr_dense_linear(scr_ctx* ctx, int32_t dtype, const scr_dense* dp, void* workspace, size_t workspace_bytes,
                                     void* stream) {
     SCR_REQUIRE_CTX(ctx);
-    if (!dp || !dp->w || !dp->x || !dp->y) return scr_fail(ctx, SCR_E_ARG, "null pointer");
+    if (!dp || !dp->w || !dp->x) return scr_fail(ctx, SCR_E_ARG, "null pointer");
     const scr_dense& d = *dp;
+    if (!d.y && !d.n_parts && (!d.residual || d.tanh_w)) return scr_fail(ctx, SCR_E_ARG, "null pointer");
+    if (d.residual && (d.groups != 1 || d.n_parts || d.act || d.gate || d.n_main < d.N || (d.tanh_w && !d.tanh_b)))
+        return scr_fail(ctx, SCR_E_ARG, "a residual end stands alone");
+    if (d.n_parts < 0 || d.n_parts > SCR_DENSE_PARTS) return scr_fail(ctx, SCR_E_ARG, "%d parts", d.n_parts);
+    for (int p = 0, start = 0; p < d.n_parts; start = d.parts[p++].n_end) {
+        const scr_dense_part& q = d.parts[p];
+        if (!q.y || q.kind < SCR_PART_STORE || q.kind > SCR_PART_GELU_GLU) return scr_fail(ctx, SCR_E_ARG, "part %d", p);
+        if (q.n_end <= start || (p + 1 == d.n_parts && q.n_end != d.N) || d.groups != 1 || d.act || d.gate)
+            return scr_fail(ctx, SCR_E_SHAPE, "parts cover the columns of one group in order");
+        if (q.kind == SCR_PART_GELU_GLU && (start % 16 || q.n_end % 16)) return scr_fail(ctx, SCR_E_SHAPE, "gate/up pairs come in runs of 8 + 8 rows");
+    }
     if (d.M <= 0 || d.N <= 0 || d.K <= 0 || d.groups <= 0) return scr_fail(ctx, SCR_E_SHAPE, "empty linear (M %d N %d K %d)", d.M, d.N, d.K);
-    if (d.n_main < d.N && (!d.y2 || d.groups != 1 || d.act)) return scr_fail(ctx, SCR_E_ARG, "a second output needs y2, one group and no activation");
+    if (!d.n_parts && d.n_main < d.N && (!d.y2 || d.groups != 1 || d.act)) return scr_fail(ctx, SCR_E_ARG, "a second output needs y2, one group and no activation");
     if (d.act && (d.N % 16 || d.groups != 1 || d.gate)) return scr_fail(ctx, SCR_E_SHAPE, "gate/up pairs come in runs of 8 + 8 rows");
     cudaStream_t st = (cudaStream_t)stream;
     if (dtype == SCR_DTYPE_F32) return plain_launch<float>(ctx, d, st);

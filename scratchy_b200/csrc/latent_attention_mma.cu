@@ -34,16 +34,6 @@ struct LmSmem {
     }
 };
 
-__device__ __forceinline__ void cp_async16(uint32_t dst, const void* src, bool ok) {
-    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(ok ? 16 : 0) : "memory");
-}
-__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
-__device__ __forceinline__ void cp_async_wait_all() { asm volatile("cp.async.wait_group 0;" ::: "memory"); }
-__device__ __forceinline__ float exp2_fast(float x) {
-    float y;
-    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-    return y;
-}
 
 // MT: 16-row tiles; NTW: 8-column tiles of the latent per warp (kv_rank <= 64 * NTW, kv_rank + rot_dim <= 64 * (NTW + 1))
 template <int MT, int NTW>

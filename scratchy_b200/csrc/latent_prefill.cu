@@ -41,33 +41,6 @@ struct LfLayout {
     }
 };
 
-__device__ __forceinline__ void lf_load_3d(uint32_t dst, const CUtensorMap* map, int c0, int c1, int c2, uint32_t bar) {
-    asm volatile("cp.async.bulk.tensor.3d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3, %4}], [%5];"
-                 ::"r"(dst), "l"(map), "r"(c0), "r"(c1), "r"(c2), "r"(bar) : "memory");
-}
-// D[tmem] (+)= A[tmem] * B[smem]^T
-__device__ __forceinline__ void umma_f16_ta(uint32_t d_tmem, uint32_t a_tmem, uint64_t b_desc, uint32_t idesc, uint32_t accumulate) {
-    asm volatile(
-        "{\n\t.reg .pred p;\n\tsetp.ne.b32 p, %4, 0;\n\t"
-        "tcgen05.mma.cta_group::1.kind::f16 [%0], [%1], %2, %3, p;\n\t}"
-        ::"r"(d_tmem), "r"(a_tmem), "l"(b_desc), "r"(idesc), "r"(accumulate) : "memory");
-}
-__device__ __forceinline__ void tmem_st_32x32(uint32_t taddr, const uint32_t (&r)[32]) {
-    asm volatile(
-        "tcgen05.st.sync.aligned.32x32b.x32.b32 [%0], "
-        "{%1,%2,%3,%4,%5,%6,%7,%8,%9,%10,%11,%12,%13,%14,%15,%16,%17,%18,%19,%20,%21,%22,%23,%24,%25,%26,%27,%28,%29,%30,%31,%32};"
-        ::"r"(taddr), "r"(r[0]), "r"(r[1]), "r"(r[2]), "r"(r[3]), "r"(r[4]), "r"(r[5]), "r"(r[6]), "r"(r[7]), "r"(r[8]), "r"(r[9]),
-        "r"(r[10]), "r"(r[11]), "r"(r[12]), "r"(r[13]), "r"(r[14]), "r"(r[15]), "r"(r[16]), "r"(r[17]), "r"(r[18]), "r"(r[19]), "r"(r[20]),
-        "r"(r[21]), "r"(r[22]), "r"(r[23]), "r"(r[24]), "r"(r[25]), "r"(r[26]), "r"(r[27]), "r"(r[28]), "r"(r[29]), "r"(r[30]), "r"(r[31])
-        : "memory");
-}
-__device__ __forceinline__ void tmem_st_wait() { asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory"); }
-__device__ __forceinline__ float lf_exp2(float x) {
-    float y;
-    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-    return y;
-}
-
 struct LfArgs {
     LfLayout lay;
     int rows, pos0, heads, vdim;
@@ -133,7 +106,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_co
             for (int t = 0; t < 2; ++t)
                 for (int c = 0; c < L.chunks; ++c) {
                     const bool rot = c >= L.dim_chunks;
-                    lf_load_3d(base + (t * L.chunks + c) * LF_Q_CHUNK, rot ? &qr_map : &q_map, (rot ? c - L.dim_chunks : c) * 64, head, q0 + t * 128, q_full());
+                    tma_load_3d(base + (t * L.chunks + c) * LF_Q_CHUNK, rot ? &qr_map : &q_map, (rot ? c - L.dim_chunks : c) * 64, head, q0 + t * 128, q_full());
                 }
             int ks = 0, vs = 0;
             uint32_t kp = 0, vp = 0;
@@ -142,12 +115,12 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_co
                 mbar_arrive_expect_tx(k_full(ks), L.k_bytes());
                 for (int c = 0; c < L.chunks; ++c) {
                     const bool rot = c >= L.dim_chunks;
-                    lf_load_3d(base + L.k + ks * L.k_bytes() + c * LF_K_CHUNK, rot ? &kr_map : &k_map, (rot ? c - L.dim_chunks : c) * 64, rot ? 0 : head, j * LF_KEYS, k_full(ks));
+                    tma_load_3d(base + L.k + ks * L.k_bytes() + c * LF_K_CHUNK, rot ? &kr_map : &k_map, (rot ? c - L.dim_chunks : c) * 64, rot ? 0 : head, j * LF_KEYS, k_full(ks));
                 }
                 if (++ks == L.k_stages) { ks = 0; kp ^= 1u; }
                 mbar_wait(v_empty(vs), vp ^ 1u, a.status, TC_ERR_EMPTY_WAIT);
                 mbar_arrive_expect_tx(v_full(vs), L.v_bytes());
-                lf_load_3d(base + L.v + vs * L.v_bytes(), &v_map, j * LF_KEYS, 0, head, v_full(vs));
+                tma_load_3d(base + L.v + vs * L.v_bytes(), &v_map, j * LF_KEYS, 0, head, v_full(vs));
                 if (++vs == L.v_stages) { vs = 0; vp ^= 1u; }
             }
         }
@@ -227,7 +200,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_co
             } else {
                 const bool grow = mx > m_ref + 8.0f;
                 if (__any_sync(0xffffffffu, grow)) {                                 // PV of the tiles before is complete (s_full)
-                    const float c = grow ? lf_exp2(m_ref - mx) : 1.0f;
+                    const float c = grow ? exp2_fast(m_ref - mx) : 1.0f;
                     if (grow) m_ref = mx;
                     l *= c;
                     for (int c0 = 0; c0 < L.vp; c0 += 32) {
@@ -244,7 +217,7 @@ latent_prefill_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_co
             float sum[4] = {0.0f, 0.0f, 0.0f, 0.0f};
 #pragma unroll
             for (int i = 0; i < 32; ++i) {
-                const float p0 = lf_exp2(fmaf(v[2 * i], a.scale_log2, -m_ref)), p1 = lf_exp2(fmaf(v[2 * i + 1], a.scale_log2, -m_ref));
+                const float p0 = exp2_fast(fmaf(v[2 * i], a.scale_log2, -m_ref)), p1 = exp2_fast(fmaf(v[2 * i + 1], a.scale_log2, -m_ref));
                 sum[i & 3] += p0 + p1;
                 hi[i] = pack_bf16x2(p0, p1);
                 lo[i] = pack_bf16x2(p0 - bf16_lo(hi[i]), p1 - bf16_hi(hi[i]));

@@ -9,13 +9,13 @@
 //   mlstm_chunk.cu       bf16 prompts, 64 tokens at a time on the tensor cores
 //   mlstm_finish_kernel  each head's output over its root mean square, the norm's weight and the output gate
 #include "seq_common.cuh"
-#include "mlstm.cuh"
+#include "memory.cuh"
 
 #include <algorithm>
 
 bool mlstm_chunk_applies(const scr_mlstm_shape& s, const scr_step& st);
 size_t mlstm_chunk_workspace(const scr_mlstm_shape& s, const scr_step& st, int sms);
-int32_t mlstm_chunk_launch(scr_ctx* ctx, const MlstmArgs& a, void* workspace, size_t workspace_bytes, cudaStream_t stream);
+int32_t mlstm_chunk_launch(scr_ctx* ctx, const MemoryArgs& a, void* workspace, size_t workspace_bytes, cudaStream_t stream);
 
 namespace {
 
@@ -24,7 +24,7 @@ namespace {
 constexpr int RC_T = 256, RC_COLS = SCR_MLSTM_SLICE, RC_ROWS = RC_T / 8;
 
 template <typename T>
-__global__ void __launch_bounds__(RC_T) mlstm_recur_kernel(MlstmArgs a) {
+__global__ void __launch_bounds__(RC_T) mlstm_recur_kernel(MemoryArgs a) {
     extern __shared__ float4 rc_smem[];
     const scr_mlstm_shape& s = a.s;
     const int dim = s.dim, vdim = s.vdim;
@@ -156,7 +156,7 @@ __global__ void __launch_bounds__(FIN_T) mlstm_finish_kernel(scr_mlstm_shape s, 
 }
 
 template <typename T>
-int32_t recur_launch(scr_ctx* ctx, const MlstmArgs& a, cudaStream_t stream) {
+int32_t recur_launch(scr_ctx* ctx, const MemoryArgs& a, cudaStream_t stream) {
     const int dim = a.s.dim;
     const size_t smem = (size_t)dim * 8 * 16 + (3 * dim + 4) * sizeof(float) + 8 * 8 * 16;
     if (smem > 220 * 1024) return scr_fail(ctx, SCR_E_UNSUPPORTED, "mlstm dim %d", dim);
@@ -182,7 +182,7 @@ extern "C" int32_t scr_mlstm_run(scr_ctx* ctx, int32_t dtype, const scr_mlstm_sh
     SCR_REQUIRE_CTX(ctx);
     if (!s || !st || !proj || !gates || !bias_i || !bias_f || !state_s || !state_n || !state_m || !out) return scr_fail(ctx, SCR_E_ARG, "null pointer");
     if (st->rows <= 0 || st->batch <= 0 || s->heads <= 0 || s->dim <= 0 || s->vdim <= 0) return scr_fail(ctx, SCR_E_SHAPE, "mlstm shape");
-    const MlstmArgs a{*s, *st, proj, ld, gates, ld_gates, bias_i, bias_f, state_s, state_n, state_m, out, ctx->dev_status};
+    const MemoryArgs a{*s, *st, proj, ld, gates, ld_gates, bias_i, bias_f, state_s, state_n, state_m, out, ctx->dev_status, nullptr};
     if (dtype == SCR_DTYPE_F32) return recur_launch<float>(ctx, a, (cudaStream_t)stream);
     if (dtype != SCR_DTYPE_BF16) return scr_fail(ctx, SCR_E_DTYPE, "dtype %d", dtype);
     if (mlstm_chunk_applies(*s, *st)) return mlstm_chunk_launch(ctx, a, workspace, workspace_bytes, (cudaStream_t)stream);

@@ -90,6 +90,30 @@ __device__ __forceinline__ void ldsm_x4_trans(uint32_t addr, uint32_t (&r)[4]) {
                  : "=r"(r[0]), "=r"(r[1]), "=r"(r[2]), "=r"(r[3]) : "r"(addr));
 }
 
+__device__ __forceinline__ float exp2_fast(float x) {
+    float y;
+    asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+    return y;
+}
+
+// 16 bytes global -> shared (zeros unless ok), in the background
+__device__ __forceinline__ void cp_async16(uint32_t dst, const void* src, bool ok) {
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(ok ? 16 : 0) : "memory");
+}
+__device__ __forceinline__ void cp_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+__device__ __forceinline__ void cp_async_wait_all() { asm volatile("cp.async.wait_group 0;" ::: "memory"); }
+
+// gelu in its tanh form, of the gate, times up
+__device__ __forceinline__ float gelu_glu(float gate, float up) {
+    return 0.5f * gate * (1.0f + tanhf(0.7978845608028654f * (gate + 0.044715f * gate * gate * gate))) * up;
+}
+
+// Tiled TMA load of a 3-D box, completion counted on `bar`
+__device__ __forceinline__ void tma_load_3d(uint32_t dst, const CUtensorMap* map, int c0, int c1, int c2, uint32_t bar) {
+    asm volatile("cp.async.bulk.tensor.3d.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1, {%2, %3, %4}], [%5];"
+                 ::"r"(dst), "l"(map), "r"(c0), "r"(c1), "r"(c2), "r"(bar) : "memory");
+}
+
 // The ends of a dense linear (scr_dense), applied to one finished f32 sum.
 struct DenseEnds {
     void* y;
@@ -98,12 +122,49 @@ struct DenseEnds {
     long long ldy, y_group, ldy2, ldg;
     int n_main, y_f32, act;
     float limit, alpha;
+    float* residual;
+    long long ld_residual;
+    const float* tanh_w;
+    const float* tanh_b;
+    float tanh_alpha;
+    int n_parts;
+    scr_dense_part parts[SCR_DENSE_PARTS];
 };
 static inline DenseEnds dense_ends(const scr_dense& d) {
-    return DenseEnds{d.y, d.y2, d.gate, d.ldy, d.y_group, d.ldy2, d.ldg, d.n_main, d.y_f32, d.act, d.limit, d.alpha};
+    DenseEnds e{d.y, d.y2, d.gate, d.ldy, d.y_group, d.ldy2, d.ldg, d.n_main, d.y_f32, d.act, d.limit, d.alpha,
+                d.residual, d.ld_residual, d.tanh_w, d.tanh_b, d.tanh_alpha, d.n_parts, {}};
+    for (int p = 0; p < d.n_parts && p < SCR_DENSE_PARTS; ++p) e.parts[p] = d.parts[p];
+    return e;
+}
+// The part column n belongs to and the column the part starts at.
+__device__ __forceinline__ int dense_part(const DenseEnds& e, int n, int& start) {
+    int p = 0;
+    start = 0;
+#pragma unroll
+    for (int i = 0; i < SCR_DENSE_PARTS - 1; ++i)
+        if (i + 1 < e.n_parts && n >= e.parts[i].n_end) {
+            p = i + 1;
+            start = e.parts[i].n_end;
+        }
+    return p;
 }
 template <typename T>
 __device__ __forceinline__ void dense_put(const DenseEnds& e, int m, int g, int n, float v) {
+    if (e.residual) {
+        float* r = e.residual + m * e.ld_residual + n;
+        v += *r;
+        *r = v;
+        if (e.tanh_w) reinterpret_cast<T*>(e.y)[m * e.ldy + n] = from_f32<T>(fmaf(tanhf(e.tanh_alpha * v), e.tanh_w[n], e.tanh_b[n]));
+        return;
+    }
+    if (e.n_parts) {
+        int start;
+        const scr_dense_part& p = e.parts[dense_part(e, n, start)];
+        const long long at = m * p.ld + n - start;
+        if (p.kind == SCR_PART_F32) reinterpret_cast<float*>(p.y)[at] = v;
+        else reinterpret_cast<T*>(p.y)[at] = from_f32<T>(p.kind == SCR_PART_SILU ? v * sigmoid_f32(v) : v);
+        return;
+    }
     if (n >= e.n_main) {
         e.y2[m * e.ldy2 + (n - e.n_main)] = v;
         return;
@@ -113,11 +174,25 @@ __device__ __forceinline__ void dense_put(const DenseEnds& e, int m, int g, int 
     if (e.y_f32) reinterpret_cast<float*>(e.y)[m * e.ldy + col] = v;
     else reinterpret_cast<T*>(e.y)[m * e.ldy + col] = from_f32<T>(v);
 }
-// act 1: the gate row n (n % 16 < 8) and its up row n + 8 become channel (n / 16) * 8 + n % 8
+// Columns n (n % 16 < 8) and n + 8 of N.  Where they are a gate and its up they become channel (n / 16) * 8 + n % 8.
 template <typename T>
-__device__ __forceinline__ void dense_put_pair(const DenseEnds& e, int m, int n, float gate, float up) {
-    const int c = (n >> 4) * 8 + (n & 7);
-    const float v = clamped_glu(gate, up, e.limit, e.alpha);
-    if (e.y_f32) reinterpret_cast<float*>(e.y)[m * e.ldy + c] = v;
-    else reinterpret_cast<T*>(e.y)[m * e.ldy + c] = from_f32<T>(v);
+__device__ __forceinline__ void dense_put_two(const DenseEnds& e, int m, int g, int n, int N, float a, float b) {
+    if (e.act) {
+        const int c = (n >> 4) * 8 + (n & 7);
+        const float v = clamped_glu(a, b, e.limit, e.alpha);
+        if (e.y_f32) reinterpret_cast<float*>(e.y)[m * e.ldy + c] = v;
+        else reinterpret_cast<T*>(e.y)[m * e.ldy + c] = from_f32<T>(v);
+        return;
+    }
+    if (e.n_parts) {
+        int start;
+        const scr_dense_part& p = e.parts[dense_part(e, n, start)];
+        if (p.kind == SCR_PART_GELU_GLU) {
+            const int c = n - start;
+            reinterpret_cast<T*>(p.y)[m * p.ld + (c >> 4) * 8 + (c & 7)] = from_f32<T>(gelu_glu(a, b));
+            return;
+        }
+    }
+    dense_put<T>(e, m, g, n, a);
+    if (n + 8 < N) dense_put<T>(e, m, g, n + 8, b);
 }

@@ -97,11 +97,17 @@ __global__ void __launch_bounds__(NORM_T) seq_norm_kernel(scr_seq_norm_args a, i
     if (!a.out) return;
     T* out = reinterpret_cast<T*>(a.out) + r * a.ld_out;
     float inv = 1.0f;
-    if (a.w_out) inv = 1.0f / sqrtf(cta_sum<NORM_T>(sum, red_b) / float(W) + a.eps);
+    if (a.w_out && !a.b_out) inv = 1.0f / sqrtf(cta_sum<NORM_T>(sum, red_b) / float(W) + a.eps);
     for (int i = threadIdx.x * VEC; i < W; i += NORM_T * VEC) {
         float v[VEC], w[VEC];
         get_vec(row + i, v);
-        if (a.w_out) {
+        if (a.b_out) {
+            float b[VEC];
+            get_vec(a.w_out + i, w);
+            get_vec(a.b_out + i, b);
+#pragma unroll
+            for (int j = 0; j < VEC; ++j) v[j] = fmaf(tanhf(a.alpha * v[j]), w[j], b[j]);
+        } else if (a.w_out) {
             get_vec(a.w_out + i, w);
 #pragma unroll
             for (int j = 0; j < VEC; ++j) v[j] = v[j] * inv * (1.0f + w[j]);
@@ -259,13 +265,13 @@ extern "C" int32_t scr_seq_embed(scr_ctx* ctx, int32_t dtype, const int32_t* ids
 extern "C" int32_t scr_seq_norm(scr_ctx* ctx, int32_t dtype, const scr_seq_norm_args* ap, void* stream) {
     SCR_REQUIRE_CTX(ctx);
     SEQ_DTYPE(dtype);
-    if (!ap || !ap->x || (ap->row_index && ap->delta)) return scr_fail(ctx, SCR_E_ARG, "null pointer, or a row index together with a delta");
+    if (!ap || !ap->x || (ap->row_index && ap->delta) || (ap->b_out && !ap->w_out)) return scr_fail(ctx, SCR_E_ARG, "null pointer, or a row index together with a delta");
     const scr_seq_norm_args& a = *ap;
     if (a.rows <= 0 || a.width <= 0) return scr_fail(ctx, SCR_E_SHAPE, "empty norm");
     const size_t smem = (size_t)a.width * sizeof(float);
     if (smem > 200 * 1024) return scr_fail(ctx, SCR_E_UNSUPPORTED, "width %d", a.width);
     const bool vec = a.width % 4 == 0 && a.ld_out % 4 == 0 && scr_aligned16(a.x) && scr_aligned16(a.delta) && scr_aligned16(a.w_delta) &&
-                     scr_aligned16(a.bias) && scr_aligned16(a.w_out) && scr_aligned16(a.out);
+                     scr_aligned16(a.bias) && scr_aligned16(a.w_out) && scr_aligned16(a.b_out) && scr_aligned16(a.out);
     auto kernel = dtype == SCR_DTYPE_F32 ? (vec ? seq_norm_kernel<float, 4> : seq_norm_kernel<float, 1>) : (vec ? seq_norm_kernel<bf16, 4> : seq_norm_kernel<bf16, 1>);
     cudaError_t e = seq_smem(kernel, smem);
     if (e != cudaSuccess) return scr_fail(ctx, SCR_E_CUDA, "seq_norm: %s", cudaGetErrorString(e));

@@ -3,7 +3,7 @@ from __future__ import annotations
 
 import ctypes
 from dataclasses import dataclass
-from typing import Dict, List, Optional, Sequence as Seq
+from typing import Dict, List, Optional, Sequence as Seq, Tuple
 
 import torch
 
@@ -132,12 +132,60 @@ class DenseLinear:
                        self.in_features, self.groups, self.out_features if n_main is None else n_main,
                        int(y.dtype == torch.float32 and w.dtype != torch.float32), int(self.glu_limit is not None),
                        self.glu_limit if self.glu_limit is not None else 0.0, self.glu_alpha)
+        self._launch(arena, code, d)
+        return y
+
+    def _launch(self, arena: Arena, code: int, d: "_lib.Dense") -> None:
+        w = self.weight
         lib, ctx = _lib.models_lib(), _lib.models_context(_dev_index(w.device))
         need = ctypes.c_size_t(0)
-        ctx.check(lib.scr_dense_workspace_size(code, M, self.out_features, self.in_features, self.groups, ctypes.byref(need)))
+        ctx.check(lib.scr_dense_workspace_size(code, d.M, d.N, d.K, self.groups, ctypes.byref(need)))
         ws = arena.get("dense.workspace", (need.value,), torch.uint8) if need.value else None
         ctx.check(lib.scr_dense_linear(ctx.handle, code, ctypes.byref(d), _ptr(ws), need, _stream(w.device)))
-        return y
+
+    def add_to(self, arena: Arena, x: torch.Tensor, residual: torch.Tensor, norm: Optional["TanhNorm"] = None,
+               out: Optional[torch.Tensor] = None) -> None:
+        """residual (f32) += x W^T, and with `norm` the norm of the new residual into `out`."""
+        d = _lib.Dense(self.weight.data_ptr(), x.data_ptr(), 0 if norm is None else out.data_ptr(), 0, 0, int(x.stride(0)), 0,
+                       0 if norm is None else int(out.stride(0)), 0, 0, 0, int(x.shape[0]), self.out_features, self.in_features, 1, self.out_features)
+        d.residual, d.ld_residual = residual.data_ptr(), int(residual.stride(0))
+        if norm is not None:
+            d.tanh_w, d.tanh_b, d.tanh_alpha = norm.w.data_ptr(), norm.b.data_ptr(), norm.alpha
+        self._launch(arena, dtype_code(self.weight.dtype), d)
+
+
+class JoinedLinear(DenseLinear):
+    """Several linears of one input as one matrix.  `parts`: (name, rows, kind) in order of their columns; a gate/up pair
+    (`interleave8`) comes first or after a multiple of 16 columns."""
+
+    def __init__(self, parts: Seq[Tuple[str, torch.Tensor, int]]):
+        super().__init__(torch.cat([w for _, w, _ in parts]))
+        self.parts, n = {}, 0
+        for name, w, kind in parts:
+            n += int(w.shape[0])
+            self.parts[name] = (n, kind)
+
+    def run(self, arena: Arena, x: torch.Tensor, outs: Dict[str, torch.Tensor]) -> None:
+        """`outs`: a 2-D tensor with dense rows for every part."""
+        d = _lib.Dense(self.weight.data_ptr(), x.data_ptr())
+        d.ldx, d.M, d.N, d.K, d.groups, d.n_main = int(x.stride(0)), int(x.shape[0]), self.out_features, self.in_features, 1, self.out_features
+        d.n_parts = len(self.parts)
+        for p, (name, (n_end, kind)) in enumerate(self.parts.items()):
+            d.parts[p] = _lib.DensePart(outs[name].data_ptr(), int(outs[name].stride(0)), n_end, kind)
+        self._launch(arena, dtype_code(self.weight.dtype), d)
+
+
+@dataclass
+class TanhNorm:
+    """Dynamic tanh in place of a norm: tanh(alpha x) * w + b."""
+    alpha: float
+    w: torch.Tensor
+    b: torch.Tensor
+
+    @classmethod
+    def take(cls, weights, name: str) -> "TanhNorm":
+        return cls(float(weights.take(f"{name}.alpha").float().reshape(())), weights.take(name).float().contiguous(),
+                   weights.take(f"{name}.b").float().contiguous())
 
 
 def seq_embed(ids: torch.Tensor, table: torch.Tensor, x: torch.Tensor, raw: Optional[torch.Tensor] = None) -> None:
@@ -150,11 +198,13 @@ def seq_embed(ids: torch.Tensor, table: torch.Tensor, x: torch.Tensor, raw: Opti
 
 def seq_norm(x: torch.Tensor, eps: float, *, delta: Optional[torch.Tensor] = None, w_delta: Optional[torch.Tensor] = None,
              bias: Optional[torch.Tensor] = None, out: Optional[torch.Tensor] = None, w_out: Optional[torch.Tensor] = None,
-             row_index: Optional[torch.Tensor] = None, out_dtype: Optional[torch.dtype] = None) -> None:
-    """The step between two sublayers on the f32 residual (`scr_seq_norm`)."""
+             row_index: Optional[torch.Tensor] = None, out_dtype: Optional[torch.dtype] = None, tanh: Optional[TanhNorm] = None) -> None:
+    """The step between two sublayers on the f32 residual (`scr_seq_norm`); `tanh` in place of `w_out`."""
+    if tanh is not None:
+        w_out = tanh.w
     rows = int(x.shape[0]) if row_index is None else int(row_index.shape[0])
     a = _lib.SeqNorm(x.data_ptr(), *(0 if t is None else t.data_ptr() for t in (delta, w_delta, bias, w_out, out, row_index)),
-                     0 if out is None else int(out.stride(0)), rows, int(x.shape[0]), int(x.shape[1]), eps)
+                     0 if out is None else int(out.stride(0)), rows, int(x.shape[0]), int(x.shape[1]), eps, 0 if tanh is None else tanh.b.data_ptr(), 0.0 if tanh is None else tanh.alpha)
     ctx = _lib.models_context(_dev_index(x.device))
     ctx.check(_lib.models_lib().scr_seq_norm(ctx.handle, dtype_code(out_dtype or (torch.float32 if out is None else out.dtype)),
                                              ctypes.byref(a), _stream(x.device)))

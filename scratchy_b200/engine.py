@@ -73,16 +73,20 @@ class Engine:
         if any(not 0 <= t < self.model.vocab for t in prompt):
             raise ValueError("token id outside the vocabulary")
         longest = len(prompt) + max_new_tokens
-        if -(-longest // self.table.block_size) > self.table.num_blocks:
+        if self.table.most_blocks(longest, self._portion) > self.table.num_blocks:
             raise ValueError(f"{longest} tokens do not fit a cache of {self.table.num_blocks * self.table.block_size}")
         self._serial += 1
         req = Request(name if name is not None else ("request", self._serial), list(prompt), max_new_tokens, tuple(stop_ids))
         self.waiting.append(req)
         return req
 
+    @property
+    def _portion(self) -> int:
+        return min(self.step_tokens, self.model.max_portion)
+
     def _blocks_to_finish(self, req: Request, seq: Optional[Sequence]) -> int:
-        have = len(seq.blocks) if seq is not None else 0
-        return max(0, -(-(len(req.prompt) + req.max_new_tokens) // self.table.block_size) - have)
+        have = seq.held if seq is not None else 0
+        return max(0, self.table.most_blocks(len(req.prompt) + req.max_new_tokens, self._portion) - have)
 
     def _admit(self) -> None:
         """Waiting requests in order, each only if everything that runs can still finish: a running sequence never has to be

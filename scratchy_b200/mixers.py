@@ -1,18 +1,21 @@
 """Sequence mixers and feed-forwards that hybrid models are put together from.  A mixer reads the normed rows of a step
-and writes its f32 output; what it remembers between steps (cache rows, recurrent state) lives in `HybridState`.
+and writes its f32 output; what it remembers between steps (its `memory`: cache rows, recurrent state) lives in `HybridState`.
+
+`WindowAttention`, `LightningAttention` and `GeluGlu` are for layers that run side by side: they state their input linears as
+parts of one matrix (`inputs`), work on its outputs (`run`), and leave their rows for an output linear they share (`o`).
 
 Tensor names are relative to the mixer's prefix in the checkpoint."""
 from __future__ import annotations
 
 import ctypes
 from dataclasses import dataclass
-from typing import Dict, Tuple
+from typing import Dict, List, Tuple
 
 import numpy as np
 import torch
 
 from . import _lib
-from .dense import Arena, DenseLinear, StepInputs, dtype_code, interleave8
+from .dense import Arena, DenseLinear, JoinedLinear, StepInputs, dtype_code, interleave8
 from .layers import GpuWeights, _dev_index, _ptr, _stream
 
 _tables: Dict[tuple, Tuple[torch.Tensor, torch.Tensor]] = {}
@@ -46,8 +49,6 @@ class LatentAttention:
     key part per token.  Few rows: attention in the latent space (W_uk folded into the queries, W_uv applied after).
     Prompts in bf16: keys and values are expanded per sequence and a tensor-core prompt kernel runs over them."""
 
-    EXPAND_FROM = 64                 # rows of one sequence from which the expanded form pays
-
     def __init__(self, weights: GpuWeights, prefix: str, spec: dict, eps: float, dtype: torch.dtype, max_pos: int):
         rot = spec["rot"]
         self.heads, self.dim, self.rot_dim = int(spec["heads"]), int(spec["dim"]), int(spec["rot_dim"])
@@ -69,6 +70,9 @@ class LatentAttention:
     def row_size(self) -> int:
         """Values a token's cache row holds."""
         return self.kv_rank + self.rot_dim
+
+    def memory(self, cache_rows: int, slots: int, device) -> torch.Tensor:
+        return torch.zeros((cache_rows, self.row_size), dtype=self.dtype, device=device)
 
     def shape(self, ctx: StepContext) -> "_lib.LatentShape":
         return _lib.LatentShape(self.heads, self.dim, self.rot_dim, self.vdim, self.kv_rank, self.q_rank, self.rot_dims, self.max_pos,
@@ -150,6 +154,9 @@ class MatrixMemory:
                 torch.zeros((slots, H, self.slices, self.dim), dtype=f32, device=device),
                 torch.zeros((slots, H, self.slices), dtype=f32, device=device))
 
+    def memory(self, cache_rows: int, slots: int, device) -> Tuple[torch.Tensor, ...]:
+        return self.state(slots, device)
+
     def run(self, ctx: StepContext, h: torch.Tensor, state: Tuple[torch.Tensor, ...], y: torch.Tensor) -> None:
         a, T, H, dt = ctx.arena, ctx.rows, self.heads, self.dtype
         lib, c = _lib.models_lib(), _lib.models_context(_dev_index(h.device))
@@ -193,3 +200,186 @@ class ClampedGlu:
         act = arena.get("ff.act", (int(h.shape[0]), self.ff), h.dtype)
         self.gate_up(arena, h, act)
         self.down(arena, act, y)
+
+
+Part = Tuple[str, torch.Tensor, int]                # (name, rows, kind) of a `JoinedLinear`
+
+
+def distance_buckets(rows: int, far: float) -> List[int]:
+    """Row of a `rows`-row bias table for every key distance 0, 1, ... up to the first that takes the last row for good: one
+    row per distance in the first half, the others spaced logarithmically up to `far`."""
+    half, out = rows // 2, []
+    while not out or out[-1] < rows - 1:
+        n = len(out)
+        if n < half:
+            out.append(n)
+        elif half == 0 or far <= half:
+            out.append(rows - 1)
+        else:                                       # (a quotient that is a whole number stays one)
+            out.append(min(rows - 1, half + int(np.floor(np.log(n / half) / np.log(far / half) * (rows - half) + 1e-12))))
+    return out
+
+
+class WindowAttention:
+    """Grouped-head attention over a sliding window and the sequence's first tokens.  Queries and keys pass a short causal
+    convolution and an RMS norm over the whole projection, the values are the keys before that norm, a bias per head and
+    distance bucket joins the scores, one sigmoid per head gates the output (times `out_scale`).
+
+    The cache holds the values and one reciprocal root mean square per token; a slot holds the last projected rows."""
+
+    def __init__(self, weights: GpuWeights, prefix: str, spec: dict, eps: float, dtype: torch.dtype, out_scale: float = 1.0):
+        self.heads, self.kv_heads, self.dim, self.taps = int(spec["heads"]), int(spec["kv_heads"]), int(spec["dim"]), int(spec["conv"])
+        self.window, self.keep_first = int(spec["mask"]["size"]), int(spec["mask"]["keep_first"])
+        self.scale, self.out_scale, self.eps, self.dtype, self.prefix = float(spec["scale"]), float(out_scale), float(eps), dtype, prefix
+        if self.heads % self.kv_heads:
+            raise ValueError(f"{prefix}: {self.heads} heads do not share {self.kv_heads} key/value heads evenly")
+        if int(spec["vdim"]) != self.dim:
+            raise ValueError(f"{prefix}: values that are keys have their size, not {spec['vdim']}")
+        take = lambda name: weights.take(f"{prefix}.{name}")
+        self.qk, self.g, self.o = torch.cat([take("q"), take("k")]).to(dtype), take("g").to(dtype), take("o").to(dtype)
+        self.norm = torch.cat([take("q.norm"), take("k.norm")]).float().contiguous()
+        self.conv = torch.cat([take("q.conv"), take("k.conv")]).float().t().contiguous()
+        if tuple(self.conv.shape) != (self.taps, self.channels):
+            raise ValueError(f"{prefix}: convolution {tuple(self.conv.shape)}, the configuration says {(self.taps, self.channels)}")
+        rel = take("rel").float()
+        self.bias = rel[torch.tensor(distance_buckets(int(rel.shape[0]), float(spec["bias_max"])), device=rel.device)].t().contiguous()
+
+    @property
+    def channels(self) -> int:
+        return (self.heads + self.kv_heads) * self.dim
+
+    @property
+    def out_features(self) -> int:
+        return self.heads * self.dim
+
+    def inputs(self) -> List[Part]:
+        return [(f"{self.prefix}.qk", self.qk, _lib.PART_STORE), (f"{self.prefix}.g", self.g, _lib.PART_F32)]
+
+    def buffers(self, ctx: StepContext) -> Dict[str, torch.Tensor]:
+        return {f"{self.prefix}.qk": ctx.arena.get("wa.qk", (ctx.rows, self.channels), self.dtype),
+                f"{self.prefix}.g": ctx.arena.get("wa.g", (ctx.rows, self.heads), torch.float32)}
+
+    def memory(self, cache_rows: int, slots: int, device) -> Tuple[torch.Tensor, ...]:
+        """(values, reciprocals, projected rows)."""
+        return (torch.zeros((cache_rows, self.kv_heads * self.dim), dtype=self.dtype, device=device),
+                torch.zeros(cache_rows, dtype=torch.float32, device=device),
+                torch.zeros((slots, max(1, self.taps - 1), self.channels), dtype=self.dtype, device=device))
+
+    def shape(self, ctx: StepContext) -> "_lib.WindowShape":
+        return _lib.WindowShape(self.heads, self.kv_heads, self.dim, self.taps, self.window, self.keep_first, int(self.bias.shape[1]),
+                                ctx.block_size, ctx.num_blocks, ctx.inputs.max_blocks, self.eps, self.scale, self.out_scale)
+
+    def run(self, ctx: StepContext, bufs: Dict[str, torch.Tensor], memory, out: torch.Tensor) -> None:
+        """`out`: the gated heads [rows, heads * dim], dense rows of any stride."""
+        qk, gate = bufs[f"{self.prefix}.qk"], bufs[f"{self.prefix}.g"]
+        cache, inv, rows = memory
+        lib, c = _lib.models_lib(), _lib.models_context(_dev_index(qk.device))
+        code, stream, ps, pt = dtype_code(self.dtype), _stream(qk.device), ctypes.byref(self.shape(ctx)), ctypes.byref(ctx.step)
+        q = ctx.arena.get("wa.q", (ctx.rows, self.heads * self.dim), self.dtype)
+        c.check(lib.scr_window_prepare(c.handle, code, ps, pt, _ptr(qk), int(qk.stride(0)), _ptr(self.conv), _ptr(self.norm), _ptr(rows), _ptr(q), _ptr(cache),
+                                       _ptr(inv), stream))
+        c.check(lib.scr_window_attention(c.handle, code, ps, pt, _ptr(q), _ptr(cache), _ptr(inv), _ptr(self.bias), _ptr(gate), int(gate.stride(0)), _ptr(out),
+                                         int(out.stride(0)), stream))
+
+
+class LightningAttention:
+    """Linear attention with a constant decay per head: a matrix state in f32, one slot per sequence; the concatenated readouts
+    pass one RMS norm and a sigmoid gate (times `out_scale`)."""
+
+    def __init__(self, weights: GpuWeights, prefix: str, spec: dict, eps: float, dtype: torch.dtype, out_scale: float = 1.0):
+        self.heads, self.dim, self.vdim = int(spec["heads"]), int(spec["dim"]), int(spec["vdim"])
+        self.out_scale, self.eps, self.dtype, self.prefix = float(out_scale), float(eps), dtype, prefix
+        take = lambda name: weights.take(f"{prefix}.{name}")
+        self.qkv = torch.cat([take(n) for n in ("q", "k", "v")]).to(dtype)
+        self.g, self.o, self.norm = take("g").to(dtype), take("o").to(dtype), take("norm").float().contiguous()
+        decay = np.asarray(spec["decay"], dtype=np.float64)
+        if decay.shape != (self.heads,):
+            raise ValueError(f"{prefix}: {decay.size} decays for {self.heads} heads")
+        powers = decay[:, None] ** np.arange(_lib.DECAY_POWERS)[None, :]
+        self.powers = torch.from_numpy(powers.astype(np.float32)).to(self.norm.device).contiguous()
+
+    @property
+    def out_features(self) -> int:
+        return self.heads * self.vdim
+
+    def inputs(self) -> List[Part]:
+        return [(f"{self.prefix}.qkv", self.qkv, _lib.PART_SILU), (f"{self.prefix}.g", self.g, _lib.PART_STORE)]
+
+    def buffers(self, ctx: StepContext) -> Dict[str, torch.Tensor]:
+        return {f"{self.prefix}.qkv": ctx.arena.get("li.qkv", (ctx.rows, self.heads * (2 * self.dim + self.vdim)), self.dtype),
+                f"{self.prefix}.g": ctx.arena.get("li.g", (ctx.rows, self.out_features), self.dtype)}
+
+    def memory(self, cache_rows: int, slots: int, device) -> torch.Tensor:
+        return torch.zeros((slots, self.heads, self.dim, self.vdim), dtype=torch.float32, device=device)
+
+    def run(self, ctx: StepContext, bufs: Dict[str, torch.Tensor], memory: torch.Tensor, out: torch.Tensor) -> None:
+        qkv, gate = bufs[f"{self.prefix}.qkv"], bufs[f"{self.prefix}.g"]
+        lib, c = _lib.models_lib(), _lib.models_context(_dev_index(qkv.device))
+        code, stream = dtype_code(self.dtype), _stream(qkv.device)
+        shape = _lib.LightningShape(self.heads, self.dim, self.vdim, self.eps, self.out_scale)
+        o = ctx.arena.get("li.out", (ctx.rows, self.out_features), torch.float32)
+        need = ctypes.c_size_t(0)
+        c.check(lib.scr_lightning_workspace(code, ctypes.byref(shape), ctypes.byref(ctx.step), ctypes.byref(need)))
+        ws = ctx.arena.get("li.workspace", (need.value,), torch.uint8) if need.value else None
+        c.check(lib.scr_lightning_run(c.handle, code, ctypes.byref(shape), ctypes.byref(ctx.step), _ptr(qkv), int(qkv.stride(0)), _ptr(self.powers), _ptr(memory),
+                                      _ptr(o), _ptr(ws), need, stream))
+        c.check(lib.scr_lightning_finish(c.handle, code, ctypes.byref(shape), _ptr(o), _ptr(self.norm), _ptr(gate), int(gate.stride(0)), ctx.rows, _ptr(out),
+                                         int(out.stride(0)), stream))
+
+
+class GeluGlu:
+    """Dense feed-forward gelu(gate) * up; the activation is an end of its input part."""
+
+    def __init__(self, weights: GpuWeights, prefix: str, spec: dict, dtype: torch.dtype):
+        if spec["kind"] != "dense":
+            raise ValueError(f"feed-forward kind {spec['kind']!r} is not supported")
+        self.prefix = prefix
+        take = lambda name: weights.take(f"{prefix}.{name}").to(dtype)
+        self.gate_up, self.o = interleave8(take("gate"), take("up")), take("down")
+        pad = int(self.gate_up.shape[0]) // 2 - int(self.o.shape[1])
+        if pad:                                            # channels were padded to whole runs of 8
+            self.o = torch.cat([self.o, torch.zeros((self.o.shape[0], pad), dtype=dtype, device=self.o.device)], 1)
+
+    @property
+    def out_features(self) -> int:
+        return int(self.o.shape[1])
+
+    def inputs(self) -> List[Part]:
+        return [(f"{self.prefix}.act", self.gate_up, _lib.PART_GELU_GLU)]
+
+
+class SideBySide:
+    """Two mixers and, where there is one, a feed-forward over the same input: one matrix before them, one after them, whose sum
+    joins the residual.  The mixers' scales are in their `out_scale`."""
+
+    def __init__(self, mixers, mlp=None):
+        self.mixers, self.mlp = list(mixers), mlp
+        branches = self.mixers + ([mlp] if mlp is not None else [])
+        parts = [p for b in reversed(branches) for p in b.inputs()]                  # the feed-forward's pairs first
+        self.inp = JoinedLinear(sorted(parts, key=lambda p: p[2] == _lib.PART_F32))  # few, narrow f32 columns last
+        self.out = DenseLinear(torch.cat([b.o for b in branches], 1))
+        self.columns, at = [], 0
+        for b in branches:
+            self.columns.append((at, at + b.out_features))
+            at += b.out_features
+            for name in ("qk", "qkv", "g", "gate_up", "o"):                          # the joined matrices hold them now
+                if hasattr(b, name):
+                    setattr(b, name, None)
+
+    def memory(self, cache_rows: int, slots: int, device) -> list:
+        return [m.memory(cache_rows, slots, device) for m in self.mixers]
+
+    def run(self, ctx: StepContext, h: torch.Tensor, memory: list, residual: torch.Tensor, norm=None) -> None:
+        """`residual` += the layer's output; with `norm` (a `TanhNorm`) `h` becomes the norm of the new residual."""
+        a = ctx.arena
+        rows = a.get("side.rows", (ctx.rows, self.out.in_features), h.dtype)
+        bufs = {}
+        for m in self.mixers:
+            bufs.update(m.buffers(ctx))
+        if self.mlp is not None:
+            lo, hi = self.columns[-1]
+            bufs[f"{self.mlp.prefix}.act"] = rows[:, lo:hi]
+        self.inp.run(a, h, bufs)
+        for m, mem, (lo, hi) in zip(self.mixers, memory, self.columns):
+            m.run(ctx, bufs, mem, rows[:, lo:hi])
+        self.out.add_to(a, rows, residual, norm, h)

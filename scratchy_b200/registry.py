@@ -12,6 +12,7 @@ import os
 # architecture name in config.json -> module, class (imported on use)
 ARCHITECTURES = {
     "Vumipel": ("scratchy_b200.vumipel", "Vumipel"),
+    "Vekurax": ("scratchy_b200.vekurax", "Vekurax"),
     "LlamaForCausalLM": ("scratchy_b200.llama_serving", "LlamaServing"),
 }
 
@@ -33,6 +34,18 @@ def architecture_of(config: dict) -> str:
 def model_class(config: dict):
     module, cls = ARCHITECTURES[architecture_of(config)]
     return getattr(importlib.import_module(module), cls)
+
+
+def prepare_library(directory: str) -> None:
+    """Compiles, where needed, the kernels that the model in `directory` runs on (for programs of a source checkout)."""
+    from . import _lib
+    from .build import DESIGNS
+    name = architecture_of(read_config(directory))
+    if name in DESIGNS:
+        _lib.models_lib(build_for=name)
+    else:
+        from .build import LIB, build_library
+        build_library(LIB)
 
 
 def load_model(directory: str, device="cuda", dtype: str = "bfloat16", max_tokens: int = 8192, max_sequences: int = 8):

@@ -25,10 +25,10 @@ def add_arguments(ap: argparse.ArgumentParser) -> None:
 
 def run(args, lines=None, out=None) -> int:
     lines, out = lines if lines is not None else sys.stdin, out if out is not None else sys.stdout
-    _lib.models_lib(build=True)
     from .engine import Engine
-    from .registry import load_model
+    from .registry import load_model, prepare_library
     try:
+        prepare_library(args.model)
         model = load_model(args.model, "cuda", args.dtype, max_tokens=args.max_tokens, max_sequences=args.max_sequences)
     except _lib.ScratchyCudaError as e:
         if e.status == -4:                       # SCR_E_DTYPE

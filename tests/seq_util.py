@@ -83,6 +83,66 @@ def random_weights(cfg, seed=0):
     return out
 
 
+def side_spec(heads=4, kv_heads=2, dim=16, taps=3, bias_max=40, size=24, keep_first=5, scale=None, left_scale=0.7, rheads=3, rdim=16, rvdim=24,
+              decay=None, right_scale=1.2, ff=72, weights_of=None):
+    """A layer of window attention beside lightning attention."""
+    out = {"type": "parallel", "mixer": {
+        "left": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "conv": taps, "bias_max": bias_max, "scale": scale or dim ** -0.5,
+                 "mask": {"size": size, "keep_first": keep_first}},
+        "left_scale": left_scale,
+        "right": {"heads": rheads, "dim": rdim, "vdim": rvdim, "decay": decay or [float(np.exp(-0.7 * 2.0 ** -i)) for i in range(rheads)]},
+        "right_scale": right_scale}, "mlp": None if ff is None else {"kind": "dense", "ff": ff}}
+    return out if weights_of is None else {**out, "weights_of": weights_of}
+
+
+def side_config(layers, width=88, vocab=210, eps=2e-5):
+    return {"architecture": "Vekurax", "layers": layers, "norm": {"eps": eps}, "vocab": vocab, "width": width}
+
+
+def side_weights(cfg, seed=0, bias_rows=10):
+    """Every tensor of a Vekurax configuration, f32 values that bf16 holds exactly."""
+    rng = np.random.default_rng(seed)
+    W, out = cfg["width"], {}
+
+    def mat(name, rows, cols, gain=1.0):
+        out[name] = round_bf16(rng.standard_normal((rows, cols)) * gain / np.sqrt(cols))
+
+    def vec(name, n, mean=0.0, std=0.2):
+        out[name] = round_bf16(mean + std * rng.standard_normal(n))
+
+    def norm(name, alpha):
+        vec(name, W, 1.0)
+        vec(name + ".b", W)
+        out[name + ".alpha"] = round_bf16(np.array(alpha)).reshape(())
+    out["embed"] = round_bf16(rng.standard_normal((cfg["vocab"], W)))
+    for i, spec in enumerate(cfg["layers"]):
+        if "weights_of" in spec:
+            continue
+        norm(f"l{i}.norm1", 0.6 + 0.1 * i)
+        m, p = spec["mixer"]["left"], f"l{i}.mix.left."
+        H, G, dim = m["heads"], m["kv_heads"], m["dim"]
+        for name, n in (("q", H * dim), ("k", G * dim)):
+            mat(p + name, n, W)
+            vec(p + name + ".norm", n, 1.2)
+            out[p + name + ".conv"] = round_bf16(0.6 * rng.standard_normal((n, m["conv"])))
+            out[p + name + ".conv"][:, -1] = round_bf16(out[p + name + ".conv"][:, -1] + 0.8)
+        out[p + "rel"] = round_bf16(rng.standard_normal((bias_rows, H)))
+        mat(p + "g", H, W, 2.0)
+        mat(p + "o", W, H * dim)
+        m, p = spec["mixer"]["right"], f"l{i}.mix.right."
+        for name, n in (("q", m["heads"] * m["dim"]), ("k", m["heads"] * m["dim"]), ("v", m["heads"] * m["vdim"]), ("g", m["heads"] * m["vdim"])):
+            mat(p + name, n, W, 1.3)
+        vec(p + "norm", m["heads"] * m["vdim"], 1.0)
+        mat(p + "o", W, m["heads"] * m["vdim"])
+        if spec.get("mlp") is not None:
+            ff = spec["mlp"]["ff"]
+            mat(f"l{i}.mlp.gate", ff, W, 1.5)
+            mat(f"l{i}.mlp.up", ff, W, 1.5)
+            mat(f"l{i}.mlp.down", W, ff)
+    norm("final.norm", 0.5)
+    return out
+
+
 def save_checkpoint(directory, cfg, weights):
     from scratchy_b200.weights import write_safetensors
     os.makedirs(directory, exist_ok=True)
@@ -96,9 +156,12 @@ def make_model(cfg, weights, dtype, **kw):
     """The framework's model on the GPU from host weights."""
     import torch
     from scratchy_b200.layers import GpuWeights
+    from scratchy_b200.vekurax import Vekurax, VekuraxConfig
     from scratchy_b200.vumipel import Vumipel, VumipelConfig
-    gw = GpuWeights({k: torch.from_numpy(v).to(torch.bfloat16).cuda() for k, v in weights.items()})
+    gw = GpuWeights({k: torch.from_numpy(np.asarray(v)).to(torch.bfloat16).cuda() for k, v in weights.items()})
     kw = {"max_tokens": 1024, "max_sequences": 6, **kw}
+    if cfg["architecture"] == "Vekurax":
+        return Vekurax(VekuraxConfig.from_dict(cfg), gw, "cuda", dtype, **kw)
     return Vumipel(VumipelConfig.from_dict(cfg), gw, "cuda", dtype, **kw)
 
 

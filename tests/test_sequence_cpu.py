@@ -83,6 +83,7 @@ def test_unknown_mixer_and_architecture_are_refused():
         registry.architecture_of({"architecture": "Nobody"})
     assert registry.architecture_of({"architectures": ["LlamaForCausalLM"]}) == "LlamaForCausalLM"
     assert registry.model_class(su.config([])).__name__ == "Vumipel"
+    assert registry.model_class(su.side_config([])).__name__ == "Vekurax"
 
 
 def test_llama_configuration_from_a_checkpoint_folder():
@@ -217,7 +218,7 @@ def test_a_step_is_cut_to_the_models_portions_and_keeps_the_order_of_wants():
 def test_trace_replay_writes_wanted_rows_and_confirms_every_step(tmp_path, monkeypatch):
     m = Recorder()
     monkeypatch.setattr(registry, "load_model", lambda *a, **k: m)
-    monkeypatch.setattr(trace._lib, "models_lib", lambda build=False: None)
+    monkeypatch.setattr(registry, "prepare_library", lambda directory: None)
     steps = [{"step": 0, "entries": [{"id": "x", "tokens": [5, 17, 3], "want": [2, 0]}], "end": []},
              {"step": 1, "entries": [{"id": "x", "tokens": [9], "want": []}], "end": []},
              {"step": 7, "entries": [{"id": "x", "tokens": [4], "want": [0]}], "end": ["x"]},
@@ -239,6 +240,6 @@ def test_a_number_format_without_a_model_is_refused_with_its_own_code(tmp_path, 
     def refuse(*a, **k):
         raise ScratchyCudaError(-4, "no")
     monkeypatch.setattr(registry, "load_model", refuse)
-    monkeypatch.setattr(trace._lib, "models_lib", lambda build=False: None)
+    monkeypatch.setattr(registry, "prepare_library", lambda directory: None)
     args = types.SimpleNamespace(model="m", dtype="float32", out=str(tmp_path), max_tokens=64, max_sequences=2)
     assert trace.run(args, [], io.StringIO()) == 3
