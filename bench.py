@@ -22,6 +22,7 @@ from __future__ import annotations
 
 import argparse
 import json
+import math
 import os
 import statistics
 import subprocess
@@ -1147,8 +1148,45 @@ def vumipel_like_llama_3b():
             "width": 3072}
 
 
+def vekurax_like_llama(size):
+    """A Vekurax of Llama-3.2-3B's or 1B's width, feed-forward, vocabulary, attention heads and number of layer runs; the 3B has
+    24 layers of its own and four that run on the weights of earlier ones, as the Vumipel has."""
+    width, heads, dim, rheads, runs, own = {"3b": (3072, 24, 128, 12, 28, 24), "1b": (2048, 32, 64, 8, 16, 16)}[size]
+    layer = {"type": "parallel", "mlp": {"kind": "dense", "ff": 8192}, "mixer": {
+        "left": {"heads": heads, "kv_heads": 8, "dim": dim, "vdim": dim, "conv": 4, "bias_max": 1024, "scale": dim ** -0.5, "mask": {"size": 4096, "keep_first": 64}},
+        "left_scale": 0.8, "right": {"heads": rheads, "dim": 128, "vdim": 256, "decay": [math.exp(-2.0 ** (-8.0 * (i + 1) / rheads)) for i in range(rheads)]},
+        "right_scale": 0.8}}
+    layers = [layer if i < own else {**layer, "weights_of": i - own + 8} for i in range(runs)]
+    return {"architecture": "Vekurax", "layers": layers, "norm": {"eps": 1e-5}, "vocab": 128256, "width": width}
+
+
+def vekurax_shape(cfg, name):
+    W = cfg["width"]
+    if name == "embed":
+        return (cfg["vocab"], W)
+    if name.endswith(".alpha"):
+        return ()
+    layer, rest = name.split(".", 1)
+    if "norm" in name and ".mix." not in name:
+        return (W,)
+    spec = cfg["layers"][int(layer[1:])]
+    if rest.startswith("mlp."):
+        return (W, spec["mlp"]["ff"]) if rest == "mlp.down" else (spec["mlp"]["ff"], W)
+    _, side, part = rest.split(".", 2)
+    m = spec["mixer"][side]
+    H, dim = m["heads"], m["dim"]
+    if side == "left":
+        n = {"q": H * dim, "k": m["kv_heads"] * dim}
+        if part in n:
+            return (n[part], W)
+        if part[2:] in ("norm", "conv"):
+            return (n[part[0]],) + ((m["conv"],) if part.endswith("conv") else ())
+        return {"rel": (32, H), "g": (H, W), "o": (W, H * dim)}[part]
+    return {"q": (H * dim, W), "k": (H * dim, W), "v": (H * m["vdim"], W), "g": (H * m["vdim"], W), "o": (W, H * m["vdim"]), "norm": (H * m["vdim"],)}[part]
+
+
 class RandomCheckpoint:
-    """Tensors of a Vumipel configuration drawn on the device when they are taken."""
+    """Tensors of a sequence model's configuration drawn on the device when they are taken."""
 
     def __init__(self, cfg, device):
         import torch
@@ -1157,6 +1195,8 @@ class RandomCheckpoint:
 
     def shape(self, name):
         c, W = self.cfg, self.cfg["width"]
+        if c["architecture"] == "Vekurax":
+            return vekurax_shape(c, name)
         fixed = {"embed": (c["vocab"], W), "final.norm": (W,), "loop.in": (W, 2 * W)}
         if name in fixed:
             return fixed[name]
@@ -1181,41 +1221,58 @@ class RandomCheckpoint:
         import torch
         shape = self.shape(name)
         t = torch.randn(shape, device=self.device, generator=self.gen)
+        if self.cfg["architecture"] == "Vekurax" and len(shape) < 2:
+            return (0.5 if not shape else 0.1 * t if name.endswith(".b") else 1.0 + 0.1 * t) * torch.ones((), device=self.device, dtype=torch.bfloat16)
         return (t * (shape[1] ** -0.5 if len(shape) == 2 and name != "embed" else 0.1) + (3.0 if name.endswith("f.b") else 0.0)).to(torch.bfloat16)
 
 
-def run_sequence_model(device, steps=20, batches=(1, 8, 32), context=2048, prompts=(512, 2048, 8192)):
-    """`--sequence-model`: prefill and decode throughput of a 2.8-billion-parameter Vumipel in bf16 (random weights), beside
-    the int4 Llama-3.2-3B decode step of the same width, depth, feed-forward and vocabulary.  Every weight is distinct and
-    the step streams 7 GB, far more than L2 holds."""
+def sequence_model(raw, device, max_tokens, max_sequences):
+    from scratchy_b200.registry import model_class
+    cls = model_class(raw)
+    module = sys.modules[cls.__module__]
+    return cls(getattr(module, cls.__name__ + "Config").from_dict(raw), RandomCheckpoint(raw, device), device, "bfloat16", max_tokens=max_tokens,
+               max_sequences=max_sequences)
+
+
+def sequence_bytes(model, raw):
+    """(weight bytes of a step, cache bytes per token of context, state bytes read and written per sequence)."""
+    if raw["architecture"] == "Vekurax":
+        weights = sum(2 * (l.branches.inp.weight.numel() + l.branches.out.weight.numel()) for l in model.layers) + 2 * model.embed.numel()
+        left, right = raw["layers"][0]["mixer"]["left"], raw["layers"][0]["mixer"]["right"]
+        n = len(model.layers)
+        return weights, n * (left["kv_heads"] * left["dim"] * 2 + 4), n * right["heads"] * right["dim"] * right["vdim"] * 8
+    weights = sum(2 * w.weight.numel() for i, _ in model.runs for m in (model.layers[i].mixer, model.layers[i].mlp)
+                  for w in vars(m).values() if hasattr(w, "weight") and w is not getattr(m, "uk_rows", None))
+    weights += 2 * model.embed.numel() + 2 * model.loop_in.weight.numel() * raw["loop"]["times"]
+    att = sum(1 for i, _ in model.runs if raw["layers"][i]["type"] == "latent_attention")
+    return weights, att * 576 * 2, (len(model.runs) - att) * 12 * 128 * 256 * 4 * 2
+
+
+def _events_timed(device, call, reps, warm=3):
+    import torch
+    for _ in range(warm):
+        call()
+    torch.cuda.synchronize(device)
+    a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    a.record()
+    for _ in range(reps):
+        call()
+    b.record()
+    torch.cuda.synchronize(device)
+    return a.elapsed_time(b) * 1e-3 / reps
+
+
+def run_sequence_model(device, raw, workload, kernels, steps=20, batches=(1, 8, 32), context=2048, prompts=(512, 2048, 8192)):
+    """Prefill and decode throughput of a sequence model in bf16 (random weights).  Every weight is distinct and the step
+    streams gigabytes, far more than L2 holds."""
     import torch
     from scratchy_b200 import _lib
-    from scratchy_b200.vumipel import Vumipel, VumipelConfig
     peaks = measured_peaks()
-    raw = vumipel_like_llama_3b()
     longest = max(max(prompts), max(batches) * (context + 64))
-    model = Vumipel(VumipelConfig.from_dict(raw), RandomCheckpoint(raw, device), device, "bfloat16", max_tokens=longest, max_sequences=max(batches))
+    model = sequence_model(raw, device, longest, max(batches))
     ctx = _lib.models_context(device.index or 0)
-    run_weights = sum(2 * w.weight.numel() for i, _ in model.runs for m in (model.layers[i].mixer, model.layers[i].mlp)
-                      for w in vars(m).values() if hasattr(w, "weight") and w is not getattr(m, "uk_rows", None))
-    run_weights += 2 * model.embed.numel() + 2 * model.loop_in.weight.numel() * raw["loop"]["times"]
-    att_runs = sum(1 for i, _ in model.runs if raw["layers"][i]["type"] == "latent_attention")
-    mem_runs = len(model.runs) - att_runs
-    out = {"workload": "Vumipel, random weights, bf16: width 3072, 24 layers (28 runs), feed-forward 8192, vocabulary 128256, 3 mlstm : 1 latent attention",
-           "weight_bytes_per_step": run_weights, "prefill": [], "decode": []}
-
-    def timed(call, reps, warm=3):
-        for _ in range(warm):
-            call()
-        torch.cuda.synchronize(device)
-        a, b = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
-        a.record()
-        for _ in range(reps):
-            call()
-        b.record()
-        torch.cuda.synchronize(device)
-        return a.elapsed_time(b) * 1e-3 / reps
-
+    run_weights, cache_token, state_sequence = sequence_bytes(model, raw)
+    out = {"workload": workload, "weight_bytes_per_step": run_weights, "prefill": [], "decode": []}
     g = torch.Generator().manual_seed(0)
     flops_per_token = 2 * (run_weights / 2 - model.embed.numel())               # (the vocabulary head runs for one position)
     for n in prompts:
@@ -1225,7 +1282,7 @@ def run_sequence_model(device, steps=20, batches=(1, 8, 32), context=2048, promp
             seq = model.table.open("p")
             model.forward([(seq, tokens)], [[n - 1]])
             model.table.close("p")
-        dt = timed(prefill, 5)
+        dt = _events_timed(device, prefill, 5)
         out["prefill"].append({"tokens": n, "ms": dt * 1e3, "tok_per_s": n / dt, "TFLOPs_linears": n * flops_per_token / dt / 1e12,
                                "frac_bf16_sustained": n * flops_per_token / dt / 1e12 / peaks["bf16_tflops_sustained"]})
     for batch in batches:
@@ -1237,20 +1294,143 @@ def run_sequence_model(device, steps=20, batches=(1, 8, 32), context=2048, promp
         dg = model.decode_graph(batch, 1 << (context).bit_length())
         launches = (ctx.launch_count() - n0) // 2                               # the warm-up step and the captured one
         dg.inputs.fill([(seq, [1]) for seq in seqs], list(range(batch)))
-        dt = timed(dg.graph.replay, steps)
+        dt = _events_timed(device, dg.graph.replay, steps)
         model.check_health()
-        cache = att_runs * batch * context * 576 * 2
-        state = mem_runs * batch * 12 * 128 * 256 * 4 * 2                       # read and written
-        moved = run_weights + cache + state
+        moved = run_weights + batch * (context * cache_token + state_sequence)
         out["decode"].append({"batch": batch, "context": context, "ms_per_step": dt * 1e3, "tok_per_s": batch / dt, "launches_per_step": int(launches),
-                              "cache_bytes": cache, "state_bytes": state, "GBps": moved / dt / 1e9, "frac_hbm": moved / dt / 1e9 / peaks["hbm_gbs"]})
+                              "cache_bytes": batch * context * cache_token, "state_bytes": batch * state_sequence, "GBps": moved / dt / 1e9,
+                              "frac_hbm": moved / dt / 1e9 / peaks["hbm_gbs"]})
         for b in range(batch):
             model.table.close(("d", b))
-    out["kernels"] = run_sequence_kernels(device, model, peaks)
+    out["kernels"] = kernels(device, model, peaks)
     del model
     torch.cuda.empty_cache()
-    out["llama_3b_int4_decode"] = run_decode(device, steps=steps, batches=batches, context=context)
     return out
+
+
+def run_sequence_models(device, design, steps):
+    """`--sequence-model DESIGN`: a sequence model of 2.8 billion parameters beside the closest one of equal width, depth,
+    feed-forward and vocabulary: the int4 Llama-3.2-3B for a Vumipel, that Vumipel for a Vekurax."""
+    vumipel = lambda: run_sequence_model(device, vumipel_like_llama_3b(), "Vumipel, random weights, bf16: width 3072, 24 layers (28 runs), feed-forward 8192, "
+                                         "vocabulary 128256, 3 mlstm : 1 latent attention", run_sequence_kernels, steps)
+    if design == "vumipel":
+        out = vumipel()
+        out["llama_3b_int4_decode"] = run_decode(device, steps=steps, batches=(1, 8, 32), context=2048)
+        return out
+    out = {}
+    for size, what in (("3b", "width 3072, 24 layers (28 runs), feed-forward 8192, 24 / 8 heads of 128 over a window of 4096 + 64, 12 lightning heads 128 x 256"),
+                       ("1b", "width 2048, 16 layers, feed-forward 8192, 32 / 8 heads of 64 over a window of 4096 + 64, 8 lightning heads 128 x 256")):
+        out[f"vekurax_{size}"] = run_sequence_model(device, vekurax_like_llama(size), f"Vekurax, random weights, bf16: {what}, vocabulary 128256", run_side_kernels, steps)
+    out["vumipel_3b"] = vumipel()
+    return out
+
+
+def step_context(device, model, arena, batch, count, kv, prompt):
+    """A step of `batch` sequences with `count` new tokens each and `kv` tokens in all, over randomly placed blocks."""
+    import torch
+    from scratchy_b200.dense import StepInputs
+    from scratchy_b200.mixers import StepContext
+    T = batch * count
+    blocks = -(-kv // model.table.block_size)
+    inputs = StepInputs(device, T, batch, 1, blocks)
+
+    class S:
+        pass
+    entries = []
+    perm = torch.randperm(batch * blocks).tolist()
+    for b in range(batch):
+        s = S()
+        s.length, s.slot, s.blocks = kv - count, b, perm[b * blocks:(b + 1) * blocks]
+        entries.append((s, [0] * count))
+    inputs.fill(entries, [0])
+    return StepContext(arena, inputs, inputs.struct(model.table.max_sequences), [(s, count) for s, _ in entries], model.table.block_size, batch * blocks, T, prompt)
+
+
+def run_side_kernels(device, model, peaks, context=2048):
+    """The kernels of a Vekurax alone at its sizes, each call on its own weights, cache or state (CUDA graph)."""
+    import ctypes
+    import torch
+    from scratchy_b200 import _lib
+    from scratchy_b200.dense import Arena, dtype_code, seq_norm
+    from scratchy_b200.layers import _ptr, _stream
+    lib, c = _lib.models_lib(), _lib.models_context(device.index or 0)
+    bf, rows, arena, W = torch.bfloat16, [], Arena(device), model.width
+    code = dtype_code(bf)
+    branches = [l.branches for l in model.layers][:8]
+    left, right = branches[0].mixers
+
+    def add(kernel, us, flops=None, nbytes=None, **more):
+        row = {"kernel": kernel, **more, "us": us * 1e6}
+        if flops:
+            row.update({"TFLOPs": flops / us / 1e12, "frac_bf16_burst": flops / us / 1e12 / peaks["bf16_tflops"]})
+        if nbytes:
+            row.update({"GBps": nbytes / us / 1e9, "frac_hbm": nbytes / us / 1e9 / peaks["hbm_gbs"]})
+        rows.append(row)
+    for M in (1, 8, 32, 512, 2048):
+        sc = step_context(device, model, arena, 1, M, M, False)
+        h = torch.randn((M, W), device=device).to(bf)
+        x = torch.zeros((M, W), device=device)
+        buf = torch.randn((M, branches[0].out.in_features), device=device).to(bf)
+        outs = {**left.buffers(sc), **right.buffers(sc), "act": buf[:, branches[0].columns[-1][0]:]}
+        in_order = [outs["act" if p.endswith(".act") else p] for p in branches[0].inp.parts]
+        names = [dict(zip(b.inp.parts, in_order)) for b in branches]            # every layer's parts under its own names
+        for name, calls, lin, moved in (("dense in (all branches)", [lambda b=b, d=d: b.inp.run(arena, h, d) for b, d in zip(branches, names)], branches[0].inp,
+                                         sum(t.numel() * t.element_size() for t in outs.values())),
+                                        ("dense out + add + tanh norm", [lambda b=b: b.out.add_to(arena, buf, x, model.final_norm, h) for b in branches], branches[0].out, M * W * 10)):
+            N, K = lin.out_features, lin.in_features
+            dt = _time_calls(device, calls, 10)
+            add(name, dt, 2.0 * M * N * K if M > 32 else None, (N * K * 2 + M * K * 2 + moved) if M <= 32 else None, M=M, N=N, K=K)
+
+    def window(batch, count, kv, prompt):
+        sc = step_context(device, model, arena, batch, count, kv, prompt)
+        T, row = batch * count, left.kv_heads * left.dim
+        copies = 2 if prompt else min(24, max(2, (256 << 20) // (batch * kv * row * 2)))
+        mem = [(torch.randn((sc.num_blocks * sc.block_size, row), device=device).to(bf), torch.ones(sc.num_blocks * sc.block_size, device=device),
+                torch.zeros((batch, left.taps - 1, left.channels), dtype=bf, device=device)) for _ in range(copies)]
+        q, gate = torch.randn((T, left.out_features), device=device).to(bf), torch.randn((T, left.heads), device=device)
+        qk, o, q2 = torch.randn((T, left.channels), device=device).to(bf), torch.empty((T, left.out_features), dtype=bf, device=device), torch.empty_like(q)
+        ps, pt = ctypes.byref(left.shape(sc)), ctypes.byref(sc.step)
+        att = lambda m: c.check(lib.scr_window_attention(c.handle, code, ps, pt, _ptr(q), _ptr(m[0]), _ptr(m[1]), _ptr(left.bias), _ptr(gate), left.heads, _ptr(o),
+                                                         left.out_features, _stream(device)))
+        prep = lambda m: c.check(lib.scr_window_prepare(c.handle, code, ps, pt, _ptr(qk), left.channels, _ptr(left.conv), _ptr(left.norm), _ptr(m[2]), _ptr(q2),
+                                                        _ptr(m[0]), _ptr(m[1]), _stream(device)))
+        return sc, copies, _time_calls(device, [lambda m=m: att(m) for m in mem] * (2 if prompt else 1), 10), _time_calls(device, [lambda m=m: prep(m) for m in mem] * (2 if prompt else 1), 10)
+    row = left.kv_heads * left.dim
+    for batch in (1, 8, 32):
+        sc, copies, dt, dp = window(batch, 1, context, False)
+        add("window attention decode", dt, None, batch * context * (row * 2 + 4), batch=batch, context=context, cache_copies=copies)
+        add("convolution, norms, cache append", dp, None, batch * (2 * left.channels * 2 + 2 * (left.taps - 1) * left.channels * 2), batch=batch)
+    for T in (2048, 8192):
+        sc, copies, dt, dp = window(1, T, T, True)
+        seen = sum(min(t + 1, left.window) for t in range(T)) + sum(min(left.keep_first, max(0, t + 1 - left.window)) for t in range(T))
+        add("window attention prompt", dt, 4.0 * left.heads * left.dim * seen, None, T=T)
+        add("convolution, norms, cache append", dp, None, T * 2 * left.channels * 2, T=T)
+    for batch, count in ((1, 1), (8, 1), (32, 1), (1, 2048), (4, 2048)):
+        sc = step_context(device, model, arena, batch, count, count + 64, count > 1)
+        T, ld = batch * count, right.heads * (2 * right.dim + right.vdim)
+        proj, o = torch.randn((T, ld), device=device).to(bf), torch.empty((T, right.out_features), device=device)
+        gate, y = torch.randn((T, right.out_features), device=device).to(bf), torch.empty((T, right.out_features), dtype=bf, device=device)
+        state_bytes = batch * right.heads * right.dim * right.vdim * 8
+        copies = 2 if count > 1 else min(24, max(2, (256 << 20) // (state_bytes // 2)))
+        states = [right.memory(0, batch, device) for _ in range(copies)]
+        shape = _lib.LightningShape(right.heads, right.dim, right.vdim, right.eps, right.out_scale)
+        need = ctypes.c_size_t(0)
+        c.check(lib.scr_lightning_workspace(code, ctypes.byref(shape), ctypes.byref(sc.step), ctypes.byref(need)))
+        ws = torch.empty(max(16, need.value), dtype=torch.uint8, device=device)
+        run = lambda s: c.check(lib.scr_lightning_run(c.handle, code, ctypes.byref(shape), ctypes.byref(sc.step), _ptr(proj), ld, _ptr(right.powers), _ptr(s), _ptr(o),
+                                                      _ptr(ws), need, _stream(device)))
+        dt = _time_calls(device, [lambda s=s: run(s) for s in states], 10)
+        if count == 1:
+            add("lightning step", dt, None, state_bytes, batch=batch, state_copies=copies)
+        else:
+            L = 64                                   # the closed form of a 64-token chunk: q k, P v, q S, k v
+            add("lightning prompt", dt, 2.0 * T * right.heads * (L / 2 * (right.dim + right.vdim) + 2 * right.dim * right.vdim), T * ld * 2 + T * right.out_features * 4,
+                batch=batch, T=count)
+        fin = lambda: c.check(lib.scr_lightning_finish(c.handle, code, ctypes.byref(shape), _ptr(o), _ptr(right.norm), _ptr(gate), right.out_features, T, _ptr(y),
+                                                       right.out_features, _stream(device)))
+        add("readout norm and gate", _time_calls(device, [fin] * 4, 10), None, T * right.out_features * 8, batch=batch, T=count)
+    c.device_status(None)
+    return rows
 
 
 def run_sequence_kernels(device, model, peaks, context=2048):
@@ -1258,9 +1438,8 @@ def run_sequence_kernels(device, model, peaks, context=2048):
     import ctypes
     import torch
     from scratchy_b200 import _lib
-    from scratchy_b200.dense import Arena, DenseLinear, StepInputs, dtype_code, seq_norm
+    from scratchy_b200.dense import Arena, dtype_code, seq_norm
     from scratchy_b200.layers import _ptr, _stream
-    from scratchy_b200.mixers import StepContext
     lib, c = _lib.models_lib(), _lib.models_context(device.index or 0)
     bf, rows, arena = torch.bfloat16, [], Arena(device)
     att = [l.mixer for l in model.layers if hasattr(l.mixer, "kv_rank")]
@@ -1285,22 +1464,7 @@ def run_sequence_kernels(device, model, peaks, context=2048):
             N, K = lins[0].out_features, lins[0].in_features
             add("dense " + name, dt, 2.0 * M * N * K if M > 32 else None, (N * K * 2 + M * K * 2 + M * cols * y.element_size()) if M <= 32 else None, M=M, N=N, K=K)
 
-    def context_of(batch, count, kv, prompt):
-        T = batch * count
-        blocks = -(-kv // model.table.block_size)
-        inputs = StepInputs(device, T, batch, 1, blocks)
-
-        class S:
-            pass
-        entries = []
-        perm = torch.randperm(batch * blocks).tolist()
-        for b in range(batch):
-            s = S()
-            s.length, s.slot, s.blocks = kv - count, b, perm[b * blocks:(b + 1) * blocks]
-            entries.append((s, [0] * count))
-        inputs.fill(entries, [0])
-        return StepContext(arena, inputs, inputs.struct(model.table.max_sequences), [(s, count) for s, _ in entries], model.table.block_size, batch * blocks, T,
-                           prompt)
+    context_of = lambda *a: step_context(device, model, arena, *a)
     m = att[0]
     for batch in (1, 8, 32):
         sc = context_of(batch, 1, context, False)
@@ -1376,9 +1540,9 @@ def main():
     ap.add_argument("--tp-separate-exchange", action="store_true",
                     help="tensor-parallel section: row-parallel matvec and all-reduce as two launches instead of "
                          "scr_linear_fp8_dynamic_allreduce (measured: equal at TP=2, 9 %% slower at TP=8)")
-    ap.add_argument("--sequence-model", action="store_true",
-                    help="prefill and decode throughput of a hybrid sequence model (Vumipel, bf16, random weights) beside the int4 Llama of "
-                         "equal size, and its kernels alone; prints one JSON line of its own")
+    ap.add_argument("--sequence-model", nargs="?", const="vumipel", choices=["vumipel", "vekurax"],
+                    help="prefill and decode throughput of a sequence model (bf16, random weights) and its kernels alone, beside the closest other model "
+                         "of equal size (int4 Llama for vumipel, the default; vumipel for vekurax); prints one JSON line of its own")
     ap.add_argument("--case", default=None, help="kind,shape,M e.g. int4,gate,2048: time one linear alone")
     args = ap.parse_args()
     if args.case:
@@ -1397,7 +1561,7 @@ def main():
         device = torch.device("cuda", 0)
         torch.cuda.set_device(device)
         sampler = ClockSampler(0)
-        res = run_sequence_model(device, steps=min(args.steps, 50))
+        res = run_sequence_models(device, args.sequence_model, min(args.steps, 50))
         print(json.dumps({"sequence_model": res, "clocks": sampler.stop()}))
         return
     if args.impl == "reference":

@@ -173,9 +173,10 @@ int32_t scr_mlstm_finish(scr_ctx* ctx, int32_t dtype, const scr_mlstm_shape* s, 
 /* ---- sliding-window attention whose values are its keys before their norm --------------------------
  * Grouped heads (query head h reads key/value head h / (heads / kv_heads)).  Queries and keys pass a causal convolution of
  * `taps` taps per channel and an RMS norm over the whole projection; the values are the convolved keys themselves.  The cache
- * therefore holds the values only, [num_blocks * block_size, kv_heads * dim] of dtype, and one f32 per token, the reciprocal
- * root mean square of its keys (key_inv); the key norm's weight is folded into the queries.
- * Position i sees j <= i with i - j < window or j < keep_first.  Score: q.k * scale + bias[h][min(i - j, n_bias - 1)]. */
+ * therefore holds the values only, [num_blocks * block_size, kv_heads * dim] of dtype, and one f32 per token, key_scale =
+ * scale * log2(e) / (root mean square of its keys); the key norm's weight is folded into the queries.
+ * Position i sees j <= i with i - j < window or j < keep_first.  Score in powers of two: q.v * key_scale +
+ * bias[h][min(i - j, n_bias - 1)], the bias of the softmax times log2(e). */
 typedef struct scr_window_shape {
     int32_t heads, kv_heads, dim, taps;
     int32_t window, keep_first, n_bias;
@@ -185,14 +186,14 @@ typedef struct scr_window_shape {
 /* proj (dtype, row stride ld): q [heads * dim] | k [kv_heads * dim] as projected; conv [taps, (heads + kv_heads) * dim] and
  * norm [(heads + kv_heads) * dim] f32.  conv_state (dtype) [num_slots, taps - 1, (heads + kv_heads) * dim] holds the last
  * projected rows of every sequence, oldest first; zeros precede position 0 whatever the slot holds.  Writes the queries
- * (dtype [rows, heads * dim], normed, times the key norm's weight), the cache rows, key_inv and conv_state. */
+ * (dtype [rows, heads * dim], normed, times the key norm's weight), the cache rows, key_scale and conv_state. */
 int32_t scr_window_prepare(scr_ctx* ctx, int32_t dtype, const scr_window_shape* s, const scr_step* st, const void* proj, int64_t ld,
-                           const float* conv, const float* norm, void* conv_state, void* q, void* cache, float* key_inv,
+                           const float* conv, const float* norm, void* conv_state, void* q, void* cache, float* key_scale,
                            void* stream);
 /* out (dtype, row stride ld_out) [rows, heads * dim] = softmax(scores) v * sigmoid(gate[t * ld_gate + h]) * out_scale.
  * Blocks that no visible key lies in may be missing from the block table (any negative number). */
 int32_t scr_window_attention(scr_ctx* ctx, int32_t dtype, const scr_window_shape* s, const scr_step* st, const void* q, const void* cache,
-                             const float* key_inv, const float* bias, const float* gate, int64_t ld_gate, void* out, int64_t ld_out,
+                             const float* key_scale, const float* bias, const float* gate, int64_t ld_gate, void* out, int64_t ld_out,
                              void* stream);
 
 /* ---- matrix memory with a constant decay per head (lightning attention) -----------------------------

@@ -77,7 +77,7 @@ __device__ __forceinline__ void dg_residual32(const DenseEnds& e, int m, int n0,
     } else {
 #pragma unroll
         for (int j = 0; j < 32; ++j)
-            if (n0 + j < N) dense_put<bf16>(e, m, 0, n0 + j, v[j]);
+            if (n0 + j < N) dense_put_residual<bf16>(e, m, n0 + j, v[j]);
     }
 }
 
@@ -86,28 +86,42 @@ __device__ __forceinline__ void dg_parts32(const DenseEnds& e, int m, int n0, in
     int start;
     const int pi = dense_part(e, n0, start);
     const scr_dense_part p = e.parts[pi];
-    if (n0 + 32 <= p.n_end) {
-        const bool glu = p.kind == SCR_PART_GELU_GLU;
-        const int cols = glu ? 16 : 32, size = p.kind == SCR_PART_F32 ? 4 : 2;
+    const bool glu = p.kind == SCR_PART_GELU_GLU;
+    if (min(n0 + 32, N) <= p.n_end && (!glu || ((n0 - start) & 15) == 0)) {
+        const int size = p.kind == SCR_PART_F32 ? 4 : 2, cols = min(32, N - n0) >> (glu ? 1 : 0);        // columns that come out
         char* dst = reinterpret_cast<char*>(p.y) + (m * p.ld + (glu ? (n0 - start) >> 1 : n0 - start)) * size;
-        if ((reinterpret_cast<uintptr_t>(dst) & 15) == 0 && (!glu || ((n0 - start) & 15) == 0)) {
-            if (p.kind == SCR_PART_F32) {
+        const bool vec = (reinterpret_cast<uintptr_t>(dst) & 15) == 0;
+        if (p.kind == SCR_PART_F32) {
 #pragma unroll
-                for (int j = 0; j < 32; j += 4) reinterpret_cast<float4*>(dst)[j >> 2] = make_float4(v[j], v[j + 1], v[j + 2], v[j + 3]);
-                return;
+            for (int j = 0; j < 32; j += 4) {
+                if (vec && j + 4 <= cols) {
+                    reinterpret_cast<float4*>(dst)[j >> 2] = make_float4(v[j], v[j + 1], v[j + 2], v[j + 3]);
+                } else {
+#pragma unroll
+                    for (int i = 0; i < 4; ++i)
+                        if (j + i < cols) reinterpret_cast<float*>(dst)[j + i] = v[j + i];
+                }
             }
-            if (glu) {
-#pragma unroll
-                for (int j = 0; j < 16; ++j) v[j] = gelu_glu(v[(j >> 3) * 16 + (j & 7)], v[(j >> 3) * 16 + 8 + (j & 7)]);
-            } else if (p.kind == SCR_PART_SILU) {
-#pragma unroll
-                for (int j = 0; j < 32; ++j) v[j] *= sigmoid_f32(v[j]);
-            }
-#pragma unroll
-            for (int j = 0; j < 32; j += 8)
-                if (j < cols) reinterpret_cast<uint4*>(dst)[j >> 3] = dg_pack8(v + j);
             return;
         }
+        if (glu) {
+#pragma unroll
+            for (int j = 0; j < 16; ++j) v[j] = gelu_glu(v[(j >> 3) * 16 + (j & 7)], v[(j >> 3) * 16 + 8 + (j & 7)]);
+        } else if (p.kind == SCR_PART_SILU) {
+#pragma unroll
+            for (int j = 0; j < 32; ++j) v[j] *= sigmoid_f32(v[j]);
+        }
+#pragma unroll
+        for (int j = 0; j < 32; j += 8) {
+            if (vec && j + 8 <= cols) {
+                reinterpret_cast<uint4*>(dst)[j >> 3] = dg_pack8(v + j);
+            } else {
+#pragma unroll
+                for (int i = 0; i < 8; ++i)
+                    if (j + i < cols) reinterpret_cast<bf16*>(dst)[j + i] = __float2bfloat16_rn(v[j + i]);
+            }
+        }
+        return;
     }
 #pragma unroll
     for (int j = 0; j < 16; ++j) {
@@ -157,7 +171,7 @@ __device__ __forceinline__ void dg_store32(const DenseEnds& e, int m, int g, int
     } else {
 #pragma unroll
         for (int j = 0; j < 32; ++j)
-            if (n0 + j < N) dense_put<bf16>(e, m, g, n0 + j, v[j]);
+            if (n0 + j < N) dense_put_own<bf16>(e, m, g, n0 + j, v[j]);
     }
 }
 
@@ -302,7 +316,12 @@ __global__ void __launch_bounds__(256) dense_gemm_finish_kernel(const float* __r
         a += src[(size_t)k * n_tail * tile_elems];
         b += src[(size_t)k * n_tail * tile_elems + 8];
     }
-    dense_put_two<bf16>(ends, m, g, n, N, a, b);
+    if (ends.residual) {
+        dense_put_residual<bf16>(ends, m, n, a);
+        if (n + 8 < N) dense_put_residual<bf16>(ends, m, n + 8, b);
+    } else {
+        dense_put_two<bf16>(ends, m, g, n, N, a, b);
+    }
 }
 
 bool dg_map(CUtensorMap* map, const void* base, uint64_t d0, uint64_t d1, uint64_t d2, uint64_t s1, uint64_t s2, uint32_t b1, uint32_t b2) {

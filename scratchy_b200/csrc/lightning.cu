@@ -110,20 +110,68 @@ __global__ void __launch_bounds__(LR_T) lightning_recur_kernel(MemoryArgs a) {
     }
 }
 
-constexpr int LN_T = 256;
-template <typename T>
+constexpr int LN_T = 512;
+__device__ __forceinline__ void ln_gate(const bf16* p, float (&g)[4]) {
+    const uint2 w = *reinterpret_cast<const uint2*>(p);
+    g[0] = bf16_lo(w.x); g[1] = bf16_hi(w.x); g[2] = bf16_lo(w.y); g[3] = bf16_hi(w.y);
+}
+__device__ __forceinline__ void ln_gate(const float* p, float (&g)[4]) {
+    const float4 w = *reinterpret_cast<const float4*>(p);
+    g[0] = w.x; g[1] = w.y; g[2] = w.z; g[3] = w.w;
+}
+__device__ __forceinline__ void ln_put(bf16* p, const float (&v)[4]) { *reinterpret_cast<uint2*>(p) = make_uint2(pack_bf16x2(v[0], v[1]), pack_bf16x2(v[2], v[3])); }
+__device__ __forceinline__ void ln_put(float* p, const float (&v)[4]) { *reinterpret_cast<float4*>(p) = make_float4(v[0], v[1], v[2], v[3]); }
+
+// One CTA per row.  KEEP: runs of 4 values a thread holds in registers between the sum and the product (0: any sizes).
+template <typename T, int KEEP>
 __global__ void __launch_bounds__(LN_T) lightning_finish_kernel(scr_lightning_shape s, const float* __restrict__ out, const float* __restrict__ norm,
                                                                 const T* __restrict__ gate, long long ld_gate, T* __restrict__ y, long long ld_y) {
     __shared__ float red[LN_T / 32];
     pdl_trigger();
     pdl_wait();
-    const int n = s.heads * s.vdim;
+    const int n = s.heads * s.vdim, tid = threadIdx.x;
     const size_t r = blockIdx.x;
     const float* o = out + r * n;
     float ss = 0.0f;
-    for (int i = threadIdx.x; i < n; i += LN_T) ss = fmaf(o[i], o[i], ss);
-    const float inv = s.out_scale / sqrtf(cta_sum<LN_T>(ss, red) / float(n) + s.eps);
-    for (int i = threadIdx.x; i < n; i += LN_T) y[r * ld_y + i] = from_f32<T>(o[i] * inv * norm[i] * sigmoid_f32(to_f32(gate[r * ld_gate + i])));
+    if constexpr (KEEP > 0) {
+        constexpr int K = KEEP;
+        float v[K][4], w[K][4], g[K][4];
+#pragma unroll
+        for (int k = 0; k < K; ++k) {
+            const int i = (k * LN_T + tid) * 4;
+            if (i >= n) continue;
+            ln_gate(o + i, v[k]);
+            ln_gate(norm + i, w[k]);
+            ln_gate(gate + r * ld_gate + i, g[k]);
+#pragma unroll
+            for (int j = 0; j < 4; ++j) ss = fmaf(v[k][j], v[k][j], ss);
+        }
+        const float inv = s.out_scale / sqrtf(cta_sum<LN_T>(ss, red) / float(n) + s.eps);
+#pragma unroll
+        for (int k = 0; k < K; ++k) {
+            const int i = (k * LN_T + tid) * 4;
+            if (i >= n) continue;
+#pragma unroll
+            for (int j = 0; j < 4; ++j) v[k][j] = v[k][j] * inv * w[k][j] * sigmoid_f32(g[k][j]);
+            ln_put(y + r * ld_y + i, v[k]);
+        }
+    } else {
+        for (int i = tid; i < n; i += LN_T) ss = fmaf(o[i], o[i], ss);
+        const float inv = s.out_scale / sqrtf(cta_sum<LN_T>(ss, red) / float(n) + s.eps);
+        for (int i = tid; i < n; i += LN_T) y[r * ld_y + i] = from_f32<T>(o[i] * inv * norm[i] * sigmoid_f32(to_f32(gate[r * ld_gate + i])));
+    }
+}
+
+template <typename T>
+int32_t finish(scr_ctx* ctx, const scr_lightning_shape& s, const float* out, const float* norm, const void* gate, int64_t ld_gate, int32_t rows, void* y,
+               int64_t ld_y, cudaStream_t stream) {
+    const int n = s.heads * s.vdim;
+    const bool vec = n % 4 == 0 && ld_gate % 4 == 0 && ld_y % 4 == 0 && scr_aligned16(out) && scr_aligned16(norm) && scr_aligned16(gate) && scr_aligned16(y);
+    auto kernel = !vec || n > 16 * LN_T ? lightning_finish_kernel<T, 0> : n > 8 * LN_T ? lightning_finish_kernel<T, 4>
+                : n > 4 * LN_T ? lightning_finish_kernel<T, 2> : lightning_finish_kernel<T, 1>;
+    const cudaError_t e = launch_pdl(kernel, dim3(rows), dim3(LN_T), 0, stream, s, out, norm, (const T*)gate, (long long)ld_gate, (T*)y, (long long)ld_y);
+    if (e != cudaSuccess) return scr_fail(ctx, SCR_E_CUDA, "lightning_finish: %s", cudaGetErrorString(e));
+    return scr_check_launch(ctx, "lightning_finish");
 }
 
 template <typename T, int RPT>
@@ -170,10 +218,6 @@ extern "C" int32_t scr_lightning_finish(scr_ctx* ctx, int32_t dtype, const scr_l
     if (!s || !out || !norm || !gate || !y) return scr_fail(ctx, SCR_E_ARG, "null pointer");
     if (rows <= 0 || s->heads <= 0 || s->vdim <= 0) return scr_fail(ctx, SCR_E_SHAPE, "%d rows", rows);
     if (dtype != SCR_DTYPE_F32 && dtype != SCR_DTYPE_BF16) return scr_fail(ctx, SCR_E_DTYPE, "dtype %d", dtype);
-    cudaStream_t cs = (cudaStream_t)stream;
-    const cudaError_t e = dtype == SCR_DTYPE_F32
-        ? launch_pdl(lightning_finish_kernel<float>, dim3(rows), dim3(LN_T), 0, cs, *s, out, norm, (const float*)gate, (long long)ld_gate, (float*)y, (long long)ld_y)
-        : launch_pdl(lightning_finish_kernel<bf16>, dim3(rows), dim3(LN_T), 0, cs, *s, out, norm, (const bf16*)gate, (long long)ld_gate, (bf16*)y, (long long)ld_y);
-    if (e != cudaSuccess) return scr_fail(ctx, SCR_E_CUDA, "lightning_finish: %s", cudaGetErrorString(e));
-    return scr_check_launch(ctx, "lightning_finish");
+    return dtype == SCR_DTYPE_F32 ? finish<float>(ctx, *s, out, norm, gate, ld_gate, rows, y, ld_y, (cudaStream_t)stream)
+                                  : finish<bf16>(ctx, *s, out, norm, gate, ld_gate, rows, y, ld_y, (cudaStream_t)stream);
 }

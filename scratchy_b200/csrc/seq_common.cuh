@@ -148,23 +148,9 @@ __device__ __forceinline__ int dense_part(const DenseEnds& e, int n, int& start)
         }
     return p;
 }
+// One sum without a residual and parts
 template <typename T>
-__device__ __forceinline__ void dense_put(const DenseEnds& e, int m, int g, int n, float v) {
-    if (e.residual) {
-        float* r = e.residual + m * e.ld_residual + n;
-        v += *r;
-        *r = v;
-        if (e.tanh_w) reinterpret_cast<T*>(e.y)[m * e.ldy + n] = from_f32<T>(fmaf(tanhf(e.tanh_alpha * v), e.tanh_w[n], e.tanh_b[n]));
-        return;
-    }
-    if (e.n_parts) {
-        int start;
-        const scr_dense_part& p = e.parts[dense_part(e, n, start)];
-        const long long at = m * p.ld + n - start;
-        if (p.kind == SCR_PART_F32) reinterpret_cast<float*>(p.y)[at] = v;
-        else reinterpret_cast<T*>(p.y)[at] = from_f32<T>(p.kind == SCR_PART_SILU ? v * sigmoid_f32(v) : v);
-        return;
-    }
+__device__ __forceinline__ void dense_put_own(const DenseEnds& e, int m, int g, int n, float v) {
     if (n >= e.n_main) {
         e.y2[m * e.ldy2 + (n - e.n_main)] = v;
         return;
@@ -173,6 +159,26 @@ __device__ __forceinline__ void dense_put(const DenseEnds& e, int m, int g, int 
     if (e.gate) v *= sigmoid_f32(to_f32(reinterpret_cast<const T*>(e.gate)[m * e.ldg + col]));
     if (e.y_f32) reinterpret_cast<float*>(e.y)[m * e.ldy + col] = v;
     else reinterpret_cast<T*>(e.y)[m * e.ldy + col] = from_f32<T>(v);
+}
+template <typename T>
+__device__ __forceinline__ void dense_put_residual(const DenseEnds& e, int m, int n, float v) {
+    float* r = e.residual + m * e.ld_residual + n;
+    v += *r;
+    *r = v;
+    if (e.tanh_w) reinterpret_cast<T*>(e.y)[m * e.ldy + n] = from_f32<T>(fmaf(tanhf(e.tanh_alpha * v), e.tanh_w[n], e.tanh_b[n]));
+}
+template <typename T>
+__device__ __forceinline__ void dense_put(const DenseEnds& e, int m, int g, int n, float v) {
+    if (e.residual) return dense_put_residual<T>(e, m, n, v);
+    if (e.n_parts) {
+        int start;
+        const scr_dense_part& p = e.parts[dense_part(e, n, start)];
+        const long long at = m * p.ld + n - start;
+        if (p.kind == SCR_PART_F32) reinterpret_cast<float*>(p.y)[at] = v;
+        else reinterpret_cast<T*>(p.y)[at] = from_f32<T>(p.kind == SCR_PART_SILU ? v * sigmoid_f32(v) : v);
+        return;
+    }
+    dense_put_own<T>(e, m, g, n, v);
 }
 // Columns n (n % 16 < 8) and n + 8 of N.  Where they are a gate and its up they become channel (n / 16) * 8 + n % 8.
 template <typename T>

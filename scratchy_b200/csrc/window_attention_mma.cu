@@ -1,7 +1,7 @@
 // Sliding-window attention for decoding and short portions, bf16, on mma.sync.  The rows that share a key/value head (the
 // tokens of a portion times the heads of a group) are the 16 rows of a tile; every warp walks key tiles of its own, 32 cache
 // rows at a time, through a ring of its own (cp.async), with no barrier between the warps:
-//   S = Q K^T with Q in registers; scale times the keys' reciprocal root mean square, bias, window; online softmax in f32 on
+//   S = Q K^T with Q in registers; the keys' scale, bias, window; online softmax in f32 on
 //   the accumulators; P as a bf16 head and remainder (two products: the weights keep about 16 bits); O += P V from the very
 //   same shared-memory rows, read transposed.
 // The warps' states meet in shared memory; the key shares of a cluster's CTAs meet through distributed shared memory.
@@ -39,7 +39,7 @@ struct WmArgs {
     scr_step st;
     const bf16* q;
     const bf16* cache;
-    const float* key_inv;
+    const float* key_scale;
     const float* bias;
     const float* gate;
     long long ld_gate;
@@ -94,7 +94,7 @@ __global__ void __launch_bounds__(WM_THREADS) window_attention_mma_kernel(const 
                 const int key = c / (NK * 2), x = c % (NK * 2);
                 if (x < chunks) cp_async16(dst + (key * LD + x * 8) * 2, src + key * row_size + x * 8, true);
             }
-            if (lane < WM_KEYS / 4) cp_async16(dst + SM::kTile + lane * 16, a.key_inv + row + lane * 4, true);
+            if (lane < WM_KEYS / 4) cp_async16(dst + SM::kTile + lane * 16, a.key_scale + row + lane * 4, true);
         }
         cp_async_commit();
     };
@@ -134,7 +134,6 @@ __global__ void __launch_bounds__(WM_THREADS) window_attention_mma_kernel(const 
     if (QREG)
 #pragma unroll
         for (int ks = 0; ks < (QREG ? NK : 0); ++ks) load_q(ks, qf[ks]);
-    const float log2e = 1.4426950408889634f, sl2 = s.scale * log2e;
     float acc[NO][4] = {}, m[2] = {-1e30f, -1e30f}, l[2] = {0.0f, 0.0f};
     for (int n = 0; i0 + n * stride < tiles.count; ++n) {
         asm volatile("cp.async.wait_group %0;" ::"n"(STAGES - 2) : "memory");
@@ -174,7 +173,7 @@ __global__ void __launch_bounds__(WM_THREADS) window_attention_mma_kernel(const 
             for (int e = 0; e < 4; ++e) {
                 const int hf = e >> 1, key = key0 + k + (e & 1), d = pos[hf] - key;
                 const float bv = beyond ? far[hf] : bias[hf][min(max(d, 0), s.n_bias - 1)];
-                float v = fmaf(sc[x][e] * (e & 1 ? iv.y : iv.x), sl2, bv * log2e);
+                float v = fmaf(sc[x][e], e & 1 ? iv.y : iv.x, bv);
                 if (!plain && !window_sees(s, pos[hf], key)) v = -INFINITY;
                 sc[x][e] = v;
                 mx[hf] = fmaxf(mx[hf], v);
@@ -321,9 +320,9 @@ cudaError_t wm_launch(const WmArgs& a, int tiles, cudaStream_t stream) {
 
 bool window_mma_applies(const scr_window_shape& s) { return s.dim % 8 == 0 && s.dim <= 256 && s.block_size % WM_KEYS == 0; }
 
-int32_t window_mma_launch(scr_ctx* ctx, const scr_window_shape& s, const scr_step& st, const void* q, const void* cache, const float* key_inv,
+int32_t window_mma_launch(scr_ctx* ctx, const scr_window_shape& s, const scr_step& st, const void* q, const void* cache, const float* key_scale,
                           const float* bias, const float* gate, int64_t ld_gate, void* out, int64_t ld_out, cudaStream_t stream) {
-    WmArgs a{s, st, (const bf16*)q, (const bf16*)cache, key_inv, bias, gate, ld_gate, (bf16*)out, ld_out, 1, ctx->dev_status};
+    WmArgs a{s, st, (const bf16*)q, (const bf16*)cache, key_scale, bias, gate, ld_gate, (bf16*)out, ld_out, 1, ctx->dev_status};
     if (st.max_kv <= 0 || st.batch > 65535) return scr_fail(ctx, SCR_E_SHAPE, "max_kv %d batch %d", st.max_kv, st.batch);
     const int tiles = scr_ceil_div(st.max_count * (s.heads / s.kv_heads), 16);
     // key shares: two CTAs per SM, at least two key tiles per warp

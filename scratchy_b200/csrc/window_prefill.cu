@@ -5,9 +5,9 @@
 // A CTA takes one head and 256 query rows of one sequence as two tiles of 128 that run in turn: while the tensor core works
 // on one tile, the softmax warps of the other work.  It walks the key tiles that any of its rows sees, those of the kept
 // first tokens and those of the window; a query tile skips the ones none of its rows sees.  320 threads:
-//   warp 0       TMA: the query tiles once, then key tiles with their reciprocal root mean squares through a ring
+//   warp 0       TMA: the query tiles once, then key tiles with their scales through a ring
 //   warp 1       owns TMEM; one thread issues, per key tile and query tile, O += P V of the tile before and S = Q K^T
-//   warps 2-5, 6-9   softmax of tile 0, tile 1 (thread = query row): S from TMEM, scale, bias and window in f32, P back to
+//   warps 2-5, 6-9   softmax of tile 0, tile 1 (thread = query row): S from TMEM, scales, bias and window in f32, P back to
 //                TMEM as a bf16 head and remainder (two products: the weights keep about 16 bits), O rescaled in TMEM
 //                only when the row maximum has grown by more than 2^8 over the reference the sums are kept in
 // TMEM per tile: S 64 columns, P 32 + 32, O 128.  Every wait is bounded (tc_common.cuh).
@@ -17,7 +17,10 @@
 
 namespace {
 
-constexpr int WF_THREADS = 320, WF_KEYS = 64, WF_MAX_STAGES = 6, WF_BIAS = 2048;      // bias entries kept in shared memory
+constexpr int WF_THREADS = 320, WF_KEYS = 64, WF_MAX_STAGES = 6, WF_BIAS = 4096;      // bias entries kept in shared memory
+// beside them, so that no index needs a limit: distances that are not there yet (masked), and those of the last tile whose
+// distances differ
+constexpr int WF_BIAS_LO = 192, WF_BIAS_HI = 96;
 constexpr uint32_t WF_Q_CHUNK = 128 * 128, WF_K_CHUNK = WF_KEYS * 128;                // 64 dimensions of 128 query rows / 64 keys
 
 struct WfLayout {
@@ -28,7 +31,7 @@ struct WfLayout {
         WfLayout l{};
         l.chunks = (s.dim + 63) / 64;
         l.vp = (s.dim + 15) / 16 * 16;
-        l.bias_n = s.n_bias <= WF_BIAS ? s.n_bias : 0;
+        l.bias_n = s.n_bias <= WF_BIAS ? WF_BIAS_LO + s.n_bias + WF_BIAS_HI : 0;
         const uint32_t q = 2 * l.chunks * WF_Q_CHUNK, fixed = q + l.bias_n * 4 + 16 + 256 + 1024;
         l.stages = (int)std::min<uint32_t>(WF_MAX_STAGES, (226 * 1024 - fixed) / (l.k_bytes() + WF_KEYS * 4));
         l.k = q;
@@ -44,7 +47,7 @@ struct WfArgs {
     WfLayout lay;
     scr_window_shape s;
     scr_step st;
-    const float* key_inv;
+    const float* key_scale;
     const float* bias;
     const float* gate;
     long long ld_gate;
@@ -69,7 +72,7 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_co
     auto o_full = [&](int t) { return bars + 8u * (5 + 2 * WF_MAX_STAGES + t); };
     volatile uint32_t* tmem_slot = reinterpret_cast<volatile uint32_t*>(gen + L.bars + 8 * (7 + 2 * WF_MAX_STAGES));
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-    const int head = blockIdx.x, q0 = blockIdx.y * 256, b = blockIdx.z;
+    const int head = blockIdx.x, q0 = ((int)gridDim.y - 1 - (int)blockIdx.y) * 256, b = blockIdx.z;      // the longest first
     const int first = a.st.segs[b * 4], count = a.st.segs[b * 4 + 1], pos0 = a.st.segs[b * 4 + 2];
 
     pdl_trigger();
@@ -111,8 +114,8 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_co
     const float* bias = a.bias + (size_t)head * s.n_bias;
     if (L.bias_n) {                                          // (a constant of the model: no wait)
         float* dst = reinterpret_cast<float*>(gen + L.bias);
-        for (int i = threadIdx.x; i < L.bias_n; i += WF_THREADS) dst[i] = bias[i];
-        bias = dst;
+        for (int i = threadIdx.x; i < L.bias_n; i += WF_THREADS) dst[i] = bias[min(max(i - WF_BIAS_LO, 0), s.n_bias - 1)];
+        bias = dst + WF_BIAS_LO;
     }
     tc_fence_before();
     __syncthreads();
@@ -143,7 +146,7 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_co
                 mbar_wait(k_empty(ks), kp ^ 1u, a.status, TC_ERR_EMPTY_WAIT);
                 mbar_arrive_expect_tx(k_full(ks), L.k_bytes() + WF_KEYS * 4);
                 for (int c = 0; c < L.chunks; ++c) tma_load_3d(base + L.k + ks * L.k_bytes() + c * WF_K_CHUNK, &k_map, c * 64, g, block * WF_KEYS, k_full(ks));
-                bulk_g2s(base + L.inv + ks * WF_KEYS * 4, a.key_inv + (size_t)block * WF_KEYS, WF_KEYS * 4, k_full(ks));
+                bulk_g2s(base + L.inv + ks * WF_KEYS * 4, a.key_scale + (size_t)block * WF_KEYS, WF_KEYS * 4, k_full(ks));
                 if (++ks == L.stages) { ks = 0; kp ^= 1u; }
             }
         }
@@ -187,14 +190,14 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_co
         const int t = warp >= 6, q = warp & 3;
         const uint32_t lanes = (uint32_t)(q * 32) << 16;
         const int row = q0 + t * 128 + q * 32 + lane, pos = pos0 + row, w_lo = pos - lane, w_hi = w_lo + 31;     // the warp's positions
-        const float log2e = 1.4426950408889634f, sl2 = s.scale * log2e, far = bias[s.n_bias - 1] * log2e;
+        const float far = bias[s.n_bias - 1];
         float m_ref = -1e30f, l = 0.0f;
         int seen = 0, ks = 0;
         uint32_t kp = 0;
         for (int j = 0; j < tiles.count; ++j) {
             if (active(t, j)) {
                 const int key0 = tiles.tile(j) * WF_KEYS;
-                mbar_wait(k_full(ks), kp, a.status, TC_ERR_FULL_WAIT);               // (long complete: the reciprocals are read here too)
+                mbar_wait(k_full(ks), kp, a.status, TC_ERR_FULL_WAIT);               // (long complete: the scales are read here too)
                 mbar_wait(s_full(t), (uint32_t)seen & 1u, a.status, TC_ERR_ACC_FULL);
                 tc_fence_after();
                 float v[64];
@@ -214,20 +217,30 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_co
 #pragma unroll
                     for (int i = 0; i < 64; i += 4) {
                         const float4 iv = inv[i >> 2];
-                        v[i] = fmaf(v[i] * iv.x, sl2, far);
-                        v[i + 1] = fmaf(v[i + 1] * iv.y, sl2, far);
-                        v[i + 2] = fmaf(v[i + 2] * iv.z, sl2, far);
-                        v[i + 3] = fmaf(v[i + 3] * iv.w, sl2, far);
+                        v[i] = fmaf(v[i], iv.x, far);
+                        v[i + 1] = fmaf(v[i + 1], iv.y, far);
+                        v[i + 2] = fmaf(v[i + 2], iv.z, far);
+                        v[i + 3] = fmaf(v[i + 3], iv.w, far);
+                    }
+                } else if (L.bias_n) {
+                    const float* bt = bias + (pos - key0);
+#pragma unroll
+                    for (int i = 0; i < 64; i += 4) {
+                        const float4 iv = inv[i >> 2];
+                        v[i] = fmaf(v[i], iv.x, bt[-i]);
+                        v[i + 1] = fmaf(v[i + 1], iv.y, bt[-i - 1]);
+                        v[i + 2] = fmaf(v[i + 2], iv.z, bt[-i - 2]);
+                        v[i + 3] = fmaf(v[i + 3], iv.w, bt[-i - 3]);
                     }
                 } else {
                     const int d0 = pos - key0, top = s.n_bias - 1;
 #pragma unroll
                     for (int i = 0; i < 64; i += 4) {
                         const float4 iv = inv[i >> 2];
-                        v[i] = fmaf(v[i] * iv.x, sl2, bias[min(max(d0 - i, 0), top)] * log2e);
-                        v[i + 1] = fmaf(v[i + 1] * iv.y, sl2, bias[min(max(d0 - i - 1, 0), top)] * log2e);
-                        v[i + 2] = fmaf(v[i + 2] * iv.z, sl2, bias[min(max(d0 - i - 2, 0), top)] * log2e);
-                        v[i + 3] = fmaf(v[i + 3] * iv.w, sl2, bias[min(max(d0 - i - 3, 0), top)] * log2e);
+                        v[i] = fmaf(v[i], iv.x, bias[min(max(d0 - i, 0), top)]);
+                        v[i + 1] = fmaf(v[i + 1], iv.y, bias[min(max(d0 - i - 1, 0), top)]);
+                        v[i + 2] = fmaf(v[i + 2], iv.z, bias[min(max(d0 - i - 2, 0), top)]);
+                        v[i + 3] = fmaf(v[i + 3], iv.w, bias[min(max(d0 - i - 3, 0), top)]);
                     }
                 }
                 if (key0 + WF_KEYS - 1 > w_lo || !(w_hi - key0 < s.window || key0 + WF_KEYS <= s.keep_first)) {
@@ -324,9 +337,9 @@ bool window_prefill_applies(const scr_window_shape& s, const scr_step& st) {
     return st.max_count >= WF_MIN_ROWS && s.block_size == WF_KEYS && s.dim % 8 == 0 && s.dim <= 128 && st.batch <= 65535 && WfLayout::of(s).stages >= 3;
 }
 
-int32_t window_prefill_launch(scr_ctx* ctx, const scr_window_shape& s, const scr_step& st, const void* q, const void* cache, const float* key_inv,
+int32_t window_prefill_launch(scr_ctx* ctx, const scr_window_shape& s, const scr_step& st, const void* q, const void* cache, const float* key_scale,
                               const float* bias, const float* gate, int64_t ld_gate, void* out, int64_t ld_out, cudaStream_t stream) {
-    const WfArgs a{WfLayout::of(s), s, st, key_inv, bias, gate, ld_gate, (bf16*)out, ld_out, ctx->dev_status};
+    const WfArgs a{WfLayout::of(s), s, st, key_scale, bias, gate, ld_gate, (bf16*)out, ld_out, ctx->dev_status};
     CUtensorMap qm, km;
     if (!wf_map(&qm, q, s.dim, s.heads, st.rows, 128) || !wf_map(&km, cache, s.dim, s.kv_heads, (uint64_t)s.num_blocks * s.block_size, WF_KEYS))
         return scr_fail(ctx, SCR_E_CUDA, "window_prefill: tensor map");

@@ -225,7 +225,7 @@ class WindowAttention:
     convolution and an RMS norm over the whole projection, the values are the keys before that norm, a bias per head and
     distance bucket joins the scores, one sigmoid per head gates the output (times `out_scale`).
 
-    The cache holds the values and one reciprocal root mean square per token; a slot holds the last projected rows."""
+    The cache holds the values and one f32 per token that turns them into keys (`key_scale`); a slot holds the last projected rows."""
 
     def __init__(self, weights: GpuWeights, prefix: str, spec: dict, eps: float, dtype: torch.dtype, out_scale: float = 1.0):
         self.heads, self.kv_heads, self.dim, self.taps = int(spec["heads"]), int(spec["kv_heads"]), int(spec["dim"]), int(spec["conv"])
@@ -242,7 +242,7 @@ class WindowAttention:
         if tuple(self.conv.shape) != (self.taps, self.channels):
             raise ValueError(f"{prefix}: convolution {tuple(self.conv.shape)}, the configuration says {(self.taps, self.channels)}")
         rel = take("rel").float()
-        self.bias = rel[torch.tensor(distance_buckets(int(rel.shape[0]), float(spec["bias_max"])), device=rel.device)].t().contiguous()
+        self.bias = rel[torch.tensor(distance_buckets(int(rel.shape[0]), float(spec["bias_max"])), device=rel.device)].t().contiguous() * float(np.log2(np.e))
 
     @property
     def channels(self) -> int:
@@ -260,7 +260,7 @@ class WindowAttention:
                 f"{self.prefix}.g": ctx.arena.get("wa.g", (ctx.rows, self.heads), torch.float32)}
 
     def memory(self, cache_rows: int, slots: int, device) -> Tuple[torch.Tensor, ...]:
-        """(values, reciprocals, projected rows)."""
+        """(values, their scales as keys, projected rows)."""
         return (torch.zeros((cache_rows, self.kv_heads * self.dim), dtype=self.dtype, device=device),
                 torch.zeros(cache_rows, dtype=torch.float32, device=device),
                 torch.zeros((slots, max(1, self.taps - 1), self.channels), dtype=self.dtype, device=device))
