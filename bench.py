@@ -1385,7 +1385,7 @@ def run_side_kernels(device, model, peaks, context=2048):
         sc = step_context(device, model, arena, batch, count, kv, prompt)
         T, row = batch * count, left.kv_heads * left.dim
         copies = 2 if prompt else min(24, max(2, (256 << 20) // (batch * kv * row * 2)))
-        mem = [(torch.randn((sc.num_blocks * sc.block_size, row), device=device).to(bf), torch.ones(sc.num_blocks * sc.block_size, device=device),
+        mem = [(torch.randn((sc.num_blocks * sc.block_size, row), device=device).to(bf), torch.full((sc.num_blocks * sc.block_size,), left.scale * math.log2(math.e), device=device),
                 torch.zeros((batch, left.taps - 1, left.channels), dtype=bf, device=device)) for _ in range(copies)]
         q, gate = torch.randn((T, left.out_features), device=device).to(bf), torch.randn((T, left.heads), device=device)
         qk, o, q2 = torch.randn((T, left.channels), device=device).to(bf), torch.empty((T, left.out_features), dtype=bf, device=device), torch.empty_like(q)

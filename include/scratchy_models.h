@@ -176,15 +176,18 @@ int32_t scr_mlstm_finish(scr_ctx* ctx, int32_t dtype, const scr_mlstm_shape* s, 
  * therefore holds the values only, [num_blocks * block_size, kv_heads * dim] of dtype, and one f32 per token, key_scale =
  * scale * log2(e) / (root mean square of its keys); the key norm's weight is folded into the queries.
  * Position i sees j <= i with i - j < window or j < keep_first.  Score in powers of two: q.v * key_scale +
- * bias[h][min(i - j, n_bias - 1)], the bias of the softmax times log2(e). */
+ * bias[h][min(i - j, n_bias - 1)], the bias of the softmax times log2(e).  A head's bias row has SCR_BIAS_LO copies of its first
+ * entry before it and SCR_BIAS_HI copies of its last one behind it (a tile of keys then needs no limits). */
+#define SCR_BIAS_LO 192
+#define SCR_BIAS_HI 96
 typedef struct scr_window_shape {
     int32_t heads, kv_heads, dim, taps;
     int32_t window, keep_first, n_bias;
     int32_t block_size, num_blocks, max_blocks;
     float eps, scale, out_scale;
 } scr_window_shape;
-/* proj (dtype, row stride ld): q [heads * dim] | k [kv_heads * dim] as projected; conv [taps, (heads + kv_heads) * dim] and
- * norm [(heads + kv_heads) * dim] f32.  conv_state (dtype) [num_slots, taps - 1, (heads + kv_heads) * dim] holds the last
+/* proj (dtype, row stride ld): q [heads * dim] | k [kv_heads * dim] as projected; conv [taps, (heads + kv_heads) * dim] f32;
+ * norm [heads * dim] f32, the query norm's weight times the key norm's of the head's keys.  conv_state (dtype) [num_slots, taps - 1, (heads + kv_heads) * dim] holds the last
  * projected rows of every sequence, oldest first; zeros precede position 0 whatever the slot holds.  Writes the queries
  * (dtype [rows, heads * dim], normed, times the key norm's weight), the cache rows, key_scale and conv_state. */
 int32_t scr_window_prepare(scr_ctx* ctx, int32_t dtype, const scr_window_shape* s, const scr_step* st, const void* proj, int64_t ld,

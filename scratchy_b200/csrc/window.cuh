@@ -33,3 +33,13 @@ __device__ __forceinline__ long long window_row(const scr_window_shape& s, const
     }
     return (long long)block * s.block_size + (pos - b * s.block_size);
 }
+
+// Rows of `heads` vectors of `dim` bf16 values: boxes of 64 dimensions of one head and `box_rows` rows, 128-byte swizzle, zeros outside.
+static inline bool window_map(CUtensorMap* map, const void* base, uint64_t dim, uint64_t heads, uint64_t rows, uint32_t box_rows) {
+    tc_encode_tiled_fn enc = tc_tensor_map_encoder();
+    if (!enc) return false;
+    const cuuint64_t dims[3] = {dim, heads, rows}, strides[2] = {dim * 2, dim * 2 * heads};
+    const cuuint32_t box[3] = {64, 1, box_rows}, one[3] = {1, 1, 1};
+    return enc(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(base), dims, strides, box, one, CU_TENSOR_MAP_INTERLEAVE_NONE,
+               CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
+}

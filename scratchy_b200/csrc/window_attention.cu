@@ -9,6 +9,8 @@
 //   window_prefill.cu              bf16: prompts on tcgen05
 #include "window.cuh"
 
+#include <algorithm>
+
 bool window_mma_applies(const scr_window_shape& s);
 int32_t window_mma_launch(scr_ctx* ctx, const scr_window_shape& s, const scr_step& st, const void* q, const void* cache, const float* key_scale,
                           const float* bias, const float* gate, int64_t ld_gate, void* out, int64_t ld_out, cudaStream_t stream);
@@ -48,149 +50,279 @@ template <> struct Vec<float, 8> {
         for (int i = 0; i < 8; i += 4) *reinterpret_cast<float4*>(p + i) = make_float4(v[i], v[i + 1], v[i + 2], v[i + 3]);
     }
 };
-template <typename T> struct Vec<T, 1> {
-    static __device__ __forceinline__ void get(const T* p, float (&v)[1]) { v[0] = to_f32(*p); }
-    static __device__ __forceinline__ void put(T* p, const float (&v)[1]) { *p = from_f32<T>(v[0]); }
-};
 
-// One CTA per ROWS rows.  A thread owns the same channels throughout, keeps their taps and the last projected values in
-// registers while it walks the rows, and moves the convolution state of a sequence of one token along itself.
-// HIST: taps - 1 where that is small, else -1.
-template <typename T, int VEC, int HIST, int ROWS>
-__global__ void __launch_bounds__(WP_T) window_prepare_kernel(scr_window_shape s, scr_step st, const T* __restrict__ proj, long long ld,
-                                                              const float* __restrict__ conv, const float* __restrict__ norm, T* state,
-                                                              T* __restrict__ q, T* __restrict__ cache, float* __restrict__ key_scale, int* status) {
-    extern __shared__ float4 wp_smem[];
-    float* y = reinterpret_cast<float*>(wp_smem);            // [ROWS][channels]
-    __shared__ float red[WP_T / 32][2 * ROWS];
-    __shared__ int at_s[ROWS], pos_s[ROWS], count_s[ROWS], slot_s[ROWS];
-    __shared__ long long row_s[ROWS];
+// What a row of a step is to the convolution: its sequence's portion, slot and cache row.
+struct PrepRow {
+    long long cache;                                         // -1: none
+    int at, pos, count, slot;                                // at: rows of the portion before this one, -1: no such row
+};
+__device__ __forceinline__ PrepRow prep_row(const scr_window_shape& s, const scr_step& st, int r, int* status) {
+    PrepRow p{-1, -1, 0, 0, 0};
+    if (r >= st.rows) return p;
+    const int b = st.tok_seg[r], first = st.segs[b * 4];
+    p.count = st.segs[b * 4 + 1];
+    p.slot = st.segs[b * 4 + 3];
+    p.pos = st.tok_pos[r];
+    if (p.count <= 0) return p;
+    if (p.slot < 0 || p.slot >= st.num_slots || r < first || r >= first + p.count || first < 0 || first + p.count > st.rows) {
+        atomicCAS(status, 0, SEQ_BAD_SLOT);
+        return p;
+    }
+    p.at = r - first;
+    p.cache = window_row(s, st.block_table, b, p.pos, status);
+    return p;
+}
+
+// One CTA per row, any sizes.  A thread owns the same channels throughout, so that it can move the convolution state of a
+// sequence of one token along.
+template <typename T>
+__global__ void __launch_bounds__(WP_T) window_prepare_any_kernel(scr_window_shape s, scr_step st, const T* __restrict__ proj, long long ld,
+                                                                  const float* __restrict__ conv, const float* __restrict__ norm, T* state,
+                                                                  T* __restrict__ q, T* __restrict__ cache, float* __restrict__ key_scale, int* status) {
+    extern __shared__ float y[];                             // [channels]
+    __shared__ float red_q[WP_T / 32], red_k[WP_T / 32];
     pdl_trigger();
     pdl_wait();
-    const int r0 = blockIdx.x * ROWS, tid = threadIdx.x;
-    const int nq = s.heads * s.dim, C = nq + s.kv_heads * s.dim, hist = HIST >= 0 ? HIST : s.taps - 1;
-    if (tid < ROWS) {                                        // at: rows of the portion before this one, -1: no such row
-        const int r = r0 + tid, b = r < st.rows ? st.tok_seg[r] : 0;
-        const int first = st.segs[b * 4], count = st.segs[b * 4 + 1], slot = st.segs[b * 4 + 3];
-        const bool in = r < st.rows && count > 0;
-        const bool ok = in && slot >= 0 && slot < st.num_slots && r >= first && r < first + count && first >= 0 && first + count <= st.rows;
-        if (in && !ok) atomicCAS(status, 0, SEQ_BAD_SLOT);
-        at_s[tid] = ok ? r - first : -1;
-        pos_s[tid] = ok ? st.tok_pos[r] : 0;
-        count_s[tid] = count;
-        slot_s[tid] = slot;
-        row_s[tid] = ok ? window_row(s, st.block_table, b, pos_s[tid], status) : -1;
+    const int r = blockIdx.x, tid = threadIdx.x, nq = s.heads * s.dim, C = nq + s.kv_heads * s.dim, hist = s.taps - 1;
+    const PrepRow p = prep_row(s, st, r, status);
+    if (p.at < 0) return;
+    T* old = state + (size_t)p.slot * hist * C;              // oldest first: row hist - d is d tokens before the portion
+    float sq = 0.0f, sk = 0.0f;
+    for (int c = tid; c < C; c += WP_T) {
+        float acc = 0.0f;
+        for (int o = hist; o >= 0; --o) {                    // the token o before this one
+            T u = from_f32<T>(0.0f);
+            if (p.pos - o >= 0) u = o <= p.at ? proj[(r - o) * ld + c] : old[(size_t)(hist - (o - p.at)) * C + c];
+            if (p.count == 1 && o < hist) old[(size_t)(hist - o - 1) * C + c] = u;
+            acc = fmaf(conv[(size_t)(hist - o) * C + c], to_f32(u), acc);
+        }
+        y[c] = acc;
+        if (c < nq) sq = fmaf(acc, acc, sq);
+        else sk = fmaf(acc, acc, sk);
     }
+    const float iq = 1.0f / sqrtf(cta_sum<WP_T>(sq, red_q) / float(nq) + s.eps);
+    const float ik = 1.0f / sqrtf(cta_sum<WP_T>(sk, red_k) / float(C - nq) + s.eps);
+    for (int c = tid; c < C; c += WP_T) {
+        if (c < nq) q[(size_t)r * nq + c] = from_f32<T>(y[c] * iq * norm[c]);
+        else if (p.cache >= 0) cache[p.cache * (C - nq) + (c - nq)] = from_f32<T>(y[c]);
+    }
+    if (tid == 0 && p.cache >= 0) key_scale[p.cache] = ik * s.scale * 1.4426950408889634f;
+}
+
+// One CTA per ROWS rows, taps <= TAPS: a thread has PER runs of 8 channels, requests the rows and the TAPS - 1 before them at
+// once, and keeps everything in registers.  What does not come from the preceding kernel is read before the wait for it.
+template <typename T, int TAPS, int PER, int ROWS>
+__global__ void __launch_bounds__(512) window_prepare_kernel(scr_window_shape s, scr_step st, const T* __restrict__ proj, long long ld,
+                                                             const float* __restrict__ conv, const float* __restrict__ norm, T* state,
+                                                             T* __restrict__ q, T* __restrict__ cache, float* __restrict__ key_scale, int* status) {
+    constexpr int N = ROWS + TAPS - 1;
+    __shared__ float red[16][2 * ROWS];
+    __shared__ PrepRow rows[ROWS];
+    pdl_trigger();
+    const int r0 = blockIdx.x * ROWS, tid = threadIdx.x, nq = s.heads * s.dim, C = nq + s.kv_heads * s.dim, hist = s.taps - 1;
+    if (tid < ROWS) rows[tid] = prep_row(s, st, r0 + tid, status);
     __syncthreads();
-    float sq[ROWS], sk[ROWS];
+    float sq[ROWS], sk[ROWS], y[PER][ROWS][8];
 #pragma unroll
     for (int i = 0; i < ROWS; ++i) sq[i] = sk[i] = 0.0f;
-    for (int c = tid * VEC; c < C; c += WP_T * VEC) {
-        constexpr int H = HIST >= 0 ? HIST : 1;
-        float w[H + 1][VEC], u[H + 1][VEC];                  // u[o]: the token o before this one
-        if (HIST >= 0)
+    if (PER > 1) pdl_wait();
 #pragma unroll
-            for (int o = 0; o <= H; ++o) Vec<float, VEC>::get(conv + (size_t)(hist - o) * C + c, w[o]);
+    for (int k = 0; k < PER; ++k) {
+        const int c = (k * blockDim.x + tid) * 8;
+        const bool in = c < C;
+        float w[TAPS][8];                                    // w[o]: of the token o before
+#pragma unroll
+        for (int o = 0; o < TAPS; ++o) {
+            if (in && o <= hist) {
+                Vec<float, 8>::get(conv + (size_t)(hist - o) * C + c, w[o]);
+            } else {
+#pragma unroll
+                for (int j = 0; j < 8; ++j) w[o][j] = 0.0f;
+            }
+        }
+        if (PER == 1) pdl_wait();
+        if (!in) continue;
+        // what came before the first row: rows of the step, or the state of its sequence
+        float u[N][8];
+        const PrepRow p0 = rows[0];
+#pragma unroll
+        for (int i = 0; i < N; ++i) {
+            const int o = TAPS - 1 - i;                      // > 0: so many before the first row
+            const T* src = nullptr;
+            if (o <= 0) src = r0 - o < st.rows ? proj + (r0 - o) * ld + c : nullptr;
+            else if (o <= hist && p0.at >= 0 && p0.pos - o >= 0)
+                src = o <= p0.at ? proj + (r0 - o) * ld + c : state + ((size_t)p0.slot * hist + (hist - (o - p0.at))) * C + c;
+            if (src) Vec<T, 8>::get(src, u[i]);
+            else
+#pragma unroll
+                for (int j = 0; j < 8; ++j) u[i][j] = 0.0f;
+        }
 #pragma unroll
         for (int i = 0; i < ROWS; ++i) {
-            const int at = at_s[i], r = r0 + i, pos = pos_s[i];
-            if (at < 0) continue;
-            T* old = state + (size_t)slot_s[i] * hist * C + c;               // oldest first: row hist - d is d tokens before the portion
-            auto before = [&](int o, float (&v)[VEC]) {
-                if (pos - o < 0) {
+            const PrepRow p = rows[i];
+            if (p.at < 0) continue;
+            float acc[8];
+            if (i > 0 && p.at < hist) {                      // a sequence starts within these rows: its own past
 #pragma unroll
-                    for (int j = 0; j < VEC; ++j) v[j] = 0.0f;
-                } else if (o <= at) {
-                    Vec<T, VEC>::get(proj + (r - o) * ld + c, v);
-                } else {
-                    Vec<T, VEC>::get(old + (size_t)(hist - (o - at)) * C, v);
-                }
-            };
-            float acc[VEC], now[VEC];
+                for (int o = 1; o < TAPS; ++o)
+                    if (o > p.at) {
+                        const bool has = o <= hist && p.pos - o >= 0;
+                        float v[8];
+                        if (has) Vec<T, 8>::get(state + ((size_t)p.slot * hist + (hist - (o - p.at))) * C + c, v);
 #pragma unroll
-            for (int j = 0; j < VEC; ++j) acc[j] = 0.0f;
-            if (HIST >= 0) {
-                if (i > 0 && at > 0) {                       // the row before is this sequence's: move along
-#pragma unroll
-                    for (int o = H; o > 0; --o)
-#pragma unroll
-                        for (int j = 0; j < VEC; ++j) u[o][j] = u[o - 1][j];
-                } else {
-#pragma unroll
-                    for (int o = H; o > 0; --o) before(o, u[o]);
-                }
-                Vec<T, VEC>::get(proj + r * ld + c, u[0]);
-                if (count_s[i] == 1) {
-#pragma unroll
-                    for (int o = H; o > 0; --o) Vec<T, VEC>::put(old + (size_t)(hist - o) * C, u[o - 1]);
-                }
-#pragma unroll
-                for (int o = H; o >= 0; --o)
-#pragma unroll
-                    for (int j = 0; j < VEC; ++j) acc[j] = fmaf(w[o][j], u[o][j], acc[j]);
-            } else {
-                for (int o = hist; o >= 0; --o) {
-                    if (o > 0) before(o, now);
-                    else Vec<T, VEC>::get(proj + r * ld + c, now);
-                    if (count_s[i] == 1 && o < hist) Vec<T, VEC>::put(old + (size_t)(hist - o - 1) * C, now);
-                    Vec<float, VEC>::get(conv + (size_t)(hist - o) * C + c, w[0]);
-#pragma unroll
-                    for (int j = 0; j < VEC; ++j) acc[j] = fmaf(w[0][j], now[j], acc[j]);
-                }
+                        for (int j = 0; j < 8; ++j) u[i + TAPS - 1 - o][j] = has ? v[j] : 0.0f;
+                    }
             }
+#pragma unroll
+            for (int j = 0; j < 8; ++j) acc[j] = 0.0f;
+#pragma unroll
+            for (int o = TAPS - 1; o >= 0; --o)
+#pragma unroll
+                for (int j = 0; j < 8; ++j) acc[j] = fmaf(w[o][j], u[i + TAPS - 1 - o][j], acc[j]);
             float ss = 0.0f;
 #pragma unroll
-            for (int j = 0; j < VEC; ++j) ss = fmaf(acc[j], acc[j], ss);
-            Vec<float, VEC>::put(y + (size_t)i * C + c, acc);
+            for (int j = 0; j < 8; ++j) {
+                ss = fmaf(acc[j], acc[j], ss);
+                y[k][i][j] = acc[j];
+            }
             if (c < nq) sq[i] += ss;
             else sk[i] += ss;
+            if (p.count == 1) {                              // one token: the state moves along (its old rows have been read)
+#pragma unroll
+                for (int o = TAPS - 1; o > 0; --o)
+                    if (o <= hist) Vec<T, 8>::put(state + ((size_t)p.slot * hist + (hist - o)) * C + c, u[i + TAPS - 1 - (o - 1)]);
+            }
         }
     }
 #pragma unroll
     for (int i = 0; i < ROWS; ++i) {
-        sq[i] = warp_sum(sq[i]);
-        sk[i] = warp_sum(sk[i]);
+        const float a = warp_sum(sq[i]), b = warp_sum(sk[i]);
         if ((tid & 31) == 0) {
-            red[tid >> 5][2 * i] = sq[i];
-            red[tid >> 5][2 * i + 1] = sk[i];
+            red[tid >> 5][2 * i] = a;
+            red[tid >> 5][2 * i + 1] = b;
         }
     }
     __syncthreads();
 #pragma unroll
     for (int i = 0; i < ROWS; ++i) {
         sq[i] = sk[i] = 0.0f;
-#pragma unroll
-        for (int w = 0; w < WP_T / 32; ++w) {
+        for (int w = 0; w < (int)blockDim.x / 32; ++w) {
             sq[i] += red[w][2 * i];
             sk[i] += red[w][2 * i + 1];
         }
         sq[i] = 1.0f / sqrtf(sq[i] / float(nq) + s.eps);
         sk[i] = 1.0f / sqrtf(sk[i] / float(C - nq) + s.eps);
     }
-    const int group = s.heads / s.kv_heads;
-    for (int c = tid * VEC; c < C; c += WP_T * VEC) {
-        float v[VEC], w[VEC], wk[VEC];
-        if (c < nq) {
-            const int h = c / s.dim;
-            Vec<float, VEC>::get(norm + c, w);
-            Vec<float, VEC>::get(norm + nq + h / group * s.dim + (c - h * s.dim), wk);
-        }
+#pragma unroll
+    for (int k = 0; k < PER; ++k) {
+        const int c = (k * blockDim.x + tid) * 8;
+        if (c >= C) continue;
+        float w[8];
+        if (c < nq) Vec<float, 8>::get(norm + c, w);
 #pragma unroll
         for (int i = 0; i < ROWS; ++i) {
-            if (at_s[i] < 0) continue;
-            Vec<float, VEC>::get(y + (size_t)i * C + c, v);
+            const PrepRow p = rows[i];
+            if (p.at < 0) continue;
             if (c < nq) {
 #pragma unroll
-                for (int j = 0; j < VEC; ++j) v[j] = v[j] * sq[i] * w[j] * wk[j];
-                Vec<T, VEC>::put(q + (size_t)(r0 + i) * nq + c, v);
-            } else if (row_s[i] >= 0) {
-                Vec<T, VEC>::put(cache + row_s[i] * (C - nq) + (c - nq), v);
+                for (int j = 0; j < 8; ++j) y[k][i][j] *= sq[i] * w[j];
+                Vec<T, 8>::put(q + (size_t)(r0 + i) * nq + c, y[k][i]);
+            } else if (p.cache >= 0) {
+                Vec<T, 8>::put(cache + p.cache * (C - nq) + (c - nq), y[k][i]);
             }
         }
     }
 #pragma unroll
     for (int i = 0; i < ROWS; ++i)
-        if (tid == i && at_s[i] >= 0 && row_s[i] >= 0) key_scale[row_s[i]] = sk[i] * s.scale * 1.4426950408889634f;
+        if (tid == i && rows[i].cache >= 0) key_scale[rows[i].cache] = sk[i] * s.scale * 1.4426950408889634f;
+}
+
+// Many rows: a CTA walks up to WP_WALK consecutive rows with the taps and the last projected values in registers, the next row's
+// values in flight; one barrier per row.
+constexpr int WP_WALK = 64;
+template <typename T, int TAPS>
+__global__ void __launch_bounds__(512) window_prepare_walk_kernel(scr_window_shape s, scr_step st, int per, const T* __restrict__ proj, long long ld,
+                                                                  const float* __restrict__ conv, const float* __restrict__ norm, T* state,
+                                                                  T* __restrict__ q, T* __restrict__ cache, float* __restrict__ key_scale, int* status) {
+    __shared__ float red[2][16][2];
+    __shared__ PrepRow rows[WP_WALK];
+    pdl_trigger();
+    const int r0 = blockIdx.x * per, n = min(per, st.rows - r0), tid = threadIdx.x, nq = s.heads * s.dim, C = nq + s.kv_heads * s.dim, hist = s.taps - 1;
+    for (int i = tid; i < n; i += blockDim.x) rows[i] = prep_row(s, st, r0 + i, status);
+    const int c = tid * 8;
+    const bool in = c < C, query = c < nq;
+    float w[TAPS][8], wn[8], u[TAPS][8], next[8];            // w[o], u[o]: of the token o before
+#pragma unroll
+    for (int o = 0; o < TAPS; ++o) {
+#pragma unroll
+        for (int j = 0; j < 8; ++j) w[o][j] = u[o][j] = 0.0f;
+        if (in && o <= hist) Vec<float, 8>::get(conv + (size_t)(hist - o) * C + c, w[o]);
+    }
+    if (query) Vec<float, 8>::get(norm + c, wn);
+    __syncthreads();
+    pdl_wait();
+    if (in) {
+#pragma unroll
+        for (int o = 1; o < TAPS; ++o)                       // the rows before the first one, where they are of this step
+            if (o <= hist && o <= rows[0].at) Vec<T, 8>::get(proj + (r0 - o) * ld + c, u[o - 1]);
+        Vec<T, 8>::get(proj + r0 * ld + c, next);
+    }
+    for (int i = 0; i < n; ++i) {
+        const PrepRow p = rows[i];
+        float acc[8], ss = 0.0f;
+        if (in) {
+#pragma unroll
+            for (int o = TAPS - 1; o > 0; --o)
+#pragma unroll
+                for (int j = 0; j < 8; ++j) u[o][j] = u[o - 1][j];
+#pragma unroll
+            for (int j = 0; j < 8; ++j) u[0][j] = next[j];
+            if (i + 1 < n) Vec<T, 8>::get(proj + (r0 + i + 1) * ld + c, next);
+            if (p.at >= 0 && p.at < hist) {                  // close to its portion's start: what lies before it is in the state
+#pragma unroll
+                for (int o = 1; o < TAPS; ++o)
+                    if (o > p.at) {
+                        const bool has = o <= hist && p.pos - o >= 0;
+                        float v[8];
+                        if (has) Vec<T, 8>::get(state + ((size_t)p.slot * hist + (hist - (o - p.at))) * C + c, v);
+#pragma unroll
+                        for (int j = 0; j < 8; ++j) u[o][j] = has ? v[j] : 0.0f;
+                    }
+            }
+#pragma unroll
+            for (int j = 0; j < 8; ++j) acc[j] = 0.0f;
+#pragma unroll
+            for (int o = TAPS - 1; o >= 0; --o)
+#pragma unroll
+                for (int j = 0; j < 8; ++j) acc[j] = fmaf(w[o][j], u[o][j], acc[j]);
+#pragma unroll
+            for (int j = 0; j < 8; ++j) ss = fmaf(acc[j], acc[j], ss);
+            if (p.at >= 0 && p.count == 1) {                 // one token: the state moves along (its old rows have been read)
+#pragma unroll
+                for (int o = TAPS - 1; o > 0; --o)
+                    if (o <= hist) Vec<T, 8>::put(state + ((size_t)p.slot * hist + (hist - o)) * C + c, u[o - 1]);
+            }
+        }
+        const float a = warp_sum(query ? ss : 0.0f), b = warp_sum(query ? 0.0f : ss);
+        if ((tid & 31) == 0) {
+            red[i & 1][tid >> 5][0] = a;
+            red[i & 1][tid >> 5][1] = b;
+        }
+        __syncthreads();                                     // (two sets of sums: the next row's writers need not wait for the readers)
+        const bool key0 = c == nq;                           // the thread of the first key channels leaves the keys' scale
+        float sum = 0.0f;
+        for (int k = 0; k < (int)blockDim.x / 32; ++k) sum += red[i & 1][k][query ? 0 : 1];
+        if (!in || p.at < 0) continue;
+        const float inv = 1.0f / sqrtf(sum / float(query ? nq : C - nq) + s.eps);
+        if (query) {
+#pragma unroll
+            for (int j = 0; j < 8; ++j) acc[j] *= inv * wn[j];
+            Vec<T, 8>::put(q + (size_t)(r0 + i) * nq + c, acc);
+        } else if (p.cache >= 0) {
+            Vec<T, 8>::put(cache + p.cache * (C - nq) + (c - nq), acc);
+            if (key0) key_scale[p.cache] = inv * s.scale * 1.4426950408889634f;
+        }
+    }
 }
 
 // New state row j is the token hist - j before the next portion.  Sources lie behind their destinations, and a thread
@@ -238,7 +370,7 @@ __global__ void __launch_bounds__(WA_WARPS * 32) window_attention_plain_kernel(s
     for (int i = threadIdx.x; i < s.dim; i += WA_WARPS * 32) qs[i] = to_f32(qp[i]);
     __syncthreads();
     const int lo = max(0, pos - s.window + 1), kept = min(s.keep_first, lo), keys = kept + pos - lo + 1;
-    const float* bh = bias + (size_t)h * s.n_bias;
+    const float* bh = bias + (size_t)h * (SCR_BIAS_LO + s.n_bias + SCR_BIAS_HI) + SCR_BIAS_LO;
     float m = -INFINITY, l = 0.0f, acc[WA_MAX];
 #pragma unroll
     for (int i = 0; i < WA_MAX; ++i) acc[i] = 0.0f;
@@ -295,18 +427,27 @@ int32_t prepare(scr_ctx* ctx, const scr_window_shape& s, const scr_step& st, con
     if (C > 50 * 1024) return scr_fail(ctx, SCR_E_UNSUPPORTED, "%d query and key channels", C);
     const bool vec = s.dim % 8 == 0 && ld % 8 == 0 && scr_aligned16(proj) && scr_aligned16(conv) && scr_aligned16(norm) && scr_aligned16(conv_state) &&
                      scr_aligned16(q) && scr_aligned16(cache);
-    const bool many = vec && s.taps <= 4 && st.rows >= 4 * ctx->sm_count && C <= 12 * 1024;
-    auto kernel = !vec ? window_prepare_kernel<T, 1, -1, 1> : window_prepare_kernel<T, 8, -1, 1>;
-    if (vec && s.taps == 1) kernel = many ? window_prepare_kernel<T, 8, 0, 4> : window_prepare_kernel<T, 8, 0, 1>;
-    if (vec && s.taps == 2) kernel = many ? window_prepare_kernel<T, 8, 1, 4> : window_prepare_kernel<T, 8, 1, 1>;
-    if (vec && s.taps == 3) kernel = many ? window_prepare_kernel<T, 8, 2, 4> : window_prepare_kernel<T, 8, 2, 1>;
-    if (vec && s.taps == 4) kernel = many ? window_prepare_kernel<T, 8, 3, 4> : window_prepare_kernel<T, 8, 3, 1>;
-    const int per = many ? 4 : 1;
-    const size_t smem = (size_t)per * C * sizeof(float);
-    cudaError_t e = seq_smem(kernel, smem);
-    if (e == cudaSuccess)
-        e = launch_pdl(kernel, dim3(scr_ceil_div(st.rows, per)), dim3(WP_T), smem, stream, s, st, (const T*)proj, (long long)ld, conv, norm, (T*)conv_state, (T*)q,
-                       (T*)cache, key_scale, ctx->dev_status);
+    cudaError_t e;
+    if (vec && s.taps <= 4 && C <= 2 * 512 * 8) {
+        const bool two = C > 512 * 8;
+        const int threads = two ? 512 : scr_ceil_div(C / 8, 32) * 32;
+        if (!two && st.rows >= 2 * ctx->sm_count) {
+            const int per = std::min(WP_WALK, std::max(4, scr_ceil_div(st.rows, ctx->sm_count)));
+            e = launch_pdl(window_prepare_walk_kernel<T, 4>, dim3(scr_ceil_div(st.rows, per)), dim3(threads), 0, stream, s, st, per, (const T*)proj, (long long)ld,
+                           conv, norm, (T*)conv_state, (T*)q, (T*)cache, key_scale, ctx->dev_status);
+        } else {
+            auto kernel = !two ? window_prepare_kernel<T, 4, 1, 1> : st.rows >= 2 * ctx->sm_count ? window_prepare_kernel<T, 4, 2, 2> : window_prepare_kernel<T, 4, 2, 1>;
+            const int per = two && st.rows >= 2 * ctx->sm_count ? 2 : 1;
+            e = launch_pdl(kernel, dim3(scr_ceil_div(st.rows, per)), dim3(threads), 0, stream, s, st, (const T*)proj, (long long)ld, conv, norm, (T*)conv_state, (T*)q,
+                           (T*)cache, key_scale, ctx->dev_status);
+        }
+    } else {
+        const size_t smem = (size_t)C * sizeof(float);
+        e = seq_smem(window_prepare_any_kernel<T>, smem);
+        if (e == cudaSuccess)
+            e = launch_pdl(window_prepare_any_kernel<T>, dim3(st.rows), dim3(WP_T), smem, stream, s, st, (const T*)proj, (long long)ld, conv, norm, (T*)conv_state,
+                           (T*)q, (T*)cache, key_scale, ctx->dev_status);
+    }
     if (e != cudaSuccess) return scr_fail(ctx, SCR_E_CUDA, "window_prepare: %s", cudaGetErrorString(e));
     const int32_t rc = scr_check_launch(ctx, "window_prepare");
     if (rc || st.max_count == 1 || s.taps == 1) return rc;

@@ -1,9 +1,10 @@
 // Sliding-window attention for decoding and short portions, bf16, on mma.sync.  The rows that share a key/value head (the
-// tokens of a portion times the heads of a group) are the 16 rows of a tile; every warp walks key tiles of its own, 32 cache
-// rows at a time, through a ring of its own (cp.async), with no barrier between the warps:
-//   S = Q K^T with Q in registers; the keys' scale, bias, window; online softmax in f32 on
-//   the accumulators; P as a bf16 head and remainder (two products: the weights keep about 16 bits); O += P V from the very
-//   same shared-memory rows, read transposed.
+// tokens of a portion times the heads of a group) come in tiles of 8; every warp walks key tiles of its own, 32 cache rows
+// at a time, through a ring of its own (tiled TMA loads from the paged cache), with no barrier between the warps:
+//   S = Q K^T with Q in registers; the keys' scale, bias, window; online softmax in f32 on the accumulators; O += P V from
+//   the very same shared-memory rows, read transposed.
+// The 8 rows fill half of an mma's 16: in P V the other half carries the remainders of the weights, P - bf16(P), so that
+// one product keeps about 16 bits of them; the two halves of O are added at the end.
 // The warps' states meet in shared memory; the key shares of a cluster's CTAs meet through distributed shared memory.
 #include "window.cuh"
 
@@ -11,16 +12,17 @@
 
 namespace {
 
-constexpr int WM_WARPS = 4, WM_THREADS = WM_WARPS * 32, WM_KEYS = 32, WM_MAX_CLUSTER = 8;
+constexpr int WM_WARPS = 4, WM_THREADS = WM_WARPS * 32, WM_ROWS = 8, WM_KEYS = 32, WM_MAX_CLUSTER = 8;
+constexpr uint32_t WM_CHUNK = WM_KEYS * 128;                 // 64 dimensions of a key tile
 
 // NK: dimensions in steps of 16 (dim <= 16 * NK); STAGES: key tiles a warp keeps in flight
 template <int NK, int STAGES>
 struct WmSmem {
-    static constexpr int kLd = NK * 16 + 8;                  // elements per key row: odd multiple of 16 bytes
-    static constexpr int kTile = WM_KEYS * kLd * 2, kStage = kTile + WM_KEYS * 4, kWarp = STAGES * kStage;
-    static constexpr int kO = 16 * (NK * 16 + 4) * 4;        // a warp's O, f32, over its ring
-    static constexpr int kRing = kWarp > kO ? kWarp : kO;
-    static constexpr int kTotal = WM_WARPS * kRing + (WM_WARPS + 1) * 16 * 2 * 4;
+    static constexpr int kChunks = (NK * 16 + 63) / 64, kOLd = NK * 16 + 4;
+    static constexpr uint32_t kTile = kChunks * WM_CHUNK, kRing = STAGES * kTile;                // per warp; the ring later holds its O
+    static constexpr uint32_t kScale = WM_WARPS * kRing, kBars = kScale + WM_WARPS * STAGES * WM_KEYS * 4;
+    static constexpr uint32_t kMl = kBars + WM_WARPS * STAGES * 8, kTotal = kMl + (WM_WARPS + 1) * WM_ROWS * 8 + 1024;
+    static_assert(WM_ROWS * kOLd * 4 <= (int)kRing, "O fits a ring");
 };
 
 __device__ __forceinline__ float wm_peer(const float* p, uint32_t rank) {
@@ -38,7 +40,6 @@ struct WmArgs {
     scr_window_shape s;
     scr_step st;
     const bf16* q;
-    const bf16* cache;
     const float* key_scale;
     const float* bias;
     const float* gate;
@@ -50,206 +51,180 @@ struct WmArgs {
 };
 
 template <int NK, int STAGES>
-__global__ void __launch_bounds__(WM_THREADS) window_attention_mma_kernel(const WmArgs a) {
-    extern __shared__ __align__(128) unsigned char wm_smem[];
+__global__ void __launch_bounds__(WM_THREADS) window_attention_mma_kernel(const __grid_constant__ CUtensorMap k_map, const __grid_constant__ WmArgs a) {
+    extern __shared__ uint8_t wm_smem[];
     using SM = WmSmem<NK, STAGES>;
-    constexpr int LD = SM::kLd, NO = NK * 2;                 // 8-column tiles of O
+    constexpr int NO = NK * 2, OLD = SM::kOLd;               // 8-column tiles of O
     constexpr bool QREG = NK <= 8;
+    const uint32_t base = (smem_u32(wm_smem) + 1023u) & ~1023u;
+    uint8_t* gen = wm_smem + (base - smem_u32(wm_smem));
     const scr_window_shape& s = a.s;
     const int dim = s.dim, G = s.kv_heads, group = s.heads / G;
     pdl_trigger();
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, gr = lane >> 2, t4 = lane & 3, lm = lane >> 3, lr = lane & 7;
     const int split = blockIdx.x % a.splits, g = blockIdx.x / a.splits % G, tile = blockIdx.x / a.splits / G, b = blockIdx.y;
     const int first = a.st.segs[b * 4], count = a.st.segs[b * 4 + 1], pos0 = a.st.segs[b * 4 + 2];
-    const int r0 = tile * 16, nrows = min(16, count * group - r0);
+    const int r0 = tile * WM_ROWS, nrows = min(WM_ROWS, count * group - r0);
     if (nrows <= 0 || first < 0 || first + count > a.st.rows) {          // (the whole cluster)
         pdl_wait();
         return;
     }
     const int p_lo = pos0 + r0 / group, p_hi = pos0 + (r0 + nrows - 1) / group;
     const WindowTiles tiles = window_tiles(s, p_lo, p_hi, WM_KEYS);
-    unsigned char* ring = wm_smem + warp * SM::kRing;
+    const uint32_t ring = base + warp * SM::kRing, bars = base + SM::kBars + warp * STAGES * 8;
+    float* scales = reinterpret_cast<float*>(gen + SM::kScale) + warp * STAGES * WM_KEYS;
     const int* table = a.st.block_table + (size_t)b * s.max_blocks;
-    const int chunks = dim / 8, stride = a.splits * WM_WARPS, i0 = split * WM_WARPS + warp;
-    const long long row_size = (long long)G * dim;
+    const int stride = a.splits * WM_WARPS, i0 = split * WM_WARPS + warp;
     // first cache row of this warp's tile number n, -1: no such tile
-    auto look_up = [&](int n) -> long long {
+    auto look_up = [&](int n) -> int {
         const int i = i0 + n * stride;
         if (i >= tiles.count) return -1;
         const int key = tiles.tile(i) * WM_KEYS, blk = key / s.block_size;
-        const int block = blk < s.max_blocks ? table[blk] : -1;
+        int block = blk < s.max_blocks ? table[blk] : -1;
         if (block < 0 || block >= s.num_blocks) {
-            if (lane == 0) atomicCAS(a.status, 0, blk < s.max_blocks ? SEQ_BAD_BLOCK : SEQ_BAD_POSITION);
-            return -1;
+            atomicCAS(a.status, 0, blk < s.max_blocks ? SEQ_BAD_BLOCK : SEQ_BAD_POSITION);
+            block = 0;
         }
-        return (long long)block * s.block_size + (key - blk * s.block_size);
+        return block * s.block_size + (key - blk * s.block_size);
     };
-    auto load = [&](int n, long long row) {
-        if (row >= 0) {
-            unsigned char* st = ring + (n % STAGES) * SM::kStage;
-            const bf16* src = a.cache + row * row_size + (size_t)g * dim;
-            const uint32_t dst = smem_u32(st);
-#pragma unroll 4
-            for (int c = lane; c < WM_KEYS * NK * 2; c += 32) {
-                const int key = c / (NK * 2), x = c % (NK * 2);
-                if (x < chunks) cp_async16(dst + (key * LD + x * 8) * 2, src + key * row_size + x * 8, true);
-            }
-            if (lane < WM_KEYS / 4) cp_async16(dst + SM::kTile + lane * 16, a.key_scale + row + lane * 4, true);
-        }
-        cp_async_commit();
+    auto load = [&](int stage, int row) {                    // lane 0
+        if (row < 0) return;
+        const uint32_t bar = bars + stage * 8;
+        mbar_arrive_expect_tx(bar, SM::kTile + WM_KEYS * 4);
+#pragma unroll
+        for (int c = 0; c < SM::kChunks; ++c) tma_load_3d(ring + stage * SM::kTile + c * WM_CHUNK, &k_map, c * 64, g, row, bar);
+        bulk_g2s(smem_u32(scales + stage * WM_KEYS), a.key_scale + row, WM_KEYS * 4, bar);
     };
-    // zero what the rows hold beyond dim (the last steps of 16 read it)
-    if (dim < NK * 16)
-        for (int i = lane; i < STAGES * WM_KEYS * (NK * 16 - dim); i += 32) {
-            const int row = i / (NK * 16 - dim), c = dim + i % (NK * 16 - dim);
-            reinterpret_cast<bf16*>(ring + row / WM_KEYS * SM::kStage)[(row % WM_KEYS) * LD + c] = __float2bfloat16_rn(0.0f);
-        }
-    pdl_wait();
+    if (lane == 0) {
 #pragma unroll
-    for (int n = 0; n < STAGES - 1; ++n) load(n, look_up(n));
-    long long next = look_up(STAGES - 1);
-
-    // this lane's two rows: gr and gr + 8 of the tile
-    int head[2], pos[2];
-    const bf16* qp[2];
-    const float* bias[2];
-    float far[2];
-#pragma unroll
-    for (int x = 0; x < 2; ++x) {
-        const int r = r0 + min(gr + x * 8, nrows - 1), t = r / group;
-        head[x] = g * group + (r - t * group);
-        pos[x] = pos0 + t;
-        qp[x] = a.q + ((size_t)(first + t) * s.heads + head[x]) * dim;
-        bias[x] = a.bias + (size_t)head[x] * s.n_bias;
-        far[x] = bias[x][s.n_bias - 1];
+        for (int n = 0; n < STAGES; ++n) mbar_init(bars + n * 8, 1);
+        fence_mbar_init();
     }
-    auto q_at = [&](int x, int c) { return c < dim ? *reinterpret_cast<const uint32_t*>(qp[x] + c) : 0u; };
-    auto load_q = [&](int ks, uint32_t (&f)[4]) {
-        f[0] = q_at(0, ks * 16 + t4 * 2);
-        f[1] = q_at(1, ks * 16 + t4 * 2);
-        f[2] = q_at(0, ks * 16 + 8 + t4 * 2);
-        f[3] = q_at(1, ks * 16 + 8 + t4 * 2);
-    };
-    uint32_t qf[QREG ? NK : 1][4];
+    pdl_wait();
+    if (lane == 0) {
+#pragma unroll
+        for (int n = 0; n < STAGES; ++n) load(n, look_up(n));
+    }
+    __syncwarp();
+
+    // this lane's row: gr of the tile
+    const int row = r0 + min(gr, nrows - 1), tok = row / group, head = g * group + (row - tok * group), pos = pos0 + tok;
+    const bf16* qp = a.q + ((size_t)(first + tok) * s.heads + head) * dim;
+    const float* bias = a.bias + (size_t)head * (SCR_BIAS_LO + s.n_bias + SCR_BIAS_HI) + SCR_BIAS_LO;
+    const float far = bias[s.n_bias - 1];
+    auto q_at = [&](int c) { return c < dim ? *reinterpret_cast<const uint32_t*>(qp + c) : 0u; };
+    uint32_t qf[QREG ? NK : 1][2];
     if (QREG)
 #pragma unroll
-        for (int ks = 0; ks < (QREG ? NK : 0); ++ks) load_q(ks, qf[ks]);
-    float acc[NO][4] = {}, m[2] = {-1e30f, -1e30f}, l[2] = {0.0f, 0.0f};
+        for (int ks = 0; ks < (QREG ? NK : 0); ++ks) {
+            qf[ks][0] = q_at(ks * 16 + t4 * 2);
+            qf[ks][1] = q_at(ks * 16 + 8 + t4 * 2);
+        }
+    float acc[NO][4] = {}, m = -1e30f, l = 0.0f;
+    int stage = 0;
+    uint32_t phase = 0;
     for (int n = 0; i0 + n * stride < tiles.count; ++n) {
-        asm volatile("cp.async.wait_group %0;" ::"n"(STAGES - 2) : "memory");
-        __syncwarp();
-        load(n + STAGES - 1, next);                          // (into the stage that the tile before has left)
-        next = look_up(n + STAGES);
-        const unsigned char* stg = ring + (n % STAGES) * SM::kStage;
-        const bf16* K = reinterpret_cast<const bf16*>(stg);
-        const float* inv = reinterpret_cast<const float*>(stg + SM::kTile);
+        const int next = lane == 0 ? look_up(n + STAGES) : -1;
+        mbar_wait(bars + stage * 8, phase, a.status, TC_ERR_FULL_WAIT);
+        const uint32_t K = ring + stage * SM::kTile;
+        const float* scale = scales + stage * WM_KEYS;
         const int key0 = tiles.tile(i0 + n * stride) * WM_KEYS;
         float sc[4][4] = {};
         {
-            const uint32_t kb = smem_u32(K + ((lm >> 1) * 8 + lr) * LD + (lm & 1) * 8);
+            const uint32_t kb = K + ((lm >> 1) * 8 + lr) * 128;
 #pragma unroll
             for (int ks = 0; ks < NK; ++ks) {
-                uint32_t kf[2][4], f[4];
-                ldsm_x4(kb + ks * 32, kf[0]);
-                ldsm_x4(kb + ks * 32 + 16 * LD * 2, kf[1]);
+                uint32_t kf[2][4], q0, q1;
+                const uint32_t at = kb + (ks >> 2) * WM_CHUNK + ((((ks & 3) * 2 + (lm & 1)) ^ lr) << 4);
+                ldsm_x4(at, kf[0]);
+                ldsm_x4(at + 16 * 128, kf[1]);
                 if (QREG) {
-#pragma unroll
-                    for (int j = 0; j < 4; ++j) f[j] = qf[QREG ? ks : 0][j];
+                    q0 = qf[QREG ? ks : 0][0];
+                    q1 = qf[QREG ? ks : 0][1];
                 } else {
-                    load_q(ks, f);
+                    q0 = q_at(ks * 16 + t4 * 2);
+                    q1 = q_at(ks * 16 + 8 + t4 * 2);
                 }
 #pragma unroll
-                for (int x = 0; x < 4; ++x) mma_16816(sc[x], f[0], f[1], f[2], f[3], kf[x >> 1][(x & 1) * 2], kf[x >> 1][(x & 1) * 2 + 1]);
+                for (int x = 0; x < 4; ++x) mma_16816(sc[x], q0, 0u, q1, 0u, kf[x >> 1][(x & 1) * 2], kf[x >> 1][(x & 1) * 2 + 1]);
             }
         }
-        const bool plain = key0 + WM_KEYS - 1 <= p_lo && (p_hi - key0 < s.window || key0 + WM_KEYS <= s.keep_first);   // all visible to all rows
-        const bool beyond = p_lo - (key0 + WM_KEYS - 1) >= s.n_bias - 1;
-        float mx[2] = {-INFINITY, -INFINITY};
+        float mx = m;
+        {
+            const bool beyond = p_lo - (key0 + WM_KEYS - 1) >= s.n_bias - 1;         // one bias for every distance of the tile
+            const float* bt = bias + (pos - key0 - t4 * 2);
 #pragma unroll
-        for (int x = 0; x < 4; ++x) {
-            const int k = x * 8 + t4 * 2;
-            const float2 iv = *reinterpret_cast<const float2*>(inv + k);
-#pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                const int hf = e >> 1, key = key0 + k + (e & 1), d = pos[hf] - key;
-                const float bv = beyond ? far[hf] : bias[hf][min(max(d, 0), s.n_bias - 1)];
-                float v = fmaf(sc[x][e], e & 1 ? iv.y : iv.x, bv);
-                if (!plain && !window_sees(s, pos[hf], key)) v = -INFINITY;
-                sc[x][e] = v;
-                mx[hf] = fmaxf(mx[hf], v);
+            for (int x = 0; x < 4; ++x) {
+                const float2 k2 = *reinterpret_cast<const float2*>(scale + x * 8 + t4 * 2);
+                sc[x][0] = fmaf(sc[x][0], k2.x, beyond ? far : bt[-x * 8]);
+                sc[x][1] = fmaf(sc[x][1], k2.y, beyond ? far : bt[-x * 8 - 1]);
             }
-        }
+            if (key0 + WM_KEYS - 1 > p_lo || !(p_hi - key0 < s.window || key0 + WM_KEYS <= s.keep_first)) {       // not all visible to all rows
 #pragma unroll
-        for (int hf = 0; hf < 2; ++hf) {
-            mx[hf] = fmaxf(mx[hf], __shfl_xor_sync(0xffffffffu, mx[hf], 1));
-            mx[hf] = fmaxf(mx[hf], __shfl_xor_sync(0xffffffffu, mx[hf], 2));
-            mx[hf] = fmaxf(mx[hf], m[hf]);
+                for (int x = 0; x < 4; ++x)
+#pragma unroll
+                    for (int e = 0; e < 2; ++e)
+                        if (!window_sees(s, pos, key0 + x * 8 + t4 * 2 + e)) sc[x][e] = -INFINITY;
+            }
+#pragma unroll
+            for (int x = 0; x < 4; ++x) mx = fmaxf(mx, fmaxf(sc[x][0], sc[x][1]));
+            mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
+            mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
         }
-        if (__any_sync(0xffffffffu, mx[0] > m[0] || mx[1] > m[1])) {
-            const float c0 = exp2_fast(m[0] - mx[0]), c1 = exp2_fast(m[1] - mx[1]);
-            l[0] *= c0;
-            l[1] *= c1;
-            m[0] = mx[0];
-            m[1] = mx[1];
+        if (__any_sync(0xffffffffu, mx > m)) {
+            const float c = exp2_fast(m - mx);
+            l *= c;
+            m = mx;
 #pragma unroll
             for (int x = 0; x < NO; ++x) {
-                acc[x][0] *= c0;
-                acc[x][1] *= c0;
-                acc[x][2] *= c1;
-                acc[x][3] *= c1;
+                acc[x][0] *= c;
+                acc[x][1] *= c;
+                acc[x][2] *= c;
+                acc[x][3] *= c;
             }
         }
-        uint32_t ph[2][4], pl[2][4];
+        uint32_t ph[4], pl[4];
 #pragma unroll
         for (int x = 0; x < 4; ++x) {
-            float p[4];
-#pragma unroll
-            for (int e = 0; e < 4; ++e) p[e] = exp2_fast(sc[x][e] - m[e >> 1]);
-            l[0] += p[0] + p[1];
-            l[1] += p[2] + p[3];
-            const uint32_t h0 = pack_bf16x2(p[0], p[1]), h1 = pack_bf16x2(p[2], p[3]);
-            ph[x >> 1][(x & 1) * 2] = h0;
-            ph[x >> 1][(x & 1) * 2 + 1] = h1;
-            pl[x >> 1][(x & 1) * 2] = pack_bf16x2(p[0] - bf16_lo(h0), p[1] - bf16_hi(h0));
-            pl[x >> 1][(x & 1) * 2 + 1] = pack_bf16x2(p[2] - bf16_lo(h1), p[3] - bf16_hi(h1));
+            const float p0 = exp2_fast(sc[x][0] - m), p1 = exp2_fast(sc[x][1] - m);
+            l += p0 + p1;
+            ph[x] = pack_bf16x2(p0, p1);
+            pl[x] = pack_bf16x2(p0 - bf16_lo(ph[x]), p1 - bf16_hi(ph[x]));
         }
-        const uint32_t vb = smem_u32(K + (lm * 8 + lr) * LD);
+        const uint32_t vb = K + (lm * 8 + lr) * 128;
 #pragma unroll
         for (int x = 0; x < NO; ++x) {
             uint32_t vf[4];
-            ldsm_x4_trans(vb + x * 16, vf);
-            mma_16816(acc[x], ph[0][0], ph[0][1], ph[0][2], ph[0][3], vf[0], vf[1]);
-            mma_16816(acc[x], ph[1][0], ph[1][1], ph[1][2], ph[1][3], vf[2], vf[3]);
-            mma_16816(acc[x], pl[0][0], pl[0][1], pl[0][2], pl[0][3], vf[0], vf[1]);
-            mma_16816(acc[x], pl[1][0], pl[1][1], pl[1][2], pl[1][3], vf[2], vf[3]);
+            ldsm_x4_trans(vb + (x >> 3) * WM_CHUNK + (((x & 7) ^ lr) << 4), vf);
+            mma_16816(acc[x], ph[0], pl[0], ph[1], pl[1], vf[0], vf[1]);
+            mma_16816(acc[x], ph[2], pl[2], ph[3], pl[3], vf[2], vf[3]);
         }
-        __syncwarp();                                        // (the next load refills this stage's predecessor only)
+        __syncwarp();                                        // every lane is done with the stage
+        if (lane == 0) load(stage, next);
+        if (++stage == STAGES) {
+            stage = 0;
+            phase ^= 1u;
+        }
     }
-    cp_async_wait_all();
     __syncwarp();
     // a warp's O and (m, l) per row; then the CTA's, then the cluster's
-    constexpr int OLD = NK * 16 + 4;
-    float* O = reinterpret_cast<float*>(ring);
-    float* ml = reinterpret_cast<float*>(wm_smem + WM_WARPS * SM::kRing);     // [warp][row][2], then the CTA's [row][2]
+    float* O = reinterpret_cast<float*>(gen + warp * SM::kRing);
+    float* ml = reinterpret_cast<float*>(gen + SM::kMl);     // [warp][row][2], then the CTA's [row][2]
+    l += __shfl_xor_sync(0xffffffffu, l, 1);
+    l += __shfl_xor_sync(0xffffffffu, l, 2);
 #pragma unroll
-    for (int hf = 0; hf < 2; ++hf) {
-        l[hf] += __shfl_xor_sync(0xffffffffu, l[hf], 1);
-        l[hf] += __shfl_xor_sync(0xffffffffu, l[hf], 2);
-        const int row = gr + hf * 8;
-#pragma unroll
-        for (int x = 0; x < NO; ++x) *reinterpret_cast<float2*>(O + row * OLD + x * 8 + t4 * 2) = make_float2(acc[x][hf * 2], acc[x][hf * 2 + 1]);
-        if (t4 == 0) {
-            ml[(warp * 16 + row) * 2] = m[hf];
-            ml[(warp * 16 + row) * 2 + 1] = l[hf];
-        }
+    for (int x = 0; x < NO; ++x) *reinterpret_cast<float2*>(O + gr * OLD + x * 8 + t4 * 2) = make_float2(acc[x][0] + acc[x][2], acc[x][1] + acc[x][3]);
+    if (t4 == 0) {
+        ml[(warp * WM_ROWS + gr) * 2] = m;
+        ml[(warp * WM_ROWS + gr) * 2 + 1] = l;
     }
     __syncthreads();
-    float* all = ml + WM_WARPS * 32;
-    if (threadIdx.x < 16) {                                  // one thread per row: the warps' weights, the CTA's sum
+    float* all = ml + WM_WARPS * WM_ROWS * 2;
+    if (threadIdx.x < WM_ROWS) {                             // one thread per row: the warps' weights, the CTA's sum
         float mm = -1e30f, ll = 0.0f;
-        for (int w = 0; w < WM_WARPS; ++w) mm = fmaxf(mm, ml[(w * 16 + threadIdx.x) * 2]);
+        for (int w = 0; w < WM_WARPS; ++w) mm = fmaxf(mm, ml[(w * WM_ROWS + threadIdx.x) * 2]);
         for (int w = 0; w < WM_WARPS; ++w) {
-            float* p = ml + (w * 16 + threadIdx.x) * 2;
+            float* p = ml + (w * WM_ROWS + threadIdx.x) * 2;
             const float c = exp2_fast(p[0] - mm);
             ll += c * p[1];
             p[0] = c;
@@ -258,27 +233,27 @@ __global__ void __launch_bounds__(WM_THREADS) window_attention_mma_kernel(const 
         all[threadIdx.x * 2 + 1] = ll;
     }
     __syncthreads();
-    float* mine = reinterpret_cast<float*>(wm_smem);         // the CTA's O, in the place of warp 0's
+    float* mine = reinterpret_cast<float*>(gen);             // the CTA's O, in the place of warp 0's
     for (int i = threadIdx.x; i < nrows * dim; i += WM_THREADS) {
-        const int row = i / dim, c = i - row * dim;
+        const int r = i / dim, c = i - r * dim;
         float v = 0.0f;
 #pragma unroll
-        for (int w = 0; w < WM_WARPS; ++w) v = fmaf(reinterpret_cast<const float*>(wm_smem + w * SM::kRing)[row * OLD + c], ml[(w * 16 + row) * 2], v);
-        mine[row * OLD + c] = v;
+        for (int w = 0; w < WM_WARPS; ++w) v = fmaf(reinterpret_cast<const float*>(gen + w * SM::kRing)[r * OLD + c], ml[(w * WM_ROWS + r) * 2], v);
+        mine[r * OLD + c] = v;
     }
     if (a.splits > 1) cluster_sync();
     else __syncthreads();
     for (int i = split * WM_THREADS + threadIdx.x; i < nrows * dim; i += a.splits * WM_THREADS) {
-        const int row = i / dim, c = i - row * dim, r = r0 + row, t = r / group, h = g * group + (r - t * group);
+        const int r = i / dim, c = i - r * dim, t = (r0 + r) / group, h = g * group + (r0 + r - t * group);
         float v, ll;
         if (a.splits == 1) {
-            v = mine[row * OLD + c];
-            ll = all[row * 2 + 1];
+            v = mine[r * OLD + c];
+            ll = all[r * 2 + 1];
         } else {
             float pm[WM_MAX_CLUSTER], mm = -1e30f;
 #pragma unroll
             for (int k = 0; k < WM_MAX_CLUSTER; ++k) {
-                pm[k] = k < a.splits ? wm_peer(all + row * 2, k) : -1e30f;
+                pm[k] = k < a.splits ? wm_peer(all + r * 2, k) : -1e30f;
                 mm = fmaxf(mm, pm[k]);
             }
             v = ll = 0.0f;
@@ -286,8 +261,8 @@ __global__ void __launch_bounds__(WM_THREADS) window_attention_mma_kernel(const 
             for (int k = 0; k < WM_MAX_CLUSTER; ++k)
                 if (k < a.splits) {
                     const float w = exp2_fast(pm[k] - mm);
-                    v = fmaf(w, wm_peer(mine + row * OLD + c, k), v);
-                    ll = fmaf(w, wm_peer(all + row * 2 + 1, k), ll);
+                    v = fmaf(w, wm_peer(mine + r * OLD + c, k), v);
+                    ll = fmaf(w, wm_peer(all + r * 2 + 1, k), ll);
                 }
         }
         const float f = sigmoid_f32(a.gate[(first + t) * a.ld_gate + h]) * s.out_scale / ll;
@@ -297,8 +272,9 @@ __global__ void __launch_bounds__(WM_THREADS) window_attention_mma_kernel(const 
 }
 
 template <int NK, int STAGES>
-cudaError_t wm_launch(const WmArgs& a, int tiles, cudaStream_t stream) {
-    const cudaError_t e = seq_smem(window_attention_mma_kernel<NK, STAGES>, WmSmem<NK, STAGES>::kTotal);
+cudaError_t wm_launch(const CUtensorMap& map, const WmArgs& a, int tiles, cudaStream_t stream) {
+    auto kernel = window_attention_mma_kernel<NK, STAGES>;
+    const cudaError_t e = seq_smem(kernel, WmSmem<NK, STAGES>::kTotal);
     if (e != cudaSuccess) return e;
     cudaLaunchConfig_t cfg = {};
     cfg.gridDim = dim3(a.splits * a.s.kv_heads * tiles, a.st.batch);
@@ -313,7 +289,7 @@ cudaError_t wm_launch(const WmArgs& a, int tiles, cudaStream_t stream) {
     attr[1].val.clusterDim.y = attr[1].val.clusterDim.z = 1;
     cfg.attrs = attr;
     cfg.numAttrs = a.splits > 1 ? 2 : 1;
-    return cudaLaunchKernelEx(&cfg, window_attention_mma_kernel<NK, STAGES>, a);
+    return cudaLaunchKernelEx(&cfg, kernel, map, a);
 }
 
 }  // namespace
@@ -322,15 +298,17 @@ bool window_mma_applies(const scr_window_shape& s) { return s.dim % 8 == 0 && s.
 
 int32_t window_mma_launch(scr_ctx* ctx, const scr_window_shape& s, const scr_step& st, const void* q, const void* cache, const float* key_scale,
                           const float* bias, const float* gate, int64_t ld_gate, void* out, int64_t ld_out, cudaStream_t stream) {
-    WmArgs a{s, st, (const bf16*)q, (const bf16*)cache, key_scale, bias, gate, ld_gate, (bf16*)out, ld_out, 1, ctx->dev_status};
+    WmArgs a{s, st, (const bf16*)q, key_scale, bias, gate, ld_gate, (bf16*)out, ld_out, 1, ctx->dev_status};
     if (st.max_kv <= 0 || st.batch > 65535) return scr_fail(ctx, SCR_E_SHAPE, "max_kv %d batch %d", st.max_kv, st.batch);
-    const int tiles = scr_ceil_div(st.max_count * (s.heads / s.kv_heads), 16);
-    // key shares: two CTAs per SM, at least two key tiles per warp
+    CUtensorMap map;
+    if (!window_map(&map, cache, s.dim, s.kv_heads, (uint64_t)s.num_blocks * s.block_size, WM_KEYS)) return scr_fail(ctx, SCR_E_CUDA, "window_attention_mma: tensor map");
+    const int tiles = scr_ceil_div(st.max_count * (s.heads / s.kv_heads), WM_ROWS);
+    // key shares: up to two CTAs per SM, at least one key tile per warp
     const long long seen = std::min<long long>(st.max_kv, (long long)s.window + s.keep_first + st.max_count);
     const long long ctas = (long long)tiles * s.kv_heads * st.batch, key_tiles = (seen + WM_KEYS - 1) / WM_KEYS;
-    while (a.splits < WM_MAX_CLUSTER && ctas * a.splits < 2ll * ctx->sm_count && key_tiles >= 2ll * WM_WARPS * a.splits) a.splits *= 2;
-    const cudaError_t e = s.dim <= 32 ? wm_launch<2, 4>(a, tiles, stream) : s.dim <= 64 ? wm_launch<4, 4>(a, tiles, stream)
-                        : s.dim <= 128 ? wm_launch<8, 3>(a, tiles, stream) : wm_launch<16, 2>(a, tiles, stream);
+    while (a.splits < WM_MAX_CLUSTER && ctas * a.splits <= ctx->sm_count && key_tiles >= 2ll * WM_WARPS * a.splits) a.splits *= 2;
+    const cudaError_t e = s.dim <= 32 ? wm_launch<2, 3>(map, a, tiles, stream) : s.dim <= 64 ? wm_launch<4, 3>(map, a, tiles, stream)
+                        : s.dim <= 128 ? wm_launch<8, 2>(map, a, tiles, stream) : wm_launch<16, 2>(map, a, tiles, stream);
     if (e != cudaSuccess) return scr_fail(ctx, SCR_E_CUDA, "window_attention_mma: %s", cudaGetErrorString(e));
     return scr_check_launch(ctx, "window_attention_mma");
 }

@@ -18,9 +18,6 @@
 namespace {
 
 constexpr int WF_THREADS = 320, WF_KEYS = 64, WF_MAX_STAGES = 6, WF_BIAS = 4096;      // bias entries kept in shared memory
-// beside them, so that no index needs a limit: distances that are not there yet (masked), and those of the last tile whose
-// distances differ
-constexpr int WF_BIAS_LO = 192, WF_BIAS_HI = 96;
 constexpr uint32_t WF_Q_CHUNK = 128 * 128, WF_K_CHUNK = WF_KEYS * 128;                // 64 dimensions of 128 query rows / 64 keys
 
 struct WfLayout {
@@ -31,7 +28,7 @@ struct WfLayout {
         WfLayout l{};
         l.chunks = (s.dim + 63) / 64;
         l.vp = (s.dim + 15) / 16 * 16;
-        l.bias_n = s.n_bias <= WF_BIAS ? WF_BIAS_LO + s.n_bias + WF_BIAS_HI : 0;
+        l.bias_n = s.n_bias <= WF_BIAS ? SCR_BIAS_LO + s.n_bias + SCR_BIAS_HI : 0;
         const uint32_t q = 2 * l.chunks * WF_Q_CHUNK, fixed = q + l.bias_n * 4 + 16 + 256 + 1024;
         l.stages = (int)std::min<uint32_t>(WF_MAX_STAGES, (226 * 1024 - fixed) / (l.k_bytes() + WF_KEYS * 4));
         l.k = q;
@@ -111,12 +108,13 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_co
         tmem_alloc(smem_u32((const void*)tmem_slot), 512);
         tmem_relinquish();
     }
-    const float* bias = a.bias + (size_t)head * s.n_bias;
+    const float* bias = a.bias + (size_t)head * (SCR_BIAS_LO + s.n_bias + SCR_BIAS_HI);
     if (L.bias_n) {                                          // (a constant of the model: no wait)
         float* dst = reinterpret_cast<float*>(gen + L.bias);
-        for (int i = threadIdx.x; i < L.bias_n; i += WF_THREADS) dst[i] = bias[min(max(i - WF_BIAS_LO, 0), s.n_bias - 1)];
-        bias = dst + WF_BIAS_LO;
+        for (int i = threadIdx.x; i < L.bias_n; i += WF_THREADS) dst[i] = bias[i];
+        bias = dst;
     }
+    bias += SCR_BIAS_LO;
     tc_fence_before();
     __syncthreads();
     tc_fence_after();
@@ -222,7 +220,7 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_co
                         v[i + 2] = fmaf(v[i + 2], iv.z, far);
                         v[i + 3] = fmaf(v[i + 3], iv.w, far);
                     }
-                } else if (L.bias_n) {
+                } else {
                     const float* bt = bias + (pos - key0);
 #pragma unroll
                     for (int i = 0; i < 64; i += 4) {
@@ -231,16 +229,6 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_co
                         v[i + 1] = fmaf(v[i + 1], iv.y, bt[-i - 1]);
                         v[i + 2] = fmaf(v[i + 2], iv.z, bt[-i - 2]);
                         v[i + 3] = fmaf(v[i + 3], iv.w, bt[-i - 3]);
-                    }
-                } else {
-                    const int d0 = pos - key0, top = s.n_bias - 1;
-#pragma unroll
-                    for (int i = 0; i < 64; i += 4) {
-                        const float4 iv = inv[i >> 2];
-                        v[i] = fmaf(v[i], iv.x, bias[min(max(d0 - i, 0), top)]);
-                        v[i + 1] = fmaf(v[i + 1], iv.y, bias[min(max(d0 - i - 1, 0), top)]);
-                        v[i + 2] = fmaf(v[i + 2], iv.z, bias[min(max(d0 - i - 2, 0), top)]);
-                        v[i + 3] = fmaf(v[i + 3], iv.w, bias[min(max(d0 - i - 3, 0), top)]);
                     }
                 }
                 if (key0 + WF_KEYS - 1 > w_lo || !(w_hi - key0 < s.window || key0 + WF_KEYS <= s.keep_first)) {
@@ -320,15 +308,6 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_co
     }
 }
 
-bool wf_map(CUtensorMap* map, const void* base, uint64_t dim, uint64_t heads, uint64_t rows, uint32_t box_rows) {
-    tc_encode_tiled_fn enc = tc_tensor_map_encoder();
-    if (!enc) return false;
-    const cuuint64_t dims[3] = {dim, heads, rows}, strides[2] = {dim * 2, dim * 2 * heads};
-    const cuuint32_t box[3] = {64, 1, box_rows}, one[3] = {1, 1, 1};
-    return enc(map, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(base), dims, strides, box, one, CU_TENSOR_MAP_INTERLEAVE_NONE,
-               CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
-}
-
 constexpr int WF_MIN_ROWS = 64;                              // rows of one sequence from which the prompt kernel pays
 
 }  // namespace
@@ -341,7 +320,7 @@ int32_t window_prefill_launch(scr_ctx* ctx, const scr_window_shape& s, const scr
                               const float* bias, const float* gate, int64_t ld_gate, void* out, int64_t ld_out, cudaStream_t stream) {
     const WfArgs a{WfLayout::of(s), s, st, key_scale, bias, gate, ld_gate, (bf16*)out, ld_out, ctx->dev_status};
     CUtensorMap qm, km;
-    if (!wf_map(&qm, q, s.dim, s.heads, st.rows, 128) || !wf_map(&km, cache, s.dim, s.kv_heads, (uint64_t)s.num_blocks * s.block_size, WF_KEYS))
+    if (!window_map(&qm, q, s.dim, s.heads, st.rows, 128) || !window_map(&km, cache, s.dim, s.kv_heads, (uint64_t)s.num_blocks * s.block_size, WF_KEYS))
         return scr_fail(ctx, SCR_E_CUDA, "window_prefill: tensor map");
     cudaError_t e = seq_smem(window_prefill_kernel, a.lay.total);
     if (e == cudaSuccess)

@@ -220,6 +220,14 @@ def distance_buckets(rows: int, far: float) -> List[int]:
     return out
 
 
+def distance_bias(rel: torch.Tensor, far: float) -> Tuple[torch.Tensor, int]:
+    """Bias of every head and distance from a table [rows, heads] of buckets, as `scr_window_attention` takes it (in powers of
+    two, padded on both sides), and how many distances it has."""
+    buckets = distance_buckets(int(rel.shape[0]), far)
+    padded = [buckets[0]] * _lib.BIAS_LO + buckets + [buckets[-1]] * _lib.BIAS_HI
+    return rel.float()[torch.tensor(padded, device=rel.device)].t().contiguous() * float(np.log2(np.e)), len(buckets)
+
+
 class WindowAttention:
     """Grouped-head attention over a sliding window and the sequence's first tokens.  Queries and keys pass a short causal
     convolution and an RMS norm over the whole projection, the values are the keys before that norm, a bias per head and
@@ -237,12 +245,12 @@ class WindowAttention:
             raise ValueError(f"{prefix}: values that are keys have their size, not {spec['vdim']}")
         take = lambda name: weights.take(f"{prefix}.{name}")
         self.qk, self.g, self.o = torch.cat([take("q"), take("k")]).to(dtype), take("g").to(dtype), take("o").to(dtype)
-        self.norm = torch.cat([take("q.norm"), take("k.norm")]).float().contiguous()
+        keys = take("k.norm").float().view(self.kv_heads, 1, self.dim).expand(-1, self.heads // self.kv_heads, -1)
+        self.norm = (take("q.norm").float() * keys.reshape(-1)).contiguous()       # a query times its head's key weights
         self.conv = torch.cat([take("q.conv"), take("k.conv")]).float().t().contiguous()
         if tuple(self.conv.shape) != (self.taps, self.channels):
             raise ValueError(f"{prefix}: convolution {tuple(self.conv.shape)}, the configuration says {(self.taps, self.channels)}")
-        rel = take("rel").float()
-        self.bias = rel[torch.tensor(distance_buckets(int(rel.shape[0]), float(spec["bias_max"])), device=rel.device)].t().contiguous() * float(np.log2(np.e))
+        self.bias, self.n_bias = distance_bias(take("rel"), float(spec["bias_max"]))
 
     @property
     def channels(self) -> int:
@@ -266,7 +274,7 @@ class WindowAttention:
                 torch.zeros((slots, max(1, self.taps - 1), self.channels), dtype=self.dtype, device=device))
 
     def shape(self, ctx: StepContext) -> "_lib.WindowShape":
-        return _lib.WindowShape(self.heads, self.kv_heads, self.dim, self.taps, self.window, self.keep_first, int(self.bias.shape[1]),
+        return _lib.WindowShape(self.heads, self.kv_heads, self.dim, self.taps, self.window, self.keep_first, self.n_bias,
                                 ctx.block_size, ctx.num_blocks, ctx.inputs.max_blocks, self.eps, self.scale, self.out_scale)
 
     def run(self, ctx: StepContext, bufs: Dict[str, torch.Tensor], memory, out: torch.Tensor) -> None:
