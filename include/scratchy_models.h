@@ -201,9 +201,9 @@ int32_t scr_window_attention(scr_ctx* ctx, int32_t dtype, const scr_window_shape
 
 /* ---- matrix memory with a constant decay per head (lightning attention) -----------------------------
  * S <- decay_h S + k v^T, o = S^T q.  proj (dtype, row stride ld): q [heads * dim] | k [heads * dim] | v [heads * vdim];
- * powers f32 [heads][SCR_DECAY_POWERS]: decay_h^n.  State per slot f32 [num_slots, heads, dim, vdim]; a sequence whose rows start
+ * powers f32 [heads][SCR_DECAY_POWERS]: decay_h^n for n = 0 .. 64, then what decay_h has beyond its f32 value.  State per slot f32 [num_slots, heads, dim, vdim]; a sequence whose rows start
  * at position 0 starts from zero whatever the slot holds.  out f32 [rows, heads * vdim]. */
-#define SCR_DECAY_POWERS 65
+#define SCR_DECAY_POWERS 66
 typedef struct scr_lightning_shape {
     int32_t heads, dim, vdim;
     float eps, out_scale;

@@ -140,6 +140,16 @@ def window_visible(T, size, keep_first):
     return (j <= i) & ((i - j < size) | (j < keep_first))
 
 
+def windowed_softmax(q, k, v, scale, bias, size, keep_first, first=0):
+    """One head: queries q at positions first, first + 1, ..., keys k and values v of positions 0, 1, ...; `bias` by distance."""
+    T = k.shape[0]
+    back = (first + np.arange(q.shape[0]))[:, None] - np.arange(T)[None, :]
+    seen = window_visible(T, size, keep_first)[first:first + q.shape[0]]
+    score = np.where(seen, q @ k.T * scale + bias[np.maximum(back, 0)], -np.inf)
+    p = np.exp(score - score.max(axis=1, keepdims=True))
+    return (p / p.sum(axis=1, keepdims=True)) @ v
+
+
 def window_attention(h, w, m, eps):
     """Grouped heads over a sliding window with kept first tokens.  Queries and keys pass a short convolution and an RMS norm
     over the whole projection; the values are the keys before that norm; a bias per distance and head joins the scores;
@@ -151,15 +161,10 @@ def window_attention(h, w, m, eps):
     q = (unit_rms(q, eps) * w["q.norm"]).reshape(T, H, dim)
     k = (unit_rms(k, eps) * w["k.norm"]).reshape(T, G, dim)
     rows = np.array([distance_bucket(n, w["rel"].shape[0], m["bias_max"]) for n in range(T)])
-    back = np.maximum(np.arange(T)[:, None] - np.arange(T)[None, :], 0)
-    seen = window_visible(T, m["mask"]["size"], m["mask"]["keep_first"])
     out = np.zeros((T, H, dim))
     for head in range(H):
         g = head // (H // G)
-        score = q[:, head] @ k[:, g].T * m["scale"] + w["rel"][rows[back], head]
-        score = np.where(seen, score, -np.inf)
-        p = np.exp(score - score.max(axis=1, keepdims=True))
-        out[:, head] = (p / p.sum(axis=1, keepdims=True)) @ v[:, g]
+        out[:, head] = windowed_softmax(q[:, head], k[:, g], v[:, g], m["scale"], w["rel"][rows, head], m["mask"]["size"], m["mask"]["keep_first"])
     out *= sigmoid(h @ w["g"].T)[:, :, None]
     return out.reshape(T, H * dim) @ w["o"].T
 
@@ -255,3 +260,7 @@ def vekurax(cfg, weights, tokens):
         x = x + y
         runs.append(x)
     return tanh_norm_of(weights, "final.norm")(x) @ embed.T, runs
+
+
+def model(cfg, weights, tokens):
+    return {"Vumipel": vumipel, "Vekurax": vekurax}[cfg["architecture"]](cfg, weights, tokens)

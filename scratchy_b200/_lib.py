@@ -135,7 +135,7 @@ class TapeLinear(ctypes.Structure):
 
 PART_STORE, PART_F32, PART_SILU, PART_GELU_GLU = 0, 1, 2, 3
 DENSE_PARTS = 6
-DECAY_POWERS = 65
+DECAY_POWERS = 66
 BIAS_LO, BIAS_HI = 192, 96
 
 

@@ -126,14 +126,12 @@ __device__ __forceinline__ void dg_parts32(const DenseEnds& e, int m, int n0, in
 #pragma unroll
     for (int j = 0; j < 16; ++j) {
         const int c = (j >> 3) * 16 + (j & 7);
-        if (n0 + c < N) dense_put_two<bf16>(e, m, 0, n0 + c, N, v[c], v[c + 8]);
+        if (n0 + c < N) dense_put_two<bf16, END_PARTS>(e, m, 0, n0 + c, N, v[c], v[c + 8]);
     }
 }
 
-// 32 consecutive columns n0.. of row m: the ends, with 16-byte stores where the destination allows
-__device__ __forceinline__ void dg_store32(const DenseEnds& e, int m, int g, int n0, int N, float (&v)[32]) {
-    if (e.residual) return dg_residual32(e, m, n0, N, v);
-    if (e.n_parts) return dg_parts32(e, m, n0, N, v);
+// A linear's own end, with 16-byte stores where the destination allows
+__device__ __forceinline__ void dg_own32(const DenseEnds& e, int m, int g, int n0, int N, const float (&v)[32]) {
     if (e.act) {
         // columns 0..7 gate, 8..15 up, 16..23 gate, 24..31 up -> channels c0 .. c0 + 16
         const int c0 = (n0 >> 4) * 8;
@@ -175,7 +173,15 @@ __device__ __forceinline__ void dg_store32(const DenseEnds& e, int m, int g, int
     }
 }
 
-template <int BN>
+// 32 consecutive columns n0.. of row m: the ends
+template <DenseEnd END>
+__device__ __forceinline__ void dg_store32(const DenseEnds& e, int m, int g, int n0, int N, float (&v)[32]) {
+    if constexpr (END == END_RESIDUAL) return dg_residual32(e, m, n0, N, v);
+    else if constexpr (END == END_PARTS) return dg_parts32(e, m, n0, N, v);
+    else dg_own32(e, m, g, n0, N, v);
+}
+
+template <int BN, DenseEnd END>
 __global__ void __launch_bounds__(DG_THREADS, 1)
 dense_gemm_kernel(const __grid_constant__ CUtensorMap x_map, const __grid_constant__ CUtensorMap w_map, int M, int N, int KT, int MT,
                   int NTB, int groups, int full, int ks_tail, float* __restrict__ slabs, DenseEnds ends, int* __restrict__ status) {
@@ -282,7 +288,7 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap x_map, const __grid_consta
                     float v[32];
 #pragma unroll
                     for (int j = 0; j < 32; ++j) v[j] = __uint_as_float(r[j]);
-                    dg_store32(ends, m, g, n0, N, v);
+                    dg_store32<END>(ends, m, g, n0, N, v);
                 }
             }
             tc_fence_before();
@@ -299,6 +305,7 @@ dense_gemm_kernel(const __grid_constant__ CUtensorMap x_map, const __grid_consta
 
 // Sums a split tile's partial tiles in order and applies the ends: one thread per row and 32 columns would leave most
 // of the GPU idle on few rows, so one thread takes a gate column and its up column (16-column runs: j and j + 8).
+template <DenseEnd END>
 __global__ void __launch_bounds__(256) dense_gemm_finish_kernel(const float* __restrict__ slabs, int ks_tail, int n_tail, int full, int MT,
                                                                 int NTB, int bn, int M, int N, DenseEnds ends) {
     pdl_trigger();
@@ -316,12 +323,7 @@ __global__ void __launch_bounds__(256) dense_gemm_finish_kernel(const float* __r
         a += src[(size_t)k * n_tail * tile_elems];
         b += src[(size_t)k * n_tail * tile_elems + 8];
     }
-    if (ends.residual) {
-        dense_put_residual<bf16>(ends, m, n, a);
-        if (n + 8 < N) dense_put_residual<bf16>(ends, m, n + 8, b);
-    } else {
-        dense_put_two<bf16>(ends, m, g, n, N, a, b);
-    }
+    dense_put_two<bf16, END>(ends, m, g, n, N, a, b);
 }
 
 bool dg_map(CUtensorMap* map, const void* base, uint64_t d0, uint64_t d1, uint64_t d2, uint64_t s1, uint64_t s2, uint32_t b1, uint32_t b2) {
@@ -334,23 +336,23 @@ bool dg_map(CUtensorMap* map, const void* base, uint64_t d0, uint64_t d1, uint64
                CU_TENSOR_MAP_SWIZZLE_128B, CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE) == CUDA_SUCCESS;
 }
 
-template <int BN>
+template <int BN, DenseEnd END>
 int32_t dg_launch(scr_ctx* ctx, const scr_dense& d, const DgPlan& p, float* slabs, cudaStream_t stream) {
     CUtensorMap x_map, w_map;
     const uint64_t xg = d.groups > 1 ? (uint64_t)d.x_group * 2 : (uint64_t)d.K * 2;
     if (!dg_map(&x_map, d.x, d.K, d.groups, d.M, xg, (uint64_t)d.ldx * 2, 1, 128) ||
         !dg_map(&w_map, d.w, d.K, d.N, d.groups, (uint64_t)d.K * 2, (uint64_t)d.N * d.K * 2, BN, 1))
         return scr_fail(ctx, SCR_E_CUDA, "dense_gemm: tensor map (M %d N %d K %d groups %d)", d.M, d.N, d.K, d.groups);
-    cudaError_t e = seq_smem(dense_gemm_kernel<BN>, DgSmem<BN>::kTotal);
+    cudaError_t e = seq_smem(dense_gemm_kernel<BN, END>, DgSmem<BN>::kTotal);
     if (e == cudaSuccess) {
         const int units = p.full + p.n_tail() * p.ks_tail;
-        e = launch_pdl(dense_gemm_kernel<BN>, dim3(std::min(units, ctx->sm_count)), dim3(DG_THREADS), DgSmem<BN>::kTotal, stream, x_map, w_map, d.M,
+        e = launch_pdl(dense_gemm_kernel<BN, END>, dim3(std::min(units, ctx->sm_count)), dim3(DG_THREADS), DgSmem<BN>::kTotal, stream, x_map, w_map, d.M,
                        d.N, scr_ceil_div(d.K, 64), p.mt, p.ntb, d.groups, p.full, p.ks_tail, slabs, dense_ends(d), ctx->dev_status);
     }
     if (e != cudaSuccess) return scr_fail(ctx, SCR_E_CUDA, "dense_gemm: %s", cudaGetErrorString(e));
     const int32_t st = scr_check_launch(ctx, "dense_gemm");
     if (st || p.ks_tail == 1) return st;
-    e = launch_pdl(dense_gemm_finish_kernel, dim3(p.n_tail() * (128 / (512 / BN))), dim3(256), 0, stream, (const float*)slabs, p.ks_tail, p.n_tail(),
+    e = launch_pdl(dense_gemm_finish_kernel<END>, dim3(p.n_tail() * (128 / (512 / BN))), dim3(256), 0, stream, (const float*)slabs, p.ks_tail, p.n_tail(),
                    p.full, p.mt, p.ntb, BN, d.M, d.N, dense_ends(d));
     if (e != cudaSuccess) return scr_fail(ctx, SCR_E_CUDA, "dense_gemm_finish: %s", cudaGetErrorString(e));
     return scr_check_launch(ctx, "dense_gemm_finish");
@@ -364,5 +366,12 @@ int32_t dense_gemm_launch(scr_ctx* ctx, const scr_dense& d, void* workspace, siz
     const DgPlan p = dg_plan(d.M, d.N, d.K, d.groups, ctx->sm_count);
     if (p.slab_floats() * sizeof(float) > workspace_bytes || (p.ks_tail > 1 && (!workspace || !scr_aligned16(workspace))))
         return scr_fail(ctx, SCR_E_WORKSPACE, "dense_gemm needs %zu bytes of workspace", p.slab_floats() * sizeof(float));
-    return p.bn == 256 ? dg_launch<256>(ctx, d, p, (float*)workspace, stream) : dg_launch<128>(ctx, d, p, (float*)workspace, stream);
+    float* slabs = (float*)workspace;
+#define DG_CASE(END) case END: return p.bn == 256 ? dg_launch<256, END>(ctx, d, p, slabs, stream) : dg_launch<128, END>(ctx, d, p, slabs, stream)
+    switch (dense_end(d)) {
+        DG_CASE(END_PARTS);
+        DG_CASE(END_RESIDUAL);
+        default: DG_CASE(END_OWN);
+    }
+#undef DG_CASE
 }

@@ -18,7 +18,7 @@ namespace {
 // (8 further on) belong to one thread.
 constexpr int PLAIN_T = 64, PLAIN_K = 16;
 
-template <typename T>
+template <typename T, DenseEnd END>
 __global__ void __launch_bounds__(256) dense_plain_kernel(const T* __restrict__ w, const T* __restrict__ x, long long ldx,
                                                           long long x_group, int M, int N, int K, DenseEnds ends) {
     __shared__ float xs[PLAIN_K][PLAIN_T + 4], ws[PLAIN_K][PLAIN_T + 4];
@@ -58,7 +58,7 @@ __global__ void __launch_bounds__(256) dense_plain_kernel(const T* __restrict__ 
         if (m >= M) continue;
 #pragma unroll
         for (int j = 0; j < 4; j += 2)
-            if (n0 + cbase + 8 * j < N) dense_put_two<T>(ends, m, g, n0 + cbase + 8 * j, N, acc[i][j], acc[i][j + 1]);
+            if (n0 + cbase + 8 * j < N) dense_put_two<T, END>(ends, m, g, n0 + cbase + 8 * j, N, acc[i][j], acc[i][j + 1]);
     }
 }
 
@@ -77,7 +77,7 @@ __device__ __forceinline__ uint32_t mv_cluster_rank() {
     return r;
 }
 
-template <int NT, int SLOTS>
+template <int NT, int SLOTS, DenseEnd END>
 __global__ void __launch_bounds__(MV_WARPS * 32, 2) dense_matvec_kernel(const bf16* __restrict__ w, const bf16* __restrict__ x,
                                                                         long long ldx, long long x_group, int M, int N, int K,
                                                                         int wpt, int cluster, DenseEnds ends) {
@@ -162,30 +162,31 @@ __global__ void __launch_bounds__(MV_WARPS * 32, 2) dense_matvec_kernel(const bf
         for (int c = 1; c < cluster; ++c) v += peers[c - 1][tile][r][m];
         return v;
     };
-    if (ends.act || ends.n_parts) {
+    if (END == END_PARTS || (END == END_OWN && ends.act)) {
         for (int i = threadIdx.x; i < tiles * 8 * M; i += MV_WARPS * 32) {
             const int r = i & 7, tile = (i >> 3) % tiles, m = (i >> 3) / tiles;
             const int n = (tile0 + tile) * 16 + r;
-            if (n < N) dense_put_two<bf16>(ends, m, grp, n, N, whole(tile, r, m), whole(tile, r + 8, m));
+            if (n < N) dense_put_two<bf16, END>(ends, m, grp, n, N, whole(tile, r, m), whole(tile, r + 8, m));
         }
     } else {
         for (int i = threadIdx.x; i < tiles * 16 * M; i += MV_WARPS * 32) {
             const int r = i & 15, tile = (i >> 4) % tiles, m = (i >> 4) / tiles;
             const int n = (tile0 + tile) * 16 + r;
-            if (n < N) dense_put<bf16>(ends, m, grp, n, whole(tile, r, m));
+            if (n < N) dense_put<bf16, END>(ends, m, grp, n, whole(tile, r, m));
         }
     }
 }
 
+template <DenseEnd END>
 int32_t matvec_launch(scr_ctx* ctx, const scr_dense& d, cudaStream_t stream) {
     const int units = (d.K + 63) / 64, tiles16 = (d.N + 15) / 16;
     // warps per tile: enough units of K for each, and enough CTAs to fill the GPU
     int wpt = 1;
     while (wpt < MV_WARPS && (units >= 4 * wpt || (units >= 2 * wpt && (tiles16 * d.groups * wpt) / MV_WARPS < 2 * ctx->sm_count))) wpt *= 2;
     const int blocks = scr_ceil_div(tiles16, MV_WARPS / wpt);
-    // few, long tiles: a cluster shares each, so that the SMs' shares come out even
+    // fewer, long tiles than SMs: a cluster shares each
     int cluster = 1;
-    while (cluster < MV_MAX_CLUSTER && blocks * d.groups * cluster < 2 * ctx->sm_count && units >= 16 * wpt * cluster) cluster *= 2;
+    while (cluster < MV_MAX_CLUSTER && blocks * d.groups * cluster < ctx->sm_count && units >= 16 * wpt * cluster) cluster *= 2;
     cudaLaunchConfig_t cfg = {};
     cfg.gridDim = dim3(blocks * cluster, d.groups);
     cfg.blockDim = dim3(MV_WARPS * 32);
@@ -201,8 +202,8 @@ int32_t matvec_launch(scr_ctx* ctx, const scr_dense& d, cudaStream_t stream) {
     const bf16 *w = (const bf16*)d.w, *x = (const bf16*)d.x;
     const long long ldx = d.ldx, xg = d.x_group;
     const DenseEnds e = dense_ends(d);
-    const cudaError_t err = d.M <= 8 ? cudaLaunchKernelEx(&cfg, dense_matvec_kernel<1, 3>, w, x, ldx, xg, d.M, d.N, d.K, wpt, cluster, e)
-                                     : cudaLaunchKernelEx(&cfg, dense_matvec_kernel<2, 2>, w, x, ldx, xg, d.M, d.N, d.K, wpt, cluster, e);
+    const cudaError_t err = d.M <= 8 ? cudaLaunchKernelEx(&cfg, dense_matvec_kernel<1, 3, END>, w, x, ldx, xg, d.M, d.N, d.K, wpt, cluster, e)
+                                     : cudaLaunchKernelEx(&cfg, dense_matvec_kernel<2, 2, END>, w, x, ldx, xg, d.M, d.N, d.K, wpt, cluster, e);
     if (err != cudaSuccess) return scr_fail(ctx, SCR_E_CUDA, "dense_matvec: %s", cudaGetErrorString(err));
     return scr_check_launch(ctx, "dense_matvec");
 }
@@ -210,7 +211,9 @@ int32_t matvec_launch(scr_ctx* ctx, const scr_dense& d, cudaStream_t stream) {
 template <typename T>
 int32_t plain_launch(scr_ctx* ctx, const scr_dense& d, cudaStream_t stream) {
     const dim3 grid(scr_ceil_div(d.N, PLAIN_T), scr_ceil_div(d.M, PLAIN_T), d.groups);
-    const cudaError_t err = launch_pdl(dense_plain_kernel<T>, grid, dim3(256), 0, stream, (const T*)d.w, (const T*)d.x,
+    const DenseEnd end = dense_end(d);
+    auto kernel = end == END_RESIDUAL ? dense_plain_kernel<T, END_RESIDUAL> : end == END_PARTS ? dense_plain_kernel<T, END_PARTS> : dense_plain_kernel<T, END_OWN>;
+    const cudaError_t err = launch_pdl(kernel, grid, dim3(256), 0, stream, (const T*)d.w, (const T*)d.x,
                                        (long long)d.ldx, (long long)d.x_group, d.M, d.N, d.K, dense_ends(d));
     if (err != cudaSuccess) return scr_fail(ctx, SCR_E_CUDA, "dense_plain: %s", cudaGetErrorString(err));
     return scr_check_launch(ctx, "dense_plain");
@@ -252,6 +255,7 @@ extern "C" int32_t scr_dense_linear(scr_ctx* ctx, int32_t dtype, const scr_dense
     if (dtype == SCR_DTYPE_F32) return plain_launch<float>(ctx, d, st);
     if (dtype != SCR_DTYPE_BF16) return scr_fail(ctx, SCR_E_DTYPE, "dtype %d", dtype);
     if (!rows_of_16_bytes(d)) return plain_launch<bf16>(ctx, d, st);
-    if (d.M <= 16) return matvec_launch(ctx, d, st);
+    if (d.M <= 16)
+        return d.residual ? matvec_launch<END_RESIDUAL>(ctx, d, st) : d.n_parts ? matvec_launch<END_PARTS>(ctx, d, st) : matvec_launch<END_OWN>(ctx, d, st);
     return dense_gemm_launch(ctx, d, workspace, workspace_bytes, st);
 }

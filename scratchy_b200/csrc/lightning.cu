@@ -1,4 +1,5 @@
-// Matrix memory with a constant decay per head (lightning attention): S <- d S + k v^T, o = S^T q, state and sums f32.
+// Matrix memory with a constant decay per head (lightning attention): S <- d S + k v^T, o = S^T q, state and sums f32.  A decay close
+// to one is applied thousands of times, so it comes as two f32 values.
 //
 //   lightning_recur_kernel    token by token: decoding, short portions, any sizes, both data types
 //   lightning_chunk.cu        bf16 prompts, 64 tokens at a time on the tensor cores
@@ -46,7 +47,7 @@ __global__ void __launch_bounds__(LR_T) lightning_recur_kernel(MemoryArgs a) {
             }
         }
     }
-    const float decay = a.powers[(size_t)h * SCR_DECAY_POWERS + 1];
+    const float decay = a.powers[(size_t)h * SCR_DECAY_POWERS + 1], rest = a.powers[(size_t)h * SCR_DECAY_POWERS + SCR_DECAY_POWERS - 1];
     pdl_wait();
     if (!ok) {
         if (count > 0 && tid == 0) atomicCAS(a.status, 0, SEQ_BAD_SLOT);
@@ -69,10 +70,10 @@ __global__ void __launch_bounds__(LR_T) lightning_recur_kernel(MemoryArgs a) {
         float4 o = make_float4(0, 0, 0, 0);
 #pragma unroll
         for (int i = 0; i < RPT; ++i) {
-            S[i].x = fmaf(k[i], v[0], decay * S[i].x);
-            S[i].y = fmaf(k[i], v[1], decay * S[i].y);
-            S[i].z = fmaf(k[i], v[2], decay * S[i].z);
-            S[i].w = fmaf(k[i], v[3], decay * S[i].w);
+            S[i].x = fmaf(decay, S[i].x, fmaf(rest, S[i].x, k[i] * v[0]));
+            S[i].y = fmaf(decay, S[i].y, fmaf(rest, S[i].y, k[i] * v[1]));
+            S[i].z = fmaf(decay, S[i].z, fmaf(rest, S[i].z, k[i] * v[2]));
+            S[i].w = fmaf(decay, S[i].w, fmaf(rest, S[i].w, k[i] * v[3]));
             o.x = fmaf(S[i].x, q[i], o.x);
             o.y = fmaf(S[i].y, q[i], o.y);
             o.z = fmaf(S[i].z, q[i], o.z);

@@ -167,30 +167,34 @@ __device__ __forceinline__ void dense_put_residual(const DenseEnds& e, int m, in
     *r = v;
     if (e.tanh_w) reinterpret_cast<T*>(e.y)[m * e.ldy + n] = from_f32<T>(fmaf(tanhf(e.tanh_alpha * v), e.tanh_w[n], e.tanh_b[n]));
 }
-template <typename T>
+// The three kinds of ends, an argument of the kernels' templates: a linear's own, several linears in one, the residual.
+enum DenseEnd { END_OWN, END_PARTS, END_RESIDUAL };
+static inline DenseEnd dense_end(const scr_dense& d) { return d.residual ? END_RESIDUAL : d.n_parts ? END_PARTS : END_OWN; }
+template <typename T, DenseEnd END>
 __device__ __forceinline__ void dense_put(const DenseEnds& e, int m, int g, int n, float v) {
-    if (e.residual) return dense_put_residual<T>(e, m, n, v);
-    if (e.n_parts) {
+    if constexpr (END == END_RESIDUAL) {
+        dense_put_residual<T>(e, m, n, v);
+    } else if constexpr (END == END_PARTS) {
         int start;
         const scr_dense_part& p = e.parts[dense_part(e, n, start)];
         const long long at = m * p.ld + n - start;
         if (p.kind == SCR_PART_F32) reinterpret_cast<float*>(p.y)[at] = v;
         else reinterpret_cast<T*>(p.y)[at] = from_f32<T>(p.kind == SCR_PART_SILU ? v * sigmoid_f32(v) : v);
-        return;
+    } else {
+        dense_put_own<T>(e, m, g, n, v);
     }
-    dense_put_own<T>(e, m, g, n, v);
 }
 // Columns n (n % 16 < 8) and n + 8 of N.  Where they are a gate and its up they become channel (n / 16) * 8 + n % 8.
-template <typename T>
+template <typename T, DenseEnd END>
 __device__ __forceinline__ void dense_put_two(const DenseEnds& e, int m, int g, int n, int N, float a, float b) {
-    if (e.act) {
+    if (END == END_OWN && e.act) {
         const int c = (n >> 4) * 8 + (n & 7);
         const float v = clamped_glu(a, b, e.limit, e.alpha);
         if (e.y_f32) reinterpret_cast<float*>(e.y)[m * e.ldy + c] = v;
         else reinterpret_cast<T*>(e.y)[m * e.ldy + c] = from_f32<T>(v);
         return;
     }
-    if (e.n_parts) {
+    if constexpr (END == END_PARTS) {
         int start;
         const scr_dense_part& p = e.parts[dense_part(e, n, start)];
         if (p.kind == SCR_PART_GELU_GLU) {
@@ -199,6 +203,6 @@ __device__ __forceinline__ void dense_put_two(const DenseEnds& e, int m, int g, 
             return;
         }
     }
-    dense_put<T>(e, m, g, n, a);
-    if (n + 8 < N) dense_put<T>(e, m, g, n + 8, b);
+    dense_put<T, END>(e, m, g, n, a);
+    if (n + 8 < N) dense_put<T, END>(e, m, g, n + 8, b);
 }

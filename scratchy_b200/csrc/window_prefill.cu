@@ -6,11 +6,12 @@
 // on one tile, the softmax warps of the other work.  It walks the key tiles that any of its rows sees, those of the kept
 // first tokens and those of the window; a query tile skips the ones none of its rows sees.  320 threads:
 //   warp 0       TMA: the query tiles once, then key tiles with their scales through a ring
-//   warp 1       owns TMEM; one thread issues, per key tile and query tile, O += P V of the tile before and S = Q K^T
-//   warps 2-5, 6-9   softmax of tile 0, tile 1 (thread = query row): S from TMEM, scales, bias and window in f32, P back to
-//                TMEM as a bf16 head and remainder (two products: the weights keep about 16 bits), O rescaled in TMEM
+//   warp 1       owns TMEM; one thread issues, per key tile, S = Q K^T of both query tiles, then O += P V of the key tile before
+//   warps 2-5, 6-9   softmax of tile 0, tile 1 (thread = query row): S from TMEM, scales, bias and window in f32, P in the place
+//                of S as a bf16 head and remainder (two products: the weights keep about 16 bits), O rescaled in TMEM
 //                only when the row maximum has grown by more than 2^8 over the reference the sums are kept in
-// TMEM per tile: S 64 columns, P 32 + 32, O 128.  Every wait is bounded (tc_common.cuh).
+// TMEM per tile: two S of 64 columns (the next one is ready when the softmax of one is done), O 128.  Every wait is bounded
+// (tc_common.cuh).
 #include "window.cuh"
 
 #include <algorithm>
@@ -64,10 +65,10 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_co
     auto q_full = [&]() { return bars; };
     auto k_full = [&](int i) { return bars + 8u * (1 + i); };
     auto k_empty = [&](int i) { return bars + 8u * (1 + WF_MAX_STAGES + i); };
-    auto s_full = [&](int t) { return bars + 8u * (1 + 2 * WF_MAX_STAGES + t); };
-    auto p_full = [&](int t) { return bars + 8u * (3 + 2 * WF_MAX_STAGES + t); };
-    auto o_full = [&](int t) { return bars + 8u * (5 + 2 * WF_MAX_STAGES + t); };
-    volatile uint32_t* tmem_slot = reinterpret_cast<volatile uint32_t*>(gen + L.bars + 8 * (7 + 2 * WF_MAX_STAGES));
+    auto s_full = [&](int t, int i) { return bars + 8u * (1 + 2 * WF_MAX_STAGES + 2 * t + (i & 1)); };        // i: the tile's i-th S
+    auto p_full = [&](int t, int i) { return bars + 8u * (5 + 2 * WF_MAX_STAGES + 2 * t + (i & 1)); };
+    auto pv_done = [&](int t) { return bars + 8u * (9 + 2 * WF_MAX_STAGES + t); };
+    volatile uint32_t* tmem_slot = reinterpret_cast<volatile uint32_t*>(gen + L.bars + 8 * (11 + 2 * WF_MAX_STAGES));
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int head = blockIdx.x, q0 = ((int)gridDim.y - 1 - (int)blockIdx.y) * 256, b = blockIdx.z;      // the longest first
     const int first = a.st.segs[b * 4], count = a.st.segs[b * 4 + 1], pos0 = a.st.segs[b * 4 + 2];
@@ -101,7 +102,10 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_co
     if (threadIdx.x == 0) {
         mbar_init(q_full(), 1);
         for (int i = 0; i < WF_MAX_STAGES; ++i) { mbar_init(k_full(i), 1); mbar_init(k_empty(i), 1); }
-        for (int t = 0; t < 2; ++t) { mbar_init(s_full(t), 1); mbar_init(p_full(t), 128); mbar_init(o_full(t), 1); }
+        for (int t = 0; t < 2; ++t) {
+            for (int i = 0; i < 2; ++i) { mbar_init(s_full(t, i), 1); mbar_init(p_full(t, i), 128); }
+            mbar_init(pv_done(t), 1);
+        }
         fence_mbar_init();
     }
     if (warp == 1) {
@@ -119,9 +123,7 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_co
     __syncthreads();
     tc_fence_after();
     const uint32_t tmem = *tmem_slot;
-    auto s_col = [&](int t) { return tmem + 256u * t; };
-    auto ph_col = [&](int t) { return tmem + 256u * t + 64u; };
-    auto pl_col = [&](int t) { return tmem + 256u * t + 96u; };
+    auto s_col = [&](int t, int i) { return tmem + 256u * t + 64u * (i & 1); };        // S, then P: 32 columns of heads, 32 of remainders
     auto o_col = [&](int t) { return tmem + 256u * t + 128u; };
     pdl_wait();
 
@@ -152,32 +154,33 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_co
         if (lane == 0) {
             const uint32_t s_desc = umma_idesc(1, 1, 128, WF_KEYS), o_desc = umma_idesc(1, 1, 128, (uint32_t)L.vp) | UMMA_B_MN_MAJOR;
             mbar_wait(q_full(), 0, a.status, TC_ERR_FULL_WAIT);
-            int ks = 0, prev = 0, done[2] = {0, 0};                                  // done: products P V issued for a query tile
+            int ks = 0, prev = 0, started[2] = {0, 0}, done[2] = {0, 0};             // S and P V issued for a query tile
             uint32_t kp = 0;
             for (int j = 0; j <= tiles.count; ++j) {
                 if (j < tiles.count) mbar_wait(k_full(ks), kp, a.status, TC_ERR_FULL_WAIT);
                 tc_fence_after();
+                for (int t = 0; t < 2; ++t) {                                        // (its S buffer: P V of two tiles before is issued)
+                    if (!active(t, j)) continue;
+                    for (int c = 0; c < L.chunks; ++c) {
+                        const uint64_t qd = umma_desc_k_sw128(base + (t * L.chunks + c) * WF_Q_CHUNK);
+                        const uint64_t kd = umma_desc_k_sw128(base + L.k + ks * L.k_bytes() + c * WF_K_CHUNK);
+#pragma unroll
+                        for (int k4 = 0; k4 < 4; ++k4) umma_f16(s_col(t, started[t]), qd + (uint64_t)(2 * k4), kd + (uint64_t)(2 * k4), s_desc, (c | k4) != 0);
+                    }
+                    umma_commit(s_full(t, started[t]));
+                    ++started[t];
+                }
                 for (int t = 0; t < 2; ++t) {
-                    if (active(t, j - 1)) {                                          // O += P(j - 1) V(j - 1)
-                        mbar_wait(p_full(t), (uint32_t)done[t] & 1u, a.status, TC_ERR_DEQ_WAIT);
-                        tc_fence_after();
-                        const uint64_t vd = umma_desc_mn_sw128(base + L.k + prev * L.k_bytes(), WF_K_CHUNK);
+                    if (!active(t, j - 1)) continue;                                 // O += P(j - 1) V(j - 1)
+                    const int i = done[t]++;
+                    mbar_wait(p_full(t, i), (uint32_t)(i >> 1) & 1u, a.status, TC_ERR_DEQ_WAIT);
+                    tc_fence_after();
+                    const uint64_t vd = umma_desc_mn_sw128(base + L.k + prev * L.k_bytes(), WF_K_CHUNK);
 #pragma unroll
-                        for (int k4 = 0; k4 < 4; ++k4) umma_f16_ta(o_col(t), ph_col(t) + 8u * k4, vd + (uint64_t)(128 * k4), o_desc, done[t] > 0 || k4 > 0);
+                    for (int k4 = 0; k4 < 4; ++k4) umma_f16_ta(o_col(t), s_col(t, i) + 8u * k4, vd + (uint64_t)(128 * k4), o_desc, i > 0 || k4 > 0);
 #pragma unroll
-                        for (int k4 = 0; k4 < 4; ++k4) umma_f16_ta(o_col(t), pl_col(t) + 8u * k4, vd + (uint64_t)(128 * k4), o_desc, 1);
-                        ++done[t];
-                        if (tiles.tile(j - 1) == own_last[t]) umma_commit(o_full(t));
-                    }
-                    if (active(t, j)) {
-                        for (int c = 0; c < L.chunks; ++c) {
-                            const uint64_t qd = umma_desc_k_sw128(base + (t * L.chunks + c) * WF_Q_CHUNK);
-                            const uint64_t kd = umma_desc_k_sw128(base + L.k + ks * L.k_bytes() + c * WF_K_CHUNK);
-#pragma unroll
-                            for (int k4 = 0; k4 < 4; ++k4) umma_f16(s_col(t), qd + (uint64_t)(2 * k4), kd + (uint64_t)(2 * k4), s_desc, (c | k4) != 0);
-                        }
-                        umma_commit(s_full(t));
-                    }
+                    for (int k4 = 0; k4 < 4; ++k4) umma_f16_ta(o_col(t), s_col(t, i) + 32u + 8u * k4, vd + (uint64_t)(128 * k4), o_desc, 1);
+                    umma_commit(pv_done(t));
                 }
                 if (j > 0) umma_commit(k_empty(prev));                               // both products of the tile before are issued
                 prev = ks;
@@ -196,13 +199,13 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_co
             if (active(t, j)) {
                 const int key0 = tiles.tile(j) * WF_KEYS;
                 mbar_wait(k_full(ks), kp, a.status, TC_ERR_FULL_WAIT);               // (long complete: the scales are read here too)
-                mbar_wait(s_full(t), (uint32_t)seen & 1u, a.status, TC_ERR_ACC_FULL);
+                mbar_wait(s_full(t, seen), (uint32_t)(seen >> 1) & 1u, a.status, TC_ERR_ACC_FULL);
                 tc_fence_after();
                 float v[64];
                 {
                     uint32_t r0[32], r1[32];
-                    tmem_ld_32x32(s_col(t) + lanes, r0);
-                    tmem_ld_32x32(s_col(t) + lanes + 32, r1);
+                    tmem_ld_32x32(s_col(t, seen) + lanes, r0);
+                    tmem_ld_32x32(s_col(t, seen) + lanes + 32, r1);
                     tmem_ld_wait();
 #pragma unroll
                     for (int i = 0; i < 32; ++i) {
@@ -246,7 +249,9 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_co
                     m_ref = fmaxf(m_ref, mx);
                 } else {
                     const bool grow = mx > m_ref + 8.0f;
-                    if (__any_sync(0xffffffffu, grow)) {                             // PV of the tiles before is complete (s_full)
+                    if (__any_sync(0xffffffffu, grow)) {
+                        mbar_wait(pv_done(t), (uint32_t)(seen - 1) & 1u, a.status, TC_ERR_ACC_FULL);
+                        tc_fence_after();
                         const float c = grow ? exp2_fast(m_ref - mx) : 1.0f;
                         if (grow) m_ref = mx;
                         l *= c;
@@ -270,17 +275,17 @@ window_prefill_kernel(const __grid_constant__ CUtensorMap q_map, const __grid_co
                     lo[i] = pack_bf16x2(p0 - bf16_lo(hi[i]), p1 - bf16_hi(hi[i]));
                 }
                 l += (sum[0] + sum[1]) + (sum[2] + sum[3]);
-                tmem_st_32x32(ph_col(t) + lanes, hi);
-                tmem_st_32x32(pl_col(t) + lanes, lo);
+                tmem_st_32x32(s_col(t, seen) + lanes, hi);
+                tmem_st_32x32(s_col(t, seen) + lanes + 32, lo);
                 tmem_st_wait();
                 tc_fence_before();
-                mbar_arrive(p_full(t));
+                mbar_arrive(p_full(t, seen));
                 ++seen;
             }
             if (++ks == L.stages) { ks = 0; kp ^= 1u; }
         }
         if (seen > 0) {
-            mbar_wait(o_full(t), 0, a.status, TC_ERR_ACC_FULL);
+            mbar_wait(pv_done(t), (uint32_t)(seen - 1) & 1u, a.status, TC_ERR_ACC_FULL);
             tc_fence_after();
             const float f = row < count ? sigmoid_f32(a.gate[(first + row) * a.ld_gate + head]) * s.out_scale / l : 0.0f;
             for (int c0 = 0; c0 < L.vp; c0 += 32) {

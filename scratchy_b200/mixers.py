@@ -290,6 +290,13 @@ class WindowAttention:
                                          int(out.stride(0)), stream))
 
 
+def decay_powers(decay: np.ndarray) -> torch.Tensor:
+    """f32 powers 0 .. 64 of every head's decay, and what the decay has beyond its f32 value."""
+    powers = decay[:, None] ** np.arange(_lib.DECAY_POWERS - 1)[None, :]
+    rest = decay - decay.astype(np.float32).astype(np.float64)
+    return torch.from_numpy(np.concatenate([powers, rest[:, None]], 1).astype(np.float32)).contiguous()
+
+
 class LightningAttention:
     """Linear attention with a constant decay per head: a matrix state in f32, one slot per sequence; the concatenated readouts
     pass one RMS norm and a sigmoid gate (times `out_scale`)."""
@@ -303,8 +310,7 @@ class LightningAttention:
         decay = np.asarray(spec["decay"], dtype=np.float64)
         if decay.shape != (self.heads,):
             raise ValueError(f"{prefix}: {decay.size} decays for {self.heads} heads")
-        powers = decay[:, None] ** np.arange(_lib.DECAY_POWERS)[None, :]
-        self.powers = torch.from_numpy(powers.astype(np.float32)).to(self.norm.device).contiguous()
+        self.powers = decay_powers(decay).to(self.norm.device)
 
     @property
     def out_features(self) -> int:

@@ -143,13 +143,17 @@ def side_weights(cfg, seed=0, bias_rows=10):
     return out
 
 
+def weights_of(cfg, seed=0):
+    return side_weights(cfg, seed) if cfg["architecture"] == "Vekurax" else random_weights(cfg, seed)
+
+
 def save_checkpoint(directory, cfg, weights):
     from scratchy_b200.weights import write_safetensors
     os.makedirs(directory, exist_ok=True)
     with open(os.path.join(directory, "config.json"), "w") as f:
         json.dump(cfg, f)
     write_safetensors(os.path.join(directory, "model.safetensors"),
-                      {k: ((v.view(np.uint32) >> 16).astype(np.uint16), "BF16") for k, v in weights.items()})
+                      {k: ((np.asarray(v, np.float32).view(np.uint32) >> 16).astype(np.uint16), "BF16") for k, v in weights.items()})
 
 
 def make_model(cfg, weights, dtype, **kw):

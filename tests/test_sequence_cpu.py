@@ -60,6 +60,50 @@ def test_attention_of_the_first_token_is_its_own_value():
     assert np.allclose(out[:1], want)
 
 
+def test_dynamic_tanh_and_gelu():
+    x = np.array([[0.0, 2.0, -1.0]])
+    assert np.allclose(plain.dynamic_tanh(x, 0.5, np.array([1.0, 2.0, 3.0]), np.array([0.1, 0.2, 0.3])), [[0.1, 2 * np.tanh(1.0) + 0.2, 3 * np.tanh(-0.5) + 0.3]])
+    assert np.allclose(plain.gelu_tanh(np.array([0.0, 1.0, -1.0, 10.0])), [0.0, 0.841192, -0.158808, 10.0], atol=1e-6)
+
+
+def test_convolution_ends_with_the_token_itself():
+    u = np.array([[1.0, 10.0], [2.0, 20.0], [3.0, 30.0]])
+    w = np.array([[0.5, 0.0, 1.0], [0.0, 2.0, 0.0]])
+    assert np.allclose(plain.causal_conv(u, w), [[1.0, 0.0], [2.0, 20.0], [3.5, 40.0]])
+
+
+def test_buckets_of_key_distances():
+    from scratchy_b200.mixers import distance_bias, distance_buckets
+    assert distance_buckets(8, 64)[:5] == [0, 1, 2, 3, 4]
+    assert [plain.distance_bucket(n, 8, 64) for n in (4, 7, 8, 15, 16, 31, 32, 63, 64, 1000)] == [4, 4, 5, 5, 6, 6, 7, 7, 7, 7]
+    for rows, far in ((8, 64), (16, 100), (32, 128), (7, 50), (2, 9), (6, 4), (10, 160), (24, 3000)):
+        t = distance_buckets(rows, far)
+        assert t[-1] == rows - 1 and all(a <= b for a, b in zip(t, t[1:])) and (len(t) == 1 or t[-2] < rows - 1)
+        assert all(t[min(n, len(t) - 1)] == plain.distance_bucket(n, rows, far) for n in range(0, 4000, 1 if far < 500 else 7))
+    assert distance_buckets(1, 20) == [0]
+    import torch
+    from scratchy_b200 import _lib
+    rel = torch.arange(16.0).reshape(8, 2)
+    bias, n = distance_bias(rel, 64)
+    assert n == 33 and bias.shape == (2, _lib.BIAS_LO + n + _lib.BIAS_HI)
+    assert torch.allclose(bias[1, _lib.BIAS_LO + 16] * np.log(2.0), rel[6, 1]) and torch.equal(bias[:, 0], bias[:, _lib.BIAS_LO]) and torch.equal(bias[:, -1], bias[:, _lib.BIAS_LO + n - 1])
+
+
+def test_windows_keep_the_first_tokens():
+    seen = plain.window_visible(7, 3, 2)
+    assert [seen[6].tolist(), seen[3].tolist(), seen[1].tolist()] == [[1, 1, 0, 0, 1, 1, 1], [1, 1, 1, 1, 0, 0, 0], [1, 1, 0, 0, 0, 0, 0]]
+    v = np.arange(7.0)[:, None]
+    out = plain.windowed_softmax(np.zeros((1, 1)), v, v, 1.0, np.zeros(7), 3, 2, first=6)
+    assert np.allclose(out, (0 + 1 + 4 + 5 + 6) / 5)
+    bias = np.array([0.0, 0, 0, 0, 0, 50.0, 0])                                # a distance of 5 stands out: key 1
+    assert np.allclose(plain.windowed_softmax(np.zeros((1, 1)), v, v, 1.0, bias, 3, 2, first=6), 1.0)
+
+
+def test_decayed_memory_forgets_at_its_rate():
+    q, k, v = np.ones((3, 1)), np.array([[1.0], [0.0], [2.0]]), np.array([[1.0, 4.0], [9.0, 9.0], [1.0, 0.0]])
+    assert np.allclose(plain.decayed_memory(q, k, v, 0.5), [[1.0, 4.0], [0.5, 2.0], [2.25, 1.0]])
+
+
 # ---------------------------------------------------------------------------------------- configuration and registry
 def test_runs_of_a_loop():
     from scratchy_b200.vumipel import VumipelConfig
@@ -72,6 +116,26 @@ def test_runs_of_a_loop():
     for bad in ((2, 2, 1), (0, 5, 1), (0, 1, 0)):
         with pytest.raises(ValueError):
             runs(bad)
+
+
+def test_layers_on_the_weights_of_earlier_ones():
+    from scratchy_b200.vekurax import VekuraxConfig
+    S = su.side_spec
+    cfg = VekuraxConfig.from_dict(su.side_config([S(size=9, keep_first=4), S(), S(weights_of=0), S(weights_of=2), S(weights_of=1)]))
+    assert cfg.owners() == [0, 1, 0, 0, 1] and (cfg.window, cfg.keep_first) == (24, 5)
+    for bad in (1, 2, -1):
+        with pytest.raises(ValueError):
+            VekuraxConfig.from_dict(su.side_config([S(), S(weights_of=bad)]))
+    with pytest.raises(ValueError, match="serial"):
+        VekuraxConfig.from_dict(su.side_config([{**S(), "type": "serial"}]))
+
+
+def test_every_design_has_the_kernels_it_needs_and_no_others():
+    from scratchy_b200 import build
+    assert set(build.DESIGNS) == set(registry.ARCHITECTURES) - {"LlamaForCausalLM"}
+    vek = set(build.LIBRARIES[build.design_path("Vekurax")])
+    assert set(build.MODELS_COMMON) < vek and "window_prefill.cu" in vek and not any(s.startswith(("latent", "mlstm", "fp8", "affine")) for s in vek)
+    assert vek < set(build.MODELS_SOURCES)
 
 
 def test_unknown_mixer_and_architecture_are_refused():
@@ -125,6 +189,35 @@ def test_sequence_table_hands_out_and_takes_back():
     assert t.free_blocks == 2 and t.free_slots == 1
     c = t.open("c")
     assert c.slot == a.slot and c.length == 0 and c.blocks == []
+
+
+def test_blocks_that_the_window_has_passed_go_back():
+    from scratchy_b200.sequences import NO_BLOCK
+    t = SequenceTable(8, 4, 2, window=6, keep_first=5)                         # the first two blocks stay
+    s = t.open("s")
+    t.extend(s, 17)
+    t.advance(s, 17)                                                           # the next token, 17, sees 12..17 and 0..4
+    assert len(s.blocks) == 5 and s.held == 4 and s.blocks[2] == NO_BLOCK and t.free_blocks == 4
+    for length in range(18, 60):
+        t.extend(s, 1)
+        t.advance(s, 1)
+        visible = {j // 4 for j in range(length + 1) if length - j < 6 or j < 5}
+        held = {i for i, b in enumerate(s.blocks) if b != NO_BLOCK}
+        assert visible - {length // 4} <= held <= visible | {length // 4 - 1} and s.held <= t.most_blocks(60, 1)
+        assert s.held + t.free_blocks == 8
+    t.close("s")
+    assert sorted(t._free_blocks) == list(range(8))
+    assert SequenceTable(8, 4, 1).most_blocks(60, 1) == 15 and t.most_blocks(9, 100) == 3 and t.most_blocks(1000, 8) == 2 + 4 + 1
+
+
+def test_generation_beyond_the_cache_with_a_window():
+    m = Recorder(num_blocks=9, block_size=4, max_sequences=3)
+    m.table = SequenceTable(9, 4, 3, window=6, keep_first=3)
+    prompts = [[1, 2, 3] * 10, [4] * 25, [5, 6]]
+    assert Engine(m, step_tokens=4).generate(prompts, 20) == [continue_alone(p, 20) for p in prompts]
+    assert m.table.free_blocks == 9
+    with pytest.raises(ValueError, match="do not fit"):
+        Engine(m, step_tokens=100).generate([[1] * 90], 6)                     # in one portion
 
 
 class Recorder:
