@@ -1466,6 +1466,14 @@ def run_sequence_kernels(device, model, peaks, context=2048):
 
     context_of = lambda *a: step_context(device, model, arena, *a)
     m = att[0]
+    for batch, count in ((1, 1), (32, 1), (1, 2048)):
+        sc = context_of(batch, count, context, count > 1)
+        T, low = batch * count, m.q_rank + m.row_size
+        d, cq, cache = torch.randn((T, low), device=device), torch.empty((T, m.q_rank), dtype=bf, device=device), torch.zeros((sc.num_blocks * sc.block_size, m.row_size), dtype=bf, device=device)
+        shape = m.shape(sc)
+        call = lambda: c.check(lib.scr_latent_prepare(c.handle, code, ctypes.byref(shape), ctypes.byref(sc.step), _ptr(d), low, _ptr(m.q_norm), _ptr(m.kv_norm), _ptr(m.cos),
+                                                      _ptr(m.sin), _ptr(cq), _ptr(cache), _stream(device)))
+        add("latent norms, rotation, cache append", _time_calls(device, [call] * 4, 10), None, T * (low * 4 + (m.q_rank + m.row_size) * 2), batch=batch, T=count)
     for batch in (1, 8, 32):
         sc = context_of(batch, 1, context, False)
         copies = max(2, (256 << 20) // (batch * context * m.row_size * 2))

@@ -237,90 +237,141 @@ __global__ void __launch_bounds__(512) window_prepare_kernel(scr_window_shape s,
         if (tid == i && rows[i].cache >= 0) key_scale[rows[i].cache] = sk[i] * s.scale * 1.4426950408889634f;
 }
 
-// Many rows: a CTA walks up to WP_WALK consecutive rows with the taps and the last projected values in registers, the next row's
-// values in flight; one barrier per row.
-constexpr int WP_WALK = 64;
+// 8 values as they are stored.
+template <typename T> struct Raw8;
+template <> struct Raw8<bf16> {
+    uint4 a;
+    __device__ __forceinline__ void load(const bf16* p) { a = *reinterpret_cast<const uint4*>(p); }
+    __device__ __forceinline__ void zero() { a = make_uint4(0, 0, 0, 0); }
+    __device__ __forceinline__ float at(int j) const {
+        const uint32_t w = j < 2 ? a.x : j < 4 ? a.y : j < 6 ? a.z : a.w;
+        return j & 1 ? bf16_hi(w) : bf16_lo(w);
+    }
+    __device__ __forceinline__ void store(bf16* p) const { *reinterpret_cast<uint4*>(p) = a; }
+};
+template <> struct Raw8<float> {
+    float4 a, b;
+    __device__ __forceinline__ void load(const float* p) {
+        a = *reinterpret_cast<const float4*>(p);
+        b = *reinterpret_cast<const float4*>(p + 4);
+    }
+    __device__ __forceinline__ void zero() { a = b = make_float4(0, 0, 0, 0); }
+    __device__ __forceinline__ float at(int j) const {
+        const float4 v = j < 4 ? a : b;
+        return (j & 3) == 0 ? v.x : (j & 3) == 1 ? v.y : (j & 3) == 2 ? v.z : v.w;
+    }
+    __device__ __forceinline__ void store(float* p) const {
+        *reinterpret_cast<float4*>(p) = a;
+        *reinterpret_cast<float4*>(p + 4) = b;
+    }
+};
+
+// Many rows: a CTA walks up to WP_WALK consecutive rows, WP_STEP at a time, with the taps and the last projected values in
+// registers; one barrier per step.
+constexpr int WP_WALK = 64, WP_STEP = 4;
 template <typename T, int TAPS>
 __global__ void __launch_bounds__(512) window_prepare_walk_kernel(scr_window_shape s, scr_step st, int per, const T* __restrict__ proj, long long ld,
                                                                   const float* __restrict__ conv, const float* __restrict__ norm, T* state,
                                                                   T* __restrict__ q, T* __restrict__ cache, float* __restrict__ key_scale, int* status) {
-    __shared__ float red[2][16][2];
+    constexpr int PAST = TAPS - 1;
+    __shared__ __align__(16) float red[2][16][2][WP_STEP];
     __shared__ PrepRow rows[WP_WALK];
     pdl_trigger();
     const int r0 = blockIdx.x * per, n = min(per, st.rows - r0), tid = threadIdx.x, nq = s.heads * s.dim, C = nq + s.kv_heads * s.dim, hist = s.taps - 1;
     for (int i = tid; i < n; i += blockDim.x) rows[i] = prep_row(s, st, r0 + i, status);
     const int c = tid * 8;
     const bool in = c < C, query = c < nq;
-    float w[TAPS][8], wn[8], u[TAPS][8], next[8];            // w[o], u[o]: of the token o before
+    float w[TAPS][8];                                        // w[o]: of the token o before
 #pragma unroll
     for (int o = 0; o < TAPS; ++o) {
 #pragma unroll
-        for (int j = 0; j < 8; ++j) w[o][j] = u[o][j] = 0.0f;
+        for (int j = 0; j < 8; ++j) w[o][j] = 0.0f;
         if (in && o <= hist) Vec<float, 8>::get(conv + (size_t)(hist - o) * C + c, w[o]);
     }
-    if (query) Vec<float, 8>::get(norm + c, wn);
+    Raw8<T> u[PAST + WP_STEP];                               // the rows of a step and the PAST before them
+#pragma unroll
+    for (int i = 0; i < PAST + WP_STEP; ++i) u[i].zero();
     __syncthreads();
     pdl_wait();
-    if (in) {
 #pragma unroll
-        for (int o = 1; o < TAPS; ++o)                       // the rows before the first one, where they are of this step
-            if (o <= hist && o <= rows[0].at) Vec<T, 8>::get(proj + (r0 - o) * ld + c, u[o - 1]);
-        Vec<T, 8>::get(proj + r0 * ld + c, next);
-    }
-    for (int i = 0; i < n; ++i) {
-        const PrepRow p = rows[i];
-        float acc[8], ss = 0.0f;
-        if (in) {
+    for (int o = 1; o < TAPS; ++o)                           // the rows before the first one, where they are of this step
+        if (in && o <= hist && o <= rows[0].at) u[PAST - o].load(proj + (r0 - o) * ld + c);
+    for (int i0 = 0; i0 < n; i0 += WP_STEP) {
+        float y[WP_STEP][8], ss[WP_STEP];
 #pragma unroll
-            for (int o = TAPS - 1; o > 0; --o)
+        for (int i = 0; i < WP_STEP; ++i)
+            if (in && i0 + i < n) u[PAST + i].load(proj + (r0 + i0 + i) * ld + c);
 #pragma unroll
-                for (int j = 0; j < 8; ++j) u[o][j] = u[o - 1][j];
+        for (int i = 0; i < WP_STEP; ++i) {
+            ss[i] = 0.0f;
+            if (!in || i0 + i >= n) continue;
+            const PrepRow p = rows[i0 + i];
 #pragma unroll
-            for (int j = 0; j < 8; ++j) u[0][j] = next[j];
-            if (i + 1 < n) Vec<T, 8>::get(proj + (r0 + i + 1) * ld + c, next);
-            if (p.at >= 0 && p.at < hist) {                  // close to its portion's start: what lies before it is in the state
+            for (int j = 0; j < 8; ++j) y[i][j] = 0.0f;
+            if (p.at >= hist) {
 #pragma unroll
-                for (int o = 1; o < TAPS; ++o)
+                for (int o = PAST; o >= 0; --o)
+#pragma unroll
+                    for (int j = 0; j < 8; ++j) y[i][j] = fmaf(w[o][j], u[PAST + i - o].at(j), y[i][j]);
+            } else if (p.at >= 0) {                          // close to its portion's start: what lies before it is in the state
+                T* old = state + (size_t)p.slot * hist * C + c;
+                Raw8<T> v[TAPS];
+#pragma unroll
+                for (int o = PAST; o >= 0; --o) {
+                    v[o] = u[PAST + i - o];
                     if (o > p.at) {
-                        const bool has = o <= hist && p.pos - o >= 0;
-                        float v[8];
-                        if (has) Vec<T, 8>::get(state + ((size_t)p.slot * hist + (hist - (o - p.at))) * C + c, v);
-#pragma unroll
-                        for (int j = 0; j < 8; ++j) u[o][j] = has ? v[j] : 0.0f;
+                        if (o <= hist && p.pos - o >= 0) v[o].load(old + (size_t)(hist - (o - p.at)) * C);
+                        else v[o].zero();
                     }
+#pragma unroll
+                    for (int j = 0; j < 8; ++j) y[i][j] = fmaf(w[o][j], v[o].at(j), y[i][j]);
+                }
+                if (p.count == 1) {                          // one token: the state moves along
+#pragma unroll
+                    for (int o = PAST; o > 0; --o)
+                        if (o <= hist) v[o - 1].store(old + (size_t)(hist - o) * C);
+                }
             }
 #pragma unroll
-            for (int j = 0; j < 8; ++j) acc[j] = 0.0f;
+            for (int j = 0; j < 8; ++j) ss[i] = fmaf(y[i][j], y[i][j], ss[i]);
+        }
 #pragma unroll
-            for (int o = TAPS - 1; o >= 0; --o)
+        for (int i = 0; i < PAST; ++i) u[i] = u[i + WP_STEP];
+        float (*sums)[2][WP_STEP] = red[(i0 / WP_STEP) & 1]; // (two sets: the next step's writers need not wait for the readers)
 #pragma unroll
-                for (int j = 0; j < 8; ++j) acc[j] = fmaf(w[o][j], u[o][j], acc[j]);
-#pragma unroll
-            for (int j = 0; j < 8; ++j) ss = fmaf(acc[j], acc[j], ss);
-            if (p.at >= 0 && p.count == 1) {                 // one token: the state moves along (its old rows have been read)
-#pragma unroll
-                for (int o = TAPS - 1; o > 0; --o)
-                    if (o <= hist) Vec<T, 8>::put(state + ((size_t)p.slot * hist + (hist - o)) * C + c, u[o - 1]);
+        for (int i = 0; i < WP_STEP; ++i) {
+            const float a = warp_sum(query ? ss[i] : 0.0f), b = warp_sum(query ? 0.0f : ss[i]);
+            if ((tid & 31) == 0) {
+                sums[tid >> 5][0][i] = a;
+                sums[tid >> 5][1][i] = b;
             }
         }
-        const float a = warp_sum(query ? ss : 0.0f), b = warp_sum(query ? 0.0f : ss);
-        if ((tid & 31) == 0) {
-            red[i & 1][tid >> 5][0] = a;
-            red[i & 1][tid >> 5][1] = b;
+        __syncthreads();
+        float inv[WP_STEP] = {0.0f, 0.0f, 0.0f, 0.0f};
+        static_assert(WP_STEP == 4, "a step's sums are one float4");
+        for (int k = 0; k < (int)blockDim.x / 32; ++k) {
+            const float4 v = *reinterpret_cast<const float4*>(sums[k][query ? 0 : 1]);
+            inv[0] += v.x;
+            inv[1] += v.y;
+            inv[2] += v.z;
+            inv[3] += v.w;
         }
-        __syncthreads();                                     // (two sets of sums: the next row's writers need not wait for the readers)
-        const bool key0 = c == nq;                           // the thread of the first key channels leaves the keys' scale
-        float sum = 0.0f;
-        for (int k = 0; k < (int)blockDim.x / 32; ++k) sum += red[i & 1][k][query ? 0 : 1];
-        if (!in || p.at < 0) continue;
-        const float inv = 1.0f / sqrtf(sum / float(query ? nq : C - nq) + s.eps);
-        if (query) {
+        float wn[8];
+        if (query) Vec<float, 8>::get(norm + c, wn);
 #pragma unroll
-            for (int j = 0; j < 8; ++j) acc[j] *= inv * wn[j];
-            Vec<T, 8>::put(q + (size_t)(r0 + i) * nq + c, acc);
-        } else if (p.cache >= 0) {
-            Vec<T, 8>::put(cache + p.cache * (C - nq) + (c - nq), acc);
-            if (key0) key_scale[p.cache] = inv * s.scale * 1.4426950408889634f;
+        for (int i = 0; i < WP_STEP; ++i) {
+            if (!in || i0 + i >= n) continue;
+            const PrepRow p = rows[i0 + i];
+            if (p.at < 0) continue;
+            const float f = 1.0f / sqrtf(inv[i] / float(query ? nq : C - nq) + s.eps);
+            if (query) {
+#pragma unroll
+                for (int j = 0; j < 8; ++j) y[i][j] *= f * wn[j];
+                Vec<T, 8>::put(q + (size_t)(r0 + i0 + i) * nq + c, y[i]);
+            } else if (p.cache >= 0) {
+                Vec<T, 8>::put(cache + p.cache * (C - nq) + (c - nq), y[i]);
+                if (c == nq) key_scale[p.cache] = f * s.scale * 1.4426950408889634f;         // (by the thread of the first key channels)
+            }
         }
     }
 }
@@ -432,7 +483,7 @@ int32_t prepare(scr_ctx* ctx, const scr_window_shape& s, const scr_step& st, con
         const bool two = C > 512 * 8;
         const int threads = two ? 512 : scr_ceil_div(C / 8, 32) * 32;
         if (!two && st.rows >= 2 * ctx->sm_count) {
-            const int per = std::min(WP_WALK, std::max(4, scr_ceil_div(st.rows, ctx->sm_count)));
+            const int per = std::min(WP_WALK, std::max(WP_STEP, scr_ceil_div(scr_ceil_div(st.rows, ctx->sm_count), WP_STEP) * WP_STEP));
             e = launch_pdl(window_prepare_walk_kernel<T, 4>, dim3(scr_ceil_div(st.rows, per)), dim3(threads), 0, stream, s, st, per, (const T*)proj, (long long)ld,
                            conv, norm, (T*)conv_state, (T*)q, (T*)cache, key_scale, ctx->dev_status);
         } else {
