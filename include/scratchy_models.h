@@ -1,6 +1,7 @@
 /*
- * scratchy_models.h — C ABI of the sequence-model kernels (sm_100a): full-precision linears, latent attention over a
- * paged cache, the matrix-memory recurrence, and the norms, embedding and sampling around them.
+ * scratchy_models.h — C ABI of the sequence-model kernels (sm_100a): full-precision linears, latent attention and
+ * sliding-window attention over a paged cache, matrix memories with gates or with a constant decay, and the norms,
+ * embedding and sampling around them.
  *
  * Built as `libscratchy_models.so`, which carries its own copy of the context functions of scratchy_cuda.h
  * (`scr_cuda_init`, `scr_device_status`, ...); a context belongs to the library that made it.  The conventions are
@@ -201,8 +202,9 @@ int32_t scr_window_attention(scr_ctx* ctx, int32_t dtype, const scr_window_shape
 
 /* ---- matrix memory with a constant decay per head (lightning attention) -----------------------------
  * S <- decay_h S + k v^T, o = S^T q.  proj (dtype, row stride ld): q [heads * dim] | k [heads * dim] | v [heads * vdim];
- * powers f32 [heads][SCR_DECAY_POWERS]: decay_h^n for n = 0 .. 64, then what decay_h has beyond its f32 value.  State per slot f32 [num_slots, heads, dim, vdim]; a sequence whose rows start
- * at position 0 starts from zero whatever the slot holds.  out f32 [rows, heads * vdim]. */
+ * powers f32 [heads][SCR_DECAY_POWERS]: decay_h^n for n = 0 .. 64, then what decay_h has beyond its f32 value.  State per
+ * slot f32 [num_slots, heads, dim, vdim]; a sequence whose rows start at position 0 starts from zero whatever the slot
+ * holds.  out f32 [rows, heads * vdim]. */
 #define SCR_DECAY_POWERS 66
 typedef struct scr_lightning_shape {
     int32_t heads, dim, vdim;

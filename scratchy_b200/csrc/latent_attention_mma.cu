@@ -34,7 +34,6 @@ struct LmSmem {
     }
 };
 
-
 // MT: 16-row tiles; NTW: 8-column tiles of the latent per warp (kv_rank <= 64 * NTW, kv_rank + rot_dim <= 64 * (NTW + 1))
 template <int MT, int NTW>
 __global__ void __launch_bounds__(LM_THREADS) latent_attention_mma_kernel(scr_latent_shape s, scr_step st, const bf16* __restrict__ q,
